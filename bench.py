@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine at the Qwen3-8B shape with random weights, on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--shape 8b|0.6b|32b] [--impl ours|reference]
-    python bench.py --design bozosun|sizizen|zerusun|vokepel [--size 1k|2k|4k]   (another design beside the Qwen3 layers of equal size; see below)
+    python bench.py --design bozosun|sizizen|zerusun|vokepel|noditar [--size 1k|2k|4k]   (another design beside the Qwen3 layers of equal size; see below)
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 from 2,048-token prefixes, timed on the
 device (CUDA events on the engine's stream) over exactly K decode steps after W warm-up steps, each step fed its
@@ -173,7 +173,22 @@ def vokepel_config(z):
             "logit_scale": 1.5, "logit_softcap": 40.0, "layers": layers, "loop": {"start": 1, "stop": 3, "times": 1}, "max_position": CONTEXT}
 
 
-DESIGN_CONFIGS = {"bozosun": bozosun_config, "sizizen": sizizen_config, "zerusun": zerusun_config, "vokepel": vokepel_config}
+def noditar_config(z):
+    """Four layers over a residual of four streams: attention through a latent of 512 without positions (heads of 128, a gate
+    per value), grouped-query attention with a distance bias, a sink and the same gate (heads of 128), and two state-space
+    layers of Mamba's second form (twice the width in heads of 64, 128 states, eight groups); a dense clamped unit in all
+    but the third, which has no feed-forward."""
+    latent = {"heads": z["heads"], "dim": z["dim"], "vdim": z["dim"], "kv_rank": 512, "scale": z["dim"] ** -0.5}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5}
+    ssm = {"heads": 2 * z["width"] // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    layers = [{"type": "latent_attention", "mixer": latent, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": dense},
+              {"type": "mamba2", "mixer": ssm, "mlp": None}, {"type": "mamba2", "mixer": ssm, "mlp": dense}]
+    return {"architecture": "Noditar", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "streams": 4, "layers": layers,
+            "max_position": CONTEXT}
+
+
+DESIGN_CONFIGS = {"bozosun": bozosun_config, "sizizen": sizizen_config, "zerusun": zerusun_config, "vokepel": vokepel_config, "noditar": noditar_config}
 
 
 def design_bench(args):
@@ -263,7 +278,7 @@ def main():
     ap.add_argument("--page-size", type=int, default=16, help="tokens per cache page (the benchmark's configuration has 16)")
     ap.add_argument("--step-options", default="", metavar="JSON",
                     help="kernel choices of the step, for comparing two forms of it on one box, e.g. '{\"norm_ahead\": \"off\"}'")
-    ap.add_argument("--design", default="", choices=["", "bozosun", "sizizen", "zerusun", "vokepel"],
+    ap.add_argument("--design", default="", choices=["", "bozosun", "sizizen", "zerusun", "vokepel", "noditar"],
                     help="instead of the headline workload: prefill and decode of this design at real layer sizes beside four "
                          "Qwen3 layers of equal size, with the time and roofline fraction of every kernel class")
     ap.add_argument("--size", default="4k", choices=sorted(DESIGN_SIZES), help="with --design: the layer sizes")

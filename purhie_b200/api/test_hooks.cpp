@@ -36,6 +36,7 @@ Json spec_json(const ModelSpec& spec) {
     j.set("vocab_size", (long long)spec.vocab_size);
     j.set("max_position", (long long)spec.max_position);
     j.set("position_columns", spec.position_columns);
+    if (spec.residual_lanes) j.set("residual_lanes", spec.residual_lanes);
     j.set("embedding", spec.embedding.to_json());
     Json layers = Json::array();
     for (const LayerSpec& l : spec.layers) {

@@ -336,6 +336,7 @@ void register_bozosun_architecture();
 void register_sizizen_architecture();
 void register_zerusun_architecture();
 void register_vokepel_architecture();
+void register_noditar_architecture();
 
 void register_builtin_architectures() {
     static std::once_flag once;
@@ -345,6 +346,7 @@ void register_builtin_architectures() {
         register_sizizen_architecture();
         register_zerusun_architecture();
         register_vokepel_architecture();
+        register_noditar_architecture();
     });
 }
 

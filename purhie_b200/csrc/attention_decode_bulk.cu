@@ -13,7 +13,8 @@
 // out-of-range coordinate (the copy engine fills zeros), scores of invisible keys are replaced by -inf, and the
 // value rows after the token's position inside its last page are zeroed in shared memory before P V, so
 // unwritten page slots may hold anything, NaN included.  Every mbarrier wait is bounded and reports through an
-// error word.  The math is that of attention_flash.cu's decode kernel.
+// error word.  A distance bias (a slope per query head) takes slope_h * (token - key) off the scaled scores; a gate (rows of
+// logits) multiplies the output by its sigmoid where it is stored or merged.  The math is that of attention_flash.cu's decode kernel.
 #include "attention_mma.cuh"
 #include "mbarrier.cuh"
 
@@ -53,7 +54,11 @@ struct BulkParams {
     float scale_log2;
     int* error_flag;
     const float* sink;             // [HQ] float32 or null: exp(sink) joins each head's denominator, once per row
+    const float* slopes;           // [HQ] float32 or null: taken off the scores per position of distance
+    const __nv_bfloat16* gate; long long gate_stride;      // rows of HQ * D logits (by token row), or null
 };
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + __expf(-x)); }
 
 struct Item {
     int i, t, g, split, z, lo, lo_page, b_first, b_last, n_blocks;
@@ -101,7 +106,7 @@ __host__ __device__ constexpr int bulk_smem_bytes(int D, int G, int stages) {
            (2 * stages + 4) * 8 + PAGE_CACHE * 4;
 }
 
-template <int D, int STAGES, int CTAS>
+template <int D, int STAGES, int CTAS, bool BIAS>
 __global__ void __launch_bounds__(BULK_THREADS, CTAS)
 attention_decode_bulk_kernel(const __grid_constant__ CUtensorMap map_kv, const BulkParams p) {
     constexpr int HALVES = D / 64;
@@ -286,6 +291,19 @@ attention_decode_bulk_kernel(const __grid_constant__ CUtensorMap map_kv, const B
 #pragma unroll
                 for (int i = 0; i < 4; ++i) o[dt][i] = 0.0f;
 
+            const float slope0 = BIAS ? p.slopes[it.g * G + min(r0, G - 1)] * LOG2E : 0.0f;
+            const float slope1 = BIAS ? p.slopes[it.g * G + min(r1, G - 1)] * LOG2E : 0.0f;
+            const float scale_log2 = BIAS ? 1.0f : p.scale_log2;
+            // (BIAS) the scores in log2 units, each row's share of the distance taken off
+            auto bias = [&](float (&s)[2][4], int key0) {
+                if constexpr (BIAS) {
+#pragma unroll
+                    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                        for (int i = 0; i < 4; ++i)
+                            s[nt][i] = fmaf(s[nt][i], p.scale_log2, (i < 2 ? slope0 : slope1) * (float)(key0 + nt * 8 + (lane & 3) * 2 + (i & 1) - it.z));
+                }
+            };
             // The scores of block j + 1 are computed in the same straight-line code as the softmax and P V of
             // block j, so that the scheduler can overlap the two dependency chains.
             const int nb = it.b_last - it.b_first + 1;
@@ -306,7 +324,8 @@ attention_decode_bulk_kernel(const __grid_constant__ CUtensorMap map_kv, const B
                     float s_next[2][4];
                     qk(smem_u32(kv + nstage * 2 * TILE), qf, s_next);
                     // not the item's last block: every key is at or before the token; only the window's start masks
-                    softmax_update<D, 16>(s_cur, key0, it.z, it.z, it.lo, it.lo, true, p.scale_log2, m, l, o);
+                    bias(s_cur, key0);
+                    softmax_update<D, 16>(s_cur, key0, it.z, it.z, it.lo, it.lo, true, scale_log2, m, l, o);
                     pv(st, s_cur, o);
 #pragma unroll
                     for (int nt = 0; nt < 2; ++nt)
@@ -322,7 +341,8 @@ attention_decode_bulk_kernel(const __grid_constant__ CUtensorMap map_kv, const B
                         }
                         __syncwarp();
                     }
-                    softmax_update<D, 16>(s_cur, key0, it.z, it.z, it.lo, it.lo, true, p.scale_log2, m, l, o);
+                    bias(s_cur, key0);
+                    softmax_update<D, 16>(s_cur, key0, it.z, it.z, it.lo, it.lo, true, scale_log2, m, l, o);
                     pv(st, s_cur, o);
                     if (tail) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // our zeros, before the next copy lands there
                 }
@@ -366,7 +386,9 @@ attention_decode_bulk_kernel(const __grid_constant__ CUtensorMap map_kv, const B
                 const int h = it.g * G + r;
                 if (p.splits == 1) {
                     if (p.sink) ll += exp2f(p.sink[h] * LOG2E - use);
-                    p.out[((size_t)it.t * p.HQ + h) * D + d] = __float2bfloat16_rn(ll == 0.0f ? 0.0f : acc / ll);
+                    float v = ll == 0.0f ? 0.0f : acc / ll;
+                    if (p.gate) v *= sigmoid_f(__bfloat162float(p.gate[(size_t)it.t * p.gate_stride + (size_t)h * D + d]));
+                    p.out[((size_t)it.t * p.HQ + h) * D + d] = __float2bfloat16_rn(v);
                 } else {
                     const size_t slot = ((size_t)it.i * p.HQ + h) * p.splits + it.split;
                     p.part_o[slot * D + d] = acc;
@@ -381,7 +403,7 @@ attention_decode_bulk_kernel(const __grid_constant__ CUtensorMap map_kv, const B
 template <int D>
 __global__ void attention_combine_bulk_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                               const int32_t* __restrict__ row_list, __nv_bfloat16* __restrict__ out, int HQ, int splits,
-                                              const float* __restrict__ sink) {
+                                              const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, long long gate_stride) {
     // One block per (row, head), a thread per element of the head.  Lane s of every warp fetches the maximum and sum
     // of split s, so that the weights of 32 splits cost one round trip, and the partial outputs are fetched eight
     // splits at a time; the sums run over the splits in ascending order whatever the block's shape.
@@ -420,7 +442,9 @@ __global__ void attention_combine_bulk_kernel(const float* __restrict__ part_o, 
         }
     }
     if (sink) ll += exp2f(sink[h] * LOG2E - use);           // the sink counts once, after the splits are merged
-    out[((size_t)t * HQ + h) * D + d] = __float2bfloat16_rn(ll == 0.0f ? 0.0f : acc / ll);
+    float v = ll == 0.0f ? 0.0f : acc / ll;
+    if (gate) v *= sigmoid_f(__bfloat162float(gate[(size_t)t * gate_stride + (size_t)h * D + d]));
+    out[((size_t)t * HQ + h) * D + d] = __float2bfloat16_rn(v);
 }
 
 int sm_count() {
@@ -477,10 +501,10 @@ bool make_page_map(CUtensorMap* out, const void* k_base, long long kv_stride_byt
     return true;
 }
 
-template <int D, int STAGES, int CTAS>
+template <int D, int STAGES, int CTAS, bool BIAS>
 int launch_config(const CUtensorMap& mkv, const BulkParams& p, int bytes, int max_ctas, cudaStream_t stream) {
     static int configured = 0;
-    auto kernel = attention_decode_bulk_kernel<D, STAGES, CTAS>;
+    auto kernel = attention_decode_bulk_kernel<D, STAGES, CTAS, BIAS>;
     if (configured < bytes) {
         if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) != cudaSuccess)
             return fail(PH_ERR_LAUNCH, "attention_decode_bulk: cannot reserve %d bytes of shared memory", bytes);
@@ -493,32 +517,33 @@ int launch_config(const CUtensorMap& mkv, const BulkParams& p, int bytes, int ma
     launch_overlapped(kernel, dim3(grid), dim3(BULK_THREADS), (size_t)bytes, stream, mkv, p);
     if (p.splits > 1)
         launch_overlapped(attention_combine_bulk_kernel<D>, dim3(p.n_rows, p.HQ), dim3(D < 128 ? D : 128), 0, stream,
-                          (const float*)p.part_o, (const float*)p.part_ml, p.row_list, p.out, p.HQ, p.splits, p.sink);
+                          (const float*)p.part_o, (const float*)p.part_ml, p.row_list, p.out, p.HQ, p.splits, p.sink, p.gate, p.gate_stride);
     return check_launch("attention_decode_bulk");
 }
 
 // Two CTAs per SM with three stages each when that fits the SM's shared memory, else two stages each, else one
 // CTA with four stages: what counts is warps per SM (the consumers wait on dependent tensor-core instructions)
 // and enough copies in flight.
-template <int D> int launch_bulk(const CUtensorMap& mkv, const BulkParams& p, int max_ctas, cudaStream_t stream) {
+template <int D, bool BIAS> int launch_bulk(const CUtensorMap& mkv, const BulkParams& p, int max_ctas, cudaStream_t stream) {
     const int G = p.HQ / p.HKV;
     constexpr int SM_BYTES = 227 * 1024;
     const int b3 = bulk_smem_bytes(D, G, 3), b2 = bulk_smem_bytes(D, G, 2), b4 = bulk_smem_bytes(D, G, 4);
-    if (2 * (b3 + 1024) <= SM_BYTES) return launch_config<D, 3, 2>(mkv, p, b3, max_ctas, stream);
-    if (2 * (b2 + 1024) <= SM_BYTES) return launch_config<D, 2, 2>(mkv, p, b2, max_ctas, stream);
-    return launch_config<D, 4, 1>(mkv, p, b4, max_ctas, stream);
+    if (2 * (b3 + 1024) <= SM_BYTES) return launch_config<D, 3, 2, BIAS>(mkv, p, b3, max_ctas, stream);
+    if (2 * (b2 + 1024) <= SM_BYTES) return launch_config<D, 2, 2, BIAS>(mkv, p, b2, max_ctas, stream);
+    return launch_config<D, 4, 1, BIAS>(mkv, p, b4, max_ctas, stream);
 }
 
 }  // namespace
 
 // num_pages: pages of the pool that k_base / v_base belong to (the copy engine needs the extent it may address).
-// sink: [HQ] float32 or null.
-PH_EXPORT int ph_attention_decode_bulk_sink(const void* q, const void* k_base, const void* v_base, long long page_stride,
-                                            int page_size, int num_pages, const int32_t* block_table, int table_stride,
-                                            const int32_t* row_list, int n_rows, const int32_t* row_seg,
-                                            const int32_t* positions, float* part_o, float* part_ml, void* out, int HQ,
-                                            int HKV, int D, int splits, int window, int chunk, float scale, int max_ctas,
-                                            int* error_flag, const float* sink, cudaStream_t stream) {
+// sink, slopes: [HQ] float32 or null.  gate: rows of HQ * D bfloat16 logits, gate_stride elements apart, or null.
+PH_EXPORT int ph_attention_decode_bulk_biased(const void* q, const void* k_base, const void* v_base, long long page_stride,
+                                              int page_size, int num_pages, const int32_t* block_table, int table_stride,
+                                              const int32_t* row_list, int n_rows, const int32_t* row_seg,
+                                              const int32_t* positions, float* part_o, float* part_ml, void* out, int HQ,
+                                              int HKV, int D, int splits, int window, int chunk, float scale, int max_ctas,
+                                              int* error_flag, const float* sink, const float* slopes, const void* gate,
+                                              long long gate_stride, cudaStream_t stream) {
     if (!q || !k_base || !v_base || !block_table || !row_seg || !positions || !out || !error_flag || n_rows < 0 ||
         HQ < 1 || HKV < 1 || HQ % HKV || page_size < 1 || num_pages < 1 || window < 0 || chunk < 0 || splits < 1 ||
         (splits > 1 && (!part_o || !part_ml)))
@@ -549,7 +574,20 @@ PH_EXPORT int ph_attention_decode_bulk_sink(const void* q, const void* k_base, c
     p.row_list = row_list; p.row_seg = row_seg; p.positions = positions; p.part_o = part_o; p.part_ml = part_ml;
     p.out = (__nv_bfloat16*)out; p.n_rows = n_rows; p.HQ = HQ; p.HKV = HKV; p.splits = splits; p.window = window; p.chunk = chunk;
     p.scale_log2 = scale * LOG2E; p.error_flag = error_flag; p.sink = sink;
-    return D == 64 ? launch_bulk<64>(mkv, p, max_ctas, stream) : launch_bulk<128>(mkv, p, max_ctas, stream);
+    p.slopes = slopes; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride;
+    if (slopes) return D == 64 ? launch_bulk<64, true>(mkv, p, max_ctas, stream) : launch_bulk<128, true>(mkv, p, max_ctas, stream);
+    return D == 64 ? launch_bulk<64, false>(mkv, p, max_ctas, stream) : launch_bulk<128, false>(mkv, p, max_ctas, stream);
+}
+
+PH_EXPORT int ph_attention_decode_bulk_sink(const void* q, const void* k_base, const void* v_base, long long page_stride,
+                                            int page_size, int num_pages, const int32_t* block_table, int table_stride,
+                                            const int32_t* row_list, int n_rows, const int32_t* row_seg,
+                                            const int32_t* positions, float* part_o, float* part_ml, void* out, int HQ,
+                                            int HKV, int D, int splits, int window, int chunk, float scale, int max_ctas,
+                                            int* error_flag, const float* sink, cudaStream_t stream) {
+    return ph_attention_decode_bulk_biased(q, k_base, v_base, page_stride, page_size, num_pages, block_table, table_stride, row_list, n_rows,
+                                           row_seg, positions, part_o, part_ml, out, HQ, HKV, D, splits, window, chunk, scale, max_ctas,
+                                           error_flag, sink, nullptr, nullptr, 0, stream);
 }
 
 PH_EXPORT int ph_attention_decode_bulk(const void* q, const void* k_base, const void* v_base, long long page_stride,

@@ -14,6 +14,8 @@
 // cut into steps or on what else is in the batch.
 // A sink (one float32 number per query head, or none) is one more term exp(sink) in the softmax's denominator: it has no
 // key and no value, is not scaled, and counts once whatever the window holds.
+// A distance bias (one slope per query head, or none) takes slope_h * (z - p) off the scaled score of the key at p.  A gate
+// (rows of HQ * DV logits, or none) multiplies the output by sigmoid(gate), element by element.
 // Formulas (reference): src/qwen_ops.cpp:26-51 (scores * scale, max-subtracted softmax, weighted sum of
 // V; query head h uses kv head h / (HQ / HKV)); window: src/attention.h:73.
 #include "common.cuh"
@@ -33,7 +35,8 @@ __global__ void attention_generic_kernel(const TQ* __restrict__ q, const TKV* __
                                          const int32_t* __restrict__ block_table, int table_stride,
                                          const int32_t* __restrict__ row_seg, const int32_t* __restrict__ positions,
                                          TO* __restrict__ out, int T, int HQ, int HKV, int D, int window, float scale, int DV, int chunk, int VS,
-                                         const float* __restrict__ sink) {
+                                         const float* __restrict__ sink, const float* __restrict__ slopes, const TQ* __restrict__ gate,
+                                         long long gate_stride) {
     __shared__ float qs[WARPS][MAX_D];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -48,6 +51,7 @@ __global__ void attention_generic_kernel(const TQ* __restrict__ q, const TKV* __
     for (int d = lane; d < D; d += 32) qs[warp][d] = to_float<TQ>(qr[d]);
     __syncwarp();
 
+    const float slope = slopes ? slopes[h] : 0.0f;
     float m = -INFINITY, l = 0.0f;
     float acc[MAX_D / 32];
 #pragma unroll
@@ -65,6 +69,7 @@ __global__ void attention_generic_kernel(const TQ* __restrict__ q, const TKV* __
             float dot = 0.0f;
             for (int d = 0; d < D; ++d) dot += qs[warp][d] * to_float<TKV>(krow[d]);
             s = dot * scale;
+            if (slopes) s -= slope * (float)(z - p);
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float pexp = (p <= z) ? expf(s - m_new) : 0.0f;
@@ -97,17 +102,22 @@ __global__ void attention_generic_kernel(const TQ* __restrict__ q, const TKV* __
 #pragma unroll
     for (int i = 0; i < MAX_D / 32; ++i) {
         const int d = lane + 32 * i;
-        if (d < DV) o[d] = from_float<TO>(acc[i] * inv);
+        if (d >= DV) continue;
+        float v = acc[i] * inv;
+        if (gate) v *= 1.0f / (1.0f + expf(-to_float<TQ>(gate[(size_t)t * gate_stride + (size_t)h * DV + d])));
+        o[d] = from_float<TO>(v);
     }
 }
 
 }  // namespace
 
-PH_EXPORT int ph_attention_generic_sink(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype,
-                                        long long page_stride, int page_size, const int32_t* block_table,
-                                        int table_stride, const int32_t* row_seg, const int32_t* positions, void* out,
-                                        int out_dtype, int T, int HQ, int HKV, int D, int window, float scale, int DV,
-                                        int chunk, int v_stride, const float* sink, cudaStream_t stream) {
+// sink, slopes: [HQ] float32 or null.  gate: rows of HQ * DV logits in q's dtype, gate_stride elements apart, or null.
+PH_EXPORT int ph_attention_generic_biased(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype,
+                                          long long page_stride, int page_size, const int32_t* block_table,
+                                          int table_stride, const int32_t* row_seg, const int32_t* positions, void* out,
+                                          int out_dtype, int T, int HQ, int HKV, int D, int window, float scale, int DV,
+                                          int chunk, int v_stride, const float* sink, const float* slopes, const void* gate,
+                                          long long gate_stride, cudaStream_t stream) {
     if (!q || !k_base || !v_base || !block_table || !row_seg || !positions || !out || T < 0 || HQ < 1 || HKV < 1 ||
         D < 1 || page_size < 1 || window < 0 || chunk < 0 || !valid_dtype(q_dtype) || !valid_dtype(kv_dtype) ||
         !valid_dtype(out_dtype))
@@ -122,10 +132,20 @@ PH_EXPORT int ph_attention_generic_sink(const void* q, int q_dtype, const void* 
 #define LAUNCH(TQ, TKV, TO)                                                                                    \
     attention_generic_kernel<TQ, TKV, TO><<<blocks, WARPS * 32, 0, stream>>>(                                  \
         (const TQ*)q, (const TKV*)k_base, (const TKV*)v_base, page_stride, page_size, block_table, table_stride, \
-        row_seg, positions, (TO*)out, T, HQ, HKV, D, window, scale, DV, chunk, v_stride, sink)
+        row_seg, positions, (TO*)out, T, HQ, HKV, D, window, scale, DV, chunk, v_stride, sink, slopes, (const TQ*)gate, gate_stride)
     PH_DISPATCH(q_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, PH_DISPATCH(out_dtype, TO, LAUNCH(TQ, TKV, TO))));
 #undef LAUNCH
     return check_launch("attention_generic");
+}
+
+PH_EXPORT int ph_attention_generic_sink(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype,
+                                        long long page_stride, int page_size, const int32_t* block_table,
+                                        int table_stride, const int32_t* row_seg, const int32_t* positions, void* out,
+                                        int out_dtype, int T, int HQ, int HKV, int D, int window, float scale, int DV,
+                                        int chunk, int v_stride, const float* sink, cudaStream_t stream) {
+    return ph_attention_generic_biased(q, q_dtype, k_base, v_base, kv_dtype, page_stride, page_size, block_table, table_stride, row_seg,
+                                       positions, out, out_dtype, T, HQ, HKV, D, window, scale, DV, chunk, v_stride, sink, nullptr, nullptr,
+                                       0, stream);
 }
 
 PH_EXPORT int ph_attention_generic(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype,

@@ -21,6 +21,8 @@
 // nothing before its own block).  Pages past the tile's last token
 // come from an out-of-range coordinate (zeros), scores of invisible keys are replaced by -inf and value rows
 // after the last token inside its page are zeroed before P V, so unwritten page slots may hold anything.
+// A distance bias (a slope per head) takes slope_h * (row - key) off the scaled scores before the softmax; a gate (rows of
+// logits, a number per output element) multiplies the output by its sigmoid where the row is stored or merged.
 // Every mbarrier wait is bounded and reports through an error word; TMEM is freed on every path.
 // Math as in the reference's flash kernel: src/attention.hip:612-701; scale 1/sqrt(D): src/attention.cpp:197.
 #include "common.cuh"
@@ -75,7 +77,18 @@ struct Tc5Params {
     float* part_o;                 // [T][HQ][splits][D] unnormalised partial outputs
     float* part_ml;                // [T][HQ][splits][2] the exponent's reference and the sum of each partial
     const float* sink;             // [HQ] float32 or null: exp(sink) joins each head's denominator, once per row
+    const float* slopes;           // [HQ] float32 or null: taken off the scores per position of distance
+    const __nv_bfloat16* gate; long long gate_stride;      // rows of HQ * D logits, or null
 };
+
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+// eight outputs times the sigmoids of eight neighbouring logits
+__device__ __forceinline__ void gate8(const __nv_bfloat16* logits, float* v) {
+    float g[8];
+    load8(logits, g);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] *= sigmoid_fast(g[i]);
+}
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
@@ -187,6 +200,7 @@ __device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, u
         ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
 }
 
+template <bool BIAS>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, const Tc5Params p) {
@@ -350,6 +364,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
         const int z = z_first + min(r, n_rows - 1);      // rows past the portion repeat the last one; never stored
         const int lo = first_seen(z, p.window, p.chunk);
         const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
+        const float slope = BIAS ? p.slopes[h] * LOG2E : 0.0f;
         float m_ref = -INFINITY;                         // the maximum the exponents refer to
         float l = 0.0f;
         bool ok = true;
@@ -375,13 +390,20 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
                     if (key0 + 2 * j + 1 > z || key0 + 2 * j + 1 < lo) s[j].y = -INFINITY;
                 }
             }
+            if constexpr (BIAS) {                            // the scores in log2 units, the distance's share taken off
+                const float base = slope * (float)(key0 - z);
+                const float2 scale2 = make_float2(p.scale_log2, p.scale_log2), slope2 = make_float2(slope, slope), base2 = make_float2(base, base);
+#pragma unroll
+                for (int j = 0; j < BN / 2; ++j)
+                    s[j] = fma2(s[j], scale2, fma2(slope2, make_float2((float)(2 * j), (float)(2 * j + 1)), base2));
+            }
             float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
             for (int j = 0; j < BN / 2; j += 2) {
                 mx0 = fmaxf(mx0, fmaxf(s[j].x, s[j].y));
                 mx1 = fmaxf(mx1, fmaxf(s[j + 1].x, s[j + 1].y));
             }
-            const float mx = fmaxf(mx0, mx1) * p.scale_log2;       // the scale is positive: the maximum commutes with it
+            const float mx = BIAS ? fmaxf(mx0, mx1) : fmaxf(mx0, mx1) * p.scale_log2;       // the scale is positive: the maximum commutes with it
             // move the reference only when the maximum has outgrown it by more than RESCALE_STEP
             float corr = 1.0f;
             if (mx > m_ref + RESCALE_STEP || (m_ref == -INFINITY && mx > -INFINITY)) {
@@ -395,7 +417,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
             uint32_t packed[BN / 2];
 #pragma unroll
             for (int j = 0; j < BN / 2; j += 2) {
-                const float2 a0 = fma2(s[j], scale2, neg2), a1 = fma2(s[j + 1], scale2, neg2);
+                const float2 a0 = BIAS ? add2(s[j], neg2) : fma2(s[j], scale2, neg2), a1 = BIAS ? add2(s[j + 1], neg2) : fma2(s[j + 1], scale2, neg2);
                 const float2 e0 = make_float2(ex2(a0.x), ex2(a0.y)), e1 = make_float2(ex2(a1.x), ex2(a1.y));
                 sum_a = add2(sum_a, e0);
                 sum_b = add2(sum_b, e1);
@@ -452,13 +474,11 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 if (r < n_rows) {
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
-                        __nv_bfloat162 h0 = __floats2bfloat162_rn(__uint_as_float(raw[j]) * inv, __uint_as_float(raw[j + 1]) * inv);
-                        __nv_bfloat162 h1 = __floats2bfloat162_rn(__uint_as_float(raw[j + 2]) * inv, __uint_as_float(raw[j + 3]) * inv);
-                        __nv_bfloat162 h2 = __floats2bfloat162_rn(__uint_as_float(raw[j + 4]) * inv, __uint_as_float(raw[j + 5]) * inv);
-                        __nv_bfloat162 h3 = __floats2bfloat162_rn(__uint_as_float(raw[j + 6]) * inv, __uint_as_float(raw[j + 7]) * inv);
-                        uint4 v;
-                        v.x = *(uint32_t*)&h0; v.y = *(uint32_t*)&h1; v.z = *(uint32_t*)&h2; v.w = *(uint32_t*)&h3;
-                        *(uint4*)(dst + c * 32 + j) = v;
+                        float v[8];
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(raw[j + e]) * inv;
+                        if (p.gate) gate8(p.gate + (size_t)(row0 + first + r) * p.gate_stride + (size_t)h * D + c * 32 + j, v);
+                        store8(dst + c * 32 + j, v);
                     }
                 }
             }
@@ -501,7 +521,7 @@ __global__ void __launch_bounds__(128)
 attention_prefill_tc5_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                      const int32_t* __restrict__ seg_start, const int32_t* __restrict__ tile_seg,
                                      const int32_t* __restrict__ tile_first, __nv_bfloat16* __restrict__ out, int HQ, int splits,
-                                     const float* __restrict__ sink) {
+                                     const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, long long gate_stride) {
     pdl_launch_dependents();
     const int tile = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int seg = tile_seg[tile], first = tile_first[tile];
@@ -533,10 +553,12 @@ attention_prefill_tc5_combine_kernel(const float* __restrict__ part_o, const flo
     }
     if (sink && l != 0.0f) l += exp2f(sink[h] * LOG2E - m);      // the sink counts once, after the splits are merged
     const float inv = l == 0.0f ? 0.0f : 1.0f / l;        // a row with no visible key gives 0; NaN stays NaN
-    __nv_bfloat162 h0 = __floats2bfloat162_rn(acc.x * inv, acc.y * inv), h1 = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-    uint2 v;
-    v.x = *(uint32_t*)&h0; v.y = *(uint32_t*)&h1;
-    *(uint2*)(out + ((size_t)(row0 + first + r) * HQ + h) * D + lane * 4) = v;
+    float v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+    if (gate) {
+        const float4 g = load4(gate + (size_t)(row0 + first + r) * gate_stride + (size_t)h * D + lane * 4);
+        v[0] *= sigmoid_fast(g.x); v[1] *= sigmoid_fast(g.y); v[2] *= sigmoid_fast(g.z); v[3] *= sigmoid_fast(g.w);
+    }
+    store4(out + ((size_t)(row0 + first + r) * HQ + h) * D + lane * 4, v);
 }
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
@@ -586,13 +608,14 @@ PH_DEFINE_LAST_ERROR(ph_flash5)
 // for few tiles that look far back.  tile_seg / tile_first: the step's prompt portions cut into tiles
 // of 128 rows (segment, first row of the tile within the portion).  num_pages: pages of the pool that k_base /
 // v_base belong to.
-// sink: [HQ] float32 or null.
-PH_EXPORT int ph_attention_prefill_tc5_sink(const void* q, int T, const void* k_base, const void* v_base, long long page_stride,
-                                            int page_size, int num_pages, const int32_t* block_table, int table_stride,
-                                            const int32_t* seg_start, const int32_t* seg_ctx_len, const int32_t* tile_seg,
-                                            const int32_t* tile_first, int n_tiles, void* out, int HQ, int HKV, int head_dim,
-                                            int window, int chunk, float scale, int splits, float* part_o, float* part_ml,
-                                            int* error_flag, const float* sink, cudaStream_t stream) {
+// sink, slopes: [HQ] float32 or null.  gate: rows of HQ * 128 bfloat16 logits, gate_stride elements apart, or null.
+PH_EXPORT int ph_attention_prefill_tc5_biased(const void* q, int T, const void* k_base, const void* v_base, long long page_stride,
+                                              int page_size, int num_pages, const int32_t* block_table, int table_stride,
+                                              const int32_t* seg_start, const int32_t* seg_ctx_len, const int32_t* tile_seg,
+                                              const int32_t* tile_first, int n_tiles, void* out, int HQ, int HKV, int head_dim,
+                                              int window, int chunk, float scale, int splits, float* part_o, float* part_ml,
+                                              int* error_flag, const float* sink, const float* slopes, const void* gate,
+                                              long long gate_stride, cudaStream_t stream) {
     if (!q || !k_base || !v_base || !block_table || !seg_start || !seg_ctx_len || !tile_seg || !tile_first || !out ||
         !error_flag || T < 1 || n_tiles < 0 || HQ < 1 || HKV < 1 || HQ % HKV || num_pages < 1 || window < 0 || chunk < 0 || !(scale > 0.0f))
         return fail(PH_ERR_ARG, "attention_prefill_tc5: bad arguments (tiles %d, HQ %d, HKV %d)", n_tiles, HQ, HKV);
@@ -604,6 +627,7 @@ PH_EXPORT int ph_attention_prefill_tc5_sink(const void* q, int T, const void* k_
     if (n_tiles > 65535) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: %d tiles exceed the grid", n_tiles);
     if (splits < 1 || splits > MERGE_MAX || (splits > 1 && (!part_o || !part_ml || (((uintptr_t)part_o) & 15))))
         return fail(PH_ERR_ARG, "attention_prefill_tc5: %d splits need 16-byte aligned scratch for the partial results", splits);
+    if (gate && (gate_stride % 8 || ((uintptr_t)gate & 15))) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: the gate's rows must be 16-byte aligned");
     if (n_tiles == 0) return PH_OK;
     const long long rows_per_page = page_stride / D;
     const long long rows = (long long)(num_pages - 1) * rows_per_page + (long long)HKV * page_size;
@@ -626,17 +650,30 @@ PH_EXPORT int ph_attention_prefill_tc5_sink(const void* q, int T, const void* k_
     p.tile_seg = tile_seg; p.tile_first = tile_first; p.n_tiles = n_tiles; p.out = (__nv_bfloat16*)out;
     p.HQ = HQ; p.HKV = HKV; p.window = window; p.chunk = chunk; p.scale_log2 = scale * LOG2E; p.error_flag = error_flag;
     p.splits = splits; p.part_o = part_o; p.part_ml = part_ml; p.sink = sink;
+    p.slopes = slopes; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride;
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(attention_prefill_tc5_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess)
+        if (cudaFuncSetAttribute(attention_prefill_tc5_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(attention_prefill_tc5_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess)
             return fail(PH_ERR_LAUNCH, "attention_prefill_tc5: cannot reserve %d bytes of shared memory", SMEM_BYTES);
         configured = true;
     }
-    launch_overlapped(attention_prefill_tc5_kernel, dim3(HQ, n_tiles, splits), dim3(THREADS), (size_t)SMEM_BYTES, stream, mq, mk, mv, p);
+    launch_overlapped(slopes ? attention_prefill_tc5_kernel<true> : attention_prefill_tc5_kernel<false>, dim3(HQ, n_tiles, splits), dim3(THREADS), (size_t)SMEM_BYTES, stream, mq, mk, mv, p);
     if (splits > 1)
         launch_overlapped(attention_prefill_tc5_combine_kernel, dim3(n_tiles, HQ, BM / 4), dim3(128), 0, stream,
-                          (const float*)part_o, (const float*)part_ml, seg_start, tile_seg, tile_first, (__nv_bfloat16*)out, HQ, splits, sink);
+                          (const float*)part_o, (const float*)part_ml, seg_start, tile_seg, tile_first, (__nv_bfloat16*)out, HQ, splits, sink, p.gate, gate_stride);
     return check_launch("attention_prefill_tc5");
+}
+
+PH_EXPORT int ph_attention_prefill_tc5_sink(const void* q, int T, const void* k_base, const void* v_base, long long page_stride,
+                                            int page_size, int num_pages, const int32_t* block_table, int table_stride,
+                                            const int32_t* seg_start, const int32_t* seg_ctx_len, const int32_t* tile_seg,
+                                            const int32_t* tile_first, int n_tiles, void* out, int HQ, int HKV, int head_dim,
+                                            int window, int chunk, float scale, int splits, float* part_o, float* part_ml,
+                                            int* error_flag, const float* sink, cudaStream_t stream) {
+    return ph_attention_prefill_tc5_biased(q, T, k_base, v_base, page_stride, page_size, num_pages, block_table, table_stride, seg_start,
+                                           seg_ctx_len, tile_seg, tile_first, n_tiles, out, HQ, HKV, head_dim, window, chunk, scale, splits,
+                                           part_o, part_ml, error_flag, sink, nullptr, nullptr, 0, stream);
 }
 
 PH_EXPORT int ph_attention_prefill_tc5(const void* q, int T, const void* k_base, const void* v_base, long long page_stride,

@@ -9,7 +9,7 @@
 //   attention_talking     for the row at position z and every key p that it sees (first_seen(z) <= p <= z):
 //                             s_g = (q_g . k_kv(g)) * scale
 //                             s_g = cap * tanh(s_g / cap)                          (cap > 0)
-//                             s_g = s_g - r1_g * ln(1 + r2_g * (z - p))            (r1, r2 given)
+//                             s_g = s_g - r1_g * ln(1 + r2_g * (z - p))            (r1, r2 given; r1 alone: r1_g * (z - p))
 //                             s'_h = sum_g talk[h][g] * s_g                        (talk given: [HQ, HQ])
 //                         then a softmax over the seen keys per head h (with exp(sink_h) in the denominator when a sink
 //                         is given), o_h = sum_p w_hp v_kv(h)p, and o_h * sigmoid(gate_h) when a gate row is given.
@@ -81,7 +81,7 @@ __global__ void attention_talking_kernel(const TQ* __restrict__ q, const TKV* __
                 for (int d = 0; d < D; ++d) dot += qh[d] * to_float<TKV>(krow[d]);
                 float v = dot * scale;
                 if (cap > 0.0f) v = cap * tanhf(v / cap);
-                if (r1) v -= r1[h] * log1pf(r2[h] * (float)(z - p));
+                if (r1) v -= r1[h] * (r2 ? log1pf(r2[h] * (float)(z - p)) : (float)(z - p));
                 s[u] = v;
             }
         }
@@ -266,8 +266,8 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
 
 }  // namespace
 
-// gate: rows of HQ * DV logits, gate_stride elements apart, in gate_dtype (null: no gate).  cap 0: no cap.  r1, r2, talk,
-// sink: float32 per head ([HQ], [HQ], [HQ, HQ], [HQ]) or null.
+// gate: rows of HQ * DV logits, gate_stride elements apart, in gate_dtype (null: no gate).  cap 0: no cap.  r1 without r2: a
+// bias linear in the distance.  r1, r2, talk, sink: float32 per head ([HQ], [HQ], [HQ, HQ], [HQ]) or null.
 PH_EXPORT int ph_attention_talking(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype, long long page_stride,
                                    int page_size, const int32_t* block_table, int table_stride, const int32_t* row_seg,
                                    const int32_t* positions, void* out, int out_dtype, int T, int HQ, int HKV, int D, int DV, int window,
@@ -275,7 +275,7 @@ PH_EXPORT int ph_attention_talking(const void* q, int q_dtype, const void* k_bas
                                    const float* sink, const void* gate, int gate_dtype, long long gate_stride, cudaStream_t stream) {
     if (!q || !k_base || !v_base || !block_table || !row_seg || !positions || !out || T < 0 || HQ < 1 || HKV < 1 || D < 1 || DV < 1 ||
         page_size < 1 || window < 0 || chunk < 0 || !valid_dtype(q_dtype) || !valid_dtype(kv_dtype) || !valid_dtype(out_dtype) ||
-        (gate && !valid_dtype(gate_dtype)) || (r1 == nullptr) != (r2 == nullptr) || cap < 0.0f)
+        (gate && !valid_dtype(gate_dtype)) || (r2 && !r1) || cap < 0.0f)
         return fail(PH_ERR_ARG, "attention_talking: bad arguments (T %d, HQ %d, HKV %d, D %d, DV %d)", T, HQ, HKV, D, DV);
     if (HQ % HKV) return fail(PH_ERR_ARG, "attention_talking: %d query heads are not a multiple of %d kv heads", HQ, HKV);
     if (HQ > MAX_HEADS) return fail(PH_ERR_UNSUPPORTED, "attention_talking: %d heads exceed the supported %d", HQ, MAX_HEADS);

@@ -163,7 +163,10 @@ __global__ void __launch_bounds__(MAX_HEADS * 32) attention_talking_mma_kernel(c
         if (p.r1) {
             // the bias depends on the distance alone: row - key takes 47 values in a block, a lane makes two of them
             __syncwarp();
-            for (int idx = lane; idx < BIAS_N - 1; idx += 32) bias[idx] = b1 * log1pf(b2 * (float)max(z_first - key0 + idx - (BK - 1), 0));
+            for (int idx = lane; idx < BIAS_N - 1; idx += 32) {
+                const float distance = (float)max(z_first - key0 + idx - (BK - 1), 0);
+                bias[idx] = b1 * (p.r2 ? log1pf(b2 * distance) : distance);
+            }
             __syncwarp();
         }
         float s[BK / 8][4];
@@ -343,7 +346,7 @@ PH_EXPORT int ph_attention_talking_mma(const void* q, const void* k_base, const 
                                        const float* talk, const float* sink, const void* gate, long long gate_stride, int splits, int T,
                                        float* part_o, float* part_ml, cudaStream_t stream) {
     if (!q || !k_base || !v_base || !block_table || !seg_start || !seg_ctx_len || !tile_seg || !tile_first || !out || n_tiles < 0 ||
-        page_size < 1 || window < 0 || chunk < 0 || (r1 == nullptr) != (r2 == nullptr) || cap < 0.0f || splits < 1 || splits > 64 ||
+        page_size < 1 || window < 0 || chunk < 0 || (r2 && !r1) || cap < 0.0f || splits < 1 || splits > 64 ||
         (splits > 1 && (!part_o || !part_ml || T < 1 || ((uintptr_t)part_o % 8))))
         return fail(PH_ERR_ARG, "attention_talking_mma: bad arguments");
     if (!ph_attention_talking_mma_supports(HQ, HKV, D, DV))

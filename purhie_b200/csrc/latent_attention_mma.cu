@@ -264,7 +264,8 @@ cudaError_t launch_latent(dim3 grid, cudaStream_t stream, const __nv_bfloat16* q
 //                         out = q_lat [T, H, ldo] bfloat16; the CTAs of the first column tile also rotate the R numbers
 //                         behind the first K into the R numbers behind the first N of the output row;
 //   expand (KN = false):  a = o_lat [T, H, K] float32, B_h = wuv[h * N + n, k] (k contiguous), out [T, H * N] bfloat16,
-//                         times sigmoid(gate[t, h]).
+//                         times sigmoid(gate[t, h]), or with a logit per value sigmoid(gate[t, h, n]).
+// Tokens of a are tok_stride elements apart.
 // One CTA of four warps per (64 columns, head, 64 tokens); K in steps of 32 through shared memory.
 constexpr int HG_BM = 64, HG_BN = 64, HG_BK = 32, HG_THREADS = 128;
 constexpr int HG_PITCH_K = HG_BK * 2 + 16;      // bytes of a row of 32 k (A tiles, and B tiles stored n by k)
@@ -285,8 +286,8 @@ template <typename T> __device__ __forceinline__ void stage8(uint8_t* dst, const
 
 template <bool KN, typename TA>
 __global__ void __launch_bounds__(HG_THREADS) head_product_kernel(
-    const TA* __restrict__ a, long long lda, const __nv_bfloat16* __restrict__ b, __nv_bfloat16* __restrict__ out, long long ldo, int T,
-    int H, int K, int N, const __nv_bfloat16* __restrict__ gate, long long gate_stride, int R, const float* __restrict__ cos_sin,
+    const TA* __restrict__ a, long long tok_stride, long long lda, const __nv_bfloat16* __restrict__ b, __nv_bfloat16* __restrict__ out, long long ldo, int T,
+    int H, int K, int N, const __nv_bfloat16* __restrict__ gate, long long gate_stride, int gate_cols, int R, const float* __restrict__ cos_sin,
     int n_rot, int max_pos, const int32_t* __restrict__ positions) {
     __shared__ __align__(16) uint8_t a_s[HG_BM * HG_PITCH_K];
     __shared__ __align__(16) uint8_t b_s[KN ? HG_BK * HG_PITCH_N : HG_BN * HG_PITCH_K];
@@ -295,7 +296,7 @@ __global__ void __launch_bounds__(HG_THREADS) head_product_kernel(
     const int n0 = blockIdx.x * HG_BN, h = blockIdx.y, t0 = blockIdx.z * HG_BM;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t a_tile = smem_u32(a_s), b_tile = smem_u32(b_s);
-    const bool vec_a = lda % 8 == 0 && reinterpret_cast<uintptr_t>(a) % 32 == 0;
+    const bool vec_a = lda % 8 == 0 && tok_stride % 8 == 0 && reinterpret_cast<uintptr_t>(a) % 16 == 0;
     const bool vec_b = (KN ? N : K) % 8 == 0 && reinterpret_cast<uintptr_t>(b) % 16 == 0;
     float acc[HG_BN / 8][4];
 #pragma unroll
@@ -307,7 +308,7 @@ __global__ void __launch_bounds__(HG_THREADS) head_product_kernel(
         // A: 64 tokens x 32 k, eight k at a time
         for (int i = threadIdx.x; i < HG_BM * (HG_BK / 8); i += HG_THREADS) {
             const int r = i / (HG_BK / 8), k = (i % (HG_BK / 8)) * 8;
-            const TA* src = a + ((size_t)(t0 + r) * H + h) * lda + k0 + k;
+            const TA* src = a + (size_t)(t0 + r) * tok_stride + (size_t)h * lda + k0 + k;
             stage8<TA>(a_s + r * HG_PITCH_K + k * 2, src, t0 + r < T ? K - k0 - k : 0, vec_a);
         }
         if (KN) {       // B: 32 k x 64 n, n contiguous in memory
@@ -344,7 +345,7 @@ __global__ void __launch_bounds__(HG_THREADS) head_product_kernel(
     }
     const int r0 = t0 + warp * 16 + (lane >> 2), r1 = r0 + 8;
     float g0 = 1.0f, g1 = 1.0f;
-    if (gate) {
+    if (gate && gate_cols == 1) {
         if (r0 < T) g0 = 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)r0 * gate_stride + h])));
         if (r1 < T) g1 = 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)r1 * gate_stride + h])));
     }
@@ -355,8 +356,14 @@ __global__ void __launch_bounds__(HG_THREADS) head_product_kernel(
 #pragma unroll
         for (int half_row = 0; half_row < 2; ++half_row) {
             const int r = half_row ? r1 : r0;
-            const float g = half_row ? g1 : g0, u = acc[nt][half_row * 2] * g, v = acc[nt][half_row * 2 + 1] * g;
+            const float g = half_row ? g1 : g0;
+            float u = acc[nt][half_row * 2] * g, v = acc[nt][half_row * 2 + 1] * g;
             if (r >= T || n >= N) continue;
+            if (gate && gate_cols > 1) {
+                const __nv_bfloat16* gr = gate + (size_t)r * gate_stride + (size_t)h * gate_cols + n;
+                u *= 1.0f / (1.0f + expf(-__bfloat162float(gr[0])));
+                if (n + 1 < N) v *= 1.0f / (1.0f + expf(-__bfloat162float(gr[1])));
+            }
             __nv_bfloat16* dst = out + ((size_t)r * H + h) * ldo + n;
             if (pairs) *(uint32_t*)dst = pack_bf16(u, v);
             else {
@@ -371,7 +378,7 @@ __global__ void __launch_bounds__(HG_THREADS) head_product_kernel(
     for (int i = threadIdx.x; i < HG_BM * R; i += HG_THREADS) {
         const int t = t0 + i / R, d = i % R;
         if (t >= T) continue;
-        const TA* r = a + ((size_t)t * H + h) * lda + K;
+        const TA* r = a + (size_t)t * tok_stride + (size_t)h * lda + K;
         float v = to_float<TA>(r[d]);
         if (d < n_rot) {
             int pos = positions[t];
@@ -388,33 +395,33 @@ __global__ void __launch_bounds__(HG_THREADS) head_product_kernel(
 
 PH_DEFINE_LAST_ERROR(ph_latent)
 
-// q [T, H, D + R] bfloat16, wuk [H * D, C] bfloat16 -> q_lat [T, H, C + R] bfloat16 = [Wuk_h^T q_plain | rotate(q_rot)]
+// q [T, H, D + R] bfloat16 (tokens q_stride elements apart), wuk [H * D, C] bfloat16 -> q_lat [T, H, C + R] bfloat16 = [Wuk_h^T q_plain | rotate(q_rot)]
 // (latent_absorb of latent_attention.cu on the tensor cores).
-PH_EXPORT int ph_latent_absorb_mma(const void* q, const void* wuk, const float* cos_sin, int n_rot, int max_pos, const int32_t* positions,
+PH_EXPORT int ph_latent_absorb_mma(const void* q, long long q_stride, const void* wuk, const float* cos_sin, int n_rot, int max_pos, const int32_t* positions,
                                    void* q_lat, int T, int H, int D, int R, int C, cudaStream_t stream) {
     if (!q || !wuk || !q_lat || T < 0 || H < 1 || D < 1 || R < 0 || C < 1 || n_rot < 0 || n_rot > R || n_rot % 2 ||
-        (n_rot && (!cos_sin || !positions)))
+        q_stride < (long long)H * (D + R) || (n_rot && (!cos_sin || !positions)))
         return fail(PH_ERR_ARG, "latent_absorb_mma: bad arguments (T %d, H %d, D %d + %d, C %d)", T, H, D, R, C);
     if (T == 0) return PH_OK;
     const dim3 grid((unsigned)((C + HG_BN - 1) / HG_BN), (unsigned)H, (unsigned)((T + HG_BM - 1) / HG_BM));
     cudaError_t e = launch_overlapped(head_product_kernel<true, __nv_bfloat16>, grid, dim3(HG_THREADS), 0, stream, (const __nv_bfloat16*)q,
-                                      (long long)(D + R), (const __nv_bfloat16*)wuk, (__nv_bfloat16*)q_lat, (long long)(C + R), T, H, D, C,
-                                      (const __nv_bfloat16*)nullptr, 0LL, R, cos_sin, n_rot, max_pos, positions);
+                                      q_stride, (long long)(D + R), (const __nv_bfloat16*)wuk, (__nv_bfloat16*)q_lat, (long long)(C + R), T, H, D, C,
+                                      (const __nv_bfloat16*)nullptr, 0LL, 1, R, cos_sin, n_rot, max_pos, positions);
     if (e != cudaSuccess) return fail(PH_ERR_LAUNCH, "latent_absorb_mma: %s", cudaGetErrorString(e));
     return check_launch("latent_absorb_mma");
 }
 
-// o_lat [T, H, C] float32, wuv [H * DV, C] bfloat16, gate [T, gate_stride] bfloat16 (head h's logit at column h; null: none)
-// -> out [T, H * DV] bfloat16 = (Wuv_h o_lat[t, h]) * sigmoid(gate[t, h]) (latent_expand on the tensor cores).
-PH_EXPORT int ph_latent_expand_mma(const void* o_lat, const void* wuv, const void* gate, long long gate_stride, void* out, int T, int H,
-                                   int C, int DV, cudaStream_t stream) {
-    if (!o_lat || !wuv || !out || T < 0 || H < 1 || C < 1 || DV < 1)
+// o_lat [T, H, C] float32, wuv [H * DV, C] bfloat16, gate [T, gate_stride] bfloat16 (null: none) with gate_cols logits per
+// head, 1 or DV -> out [T, H * DV] bfloat16 = (Wuv_h o_lat[t, h]) * sigmoid(gate) (latent_expand on the tensor cores).
+PH_EXPORT int ph_latent_expand_mma(const void* o_lat, const void* wuv, const void* gate, long long gate_stride, int gate_cols, void* out,
+                                   int T, int H, int C, int DV, cudaStream_t stream) {
+    if (!o_lat || !wuv || !out || T < 0 || H < 1 || C < 1 || DV < 1 || (gate && gate_cols != 1 && gate_cols != DV))
         return fail(PH_ERR_ARG, "latent_expand_mma: bad arguments (T %d, H %d, C %d, DV %d)", T, H, C, DV);
     if (T == 0) return PH_OK;
     const dim3 grid((unsigned)((DV + HG_BN - 1) / HG_BN), (unsigned)H, (unsigned)((T + HG_BM - 1) / HG_BM));
-    cudaError_t e = launch_overlapped(head_product_kernel<false, float>, grid, dim3(HG_THREADS), 0, stream, (const float*)o_lat, (long long)C,
+    cudaError_t e = launch_overlapped(head_product_kernel<false, float>, grid, dim3(HG_THREADS), 0, stream, (const float*)o_lat, (long long)H * C, (long long)C,
                                       (const __nv_bfloat16*)wuv, (__nv_bfloat16*)out, (long long)DV, T, H, C, DV,
-                                      (const __nv_bfloat16*)gate, gate_stride, 0, (const float*)nullptr, 0, 0, (const int32_t*)nullptr);
+                                      (const __nv_bfloat16*)gate, gate_stride, gate_cols, 0, (const float*)nullptr, 0, 0, (const int32_t*)nullptr);
     if (e != cudaSuccess) return fail(PH_ERR_LAUNCH, "latent_expand_mma: %s", cudaGetErrorString(e));
     return check_launch("latent_expand_mma");
 }
@@ -447,9 +454,11 @@ PH_EXPORT int ph_latent_attention(const void* q, const void* k_base, long long p
     e = launch_latent<CP, RP>(grid, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_base, page_stride, page_size, block_table,   \
                               table_stride, seg_start, seg_ctx_len, tile_seg, tile_first, (float*)out, part_o, part_ml, H, C, R, window, \
                               scale_log2, splits)
-    if (C <= 128) { if (R <= 16) LAUNCH(128, 16); else LAUNCH(128, 64); }
-    else if (C <= 256) { if (R <= 16) LAUNCH(256, 16); else LAUNCH(256, 64); }
-    else { if (R <= 16) LAUNCH(512, 16); else LAUNCH(512, 64); }
+#define LAUNCH_R(CP) do { if (R == 0) LAUNCH(CP, 0); else if (R <= 16) LAUNCH(CP, 16); else LAUNCH(CP, 64); } while (0)
+    if (C <= 128) LAUNCH_R(128);
+    else if (C <= 256) LAUNCH_R(256);
+    else LAUNCH_R(512);
+#undef LAUNCH_R
 #undef LAUNCH
     if (e != cudaSuccess) return fail(PH_ERR_LAUNCH, "latent_attention: %s", cudaGetErrorString(e));
     if (splits > 1) {

@@ -9,6 +9,9 @@
 // v <- (1 - lambda) v + lambda v_first (mode 2), that first layer storing its own v as v_first (mode 1); the blended
 // v is what goes to the cache.  The table row of a position holds n_rot / 2 cosines, then
 // n_rot / 2 sines, one per pair.
+// The product's rows may go on behind the v heads (row_width): rows of a gate's logits, HQ heads of DV, which a later kernel
+// reads where they are, or, when they came as partial sums or without their row's factor, which heads of their own add up,
+// scale and store (gate_out).
 // Sums and angles are float32; the cos/sin table is made on the host in double precision.
 // Reference: src/attention.hip:273-313 (attn_prep: bias, norm, rotation, cache write), :219-240
 // (the norm and the rotation), src/qwen_ops.cpp:15-24 (rotate-half pairing).
@@ -55,19 +58,20 @@ __global__ void qk_norm_rope_kernel(const TI* __restrict__ qkv, int splits, long
                                     const int32_t* __restrict__ slot_mapping, TQ* __restrict__ q_out,
                                     TKV* __restrict__ k_base, TKV* __restrict__ v_base, long long page_stride,
                                     int page_size, int HQ, int HKV, int D, int interleaved, RowFactor rf, int DV,
-                                    float* __restrict__ v_first, const float* __restrict__ v_lambda, int v_mode) {
+                                    float* __restrict__ v_first, const float* __restrict__ v_lambda, int v_mode, long long row_width,
+                                    TQ* __restrict__ gate_out) {
     __shared__ float buf[WARPS][MAX_D];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int head = blockIdx.y * WARPS + warp;
     const int t = blockIdx.x;
-    const int n_heads = HQ + 2 * HKV;
+    const int n_heads = HQ + 2 * HKV + (gate_out ? HQ : 0);
     if (head >= n_heads) return;
-    const int width = (HQ + HKV) * D + HKV * DV;
     const bool is_q = head < HQ, is_k = !is_q && head < HQ + HKV;
     const size_t head_at = (is_q || is_k) ? (size_t)head * D : (size_t)(HQ + HKV) * D + (size_t)(head - HQ - HKV) * DV;
     const int hd = (is_q || is_k) ? D : DV;                    // this head's width
-    const TI* src = qkv + (size_t)t * width + head_at;
-    const float* b = bias ? bias + head_at : nullptr;
+    const TI* src = qkv + (size_t)t * row_width + head_at;
+    const bool is_gate = head >= HQ + 2 * HKV;
+    const float* b = bias && !is_gate ? bias + head_at : nullptr;
     float* row = buf[warp];
     const float rs = row_factor(rf, t);
 
@@ -81,6 +85,12 @@ __global__ void qk_norm_rope_kernel(const TI* __restrict__ qkv, int splits, long
         ss += v * v;
     }
     const float* w = is_q ? q_w : (is_k ? k_w : nullptr);
+    if (is_gate) {
+        __syncwarp();
+        TQ* dst = gate_out + ((size_t)t * HQ + (head - HQ - 2 * HKV)) * DV;
+        for (int d = lane; d < DV; d += 32) dst[d] = from_float<TQ>(row[d]);
+        return;
+    }
     if (!is_q && !is_k) {
         // v head: copy, or blend with the step's first values
         if (!slot_mapping) return;
@@ -176,13 +186,14 @@ __global__ void qk_norm_rope_d128_kernel(const TI* __restrict__ qkv, int splits,
                                          const int32_t* __restrict__ slot_mapping, TQ* __restrict__ q_out,
                                          TKV* __restrict__ k_base, TKV* __restrict__ v_base, long long page_stride,
                                          int page_size, int HQ, int HKV, RowFactor rf, int interleaved,
-                                         float* __restrict__ v_first, const float* __restrict__ v_lambda, int v_mode) {
+                                         float* __restrict__ v_first, const float* __restrict__ v_lambda, int v_mode, long long row_width,
+                                         TQ* __restrict__ gate_out) {
     constexpr int D = 128;
     pdl_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int head0 = (blockIdx.y * WARPS + warp) * HPW;      // this warp's HPW consecutive heads of token t
     const int t = blockIdx.x;
-    const int n_heads = HQ + 2 * HKV;
+    const int n_heads = HQ + 2 * HKV + (gate_out ? HQ : 0);
     if (head0 >= n_heads) return;
     const int d0 = lane * 4;
     // what no kernel of this step writes (positions, slots, the table, the norms' weights) is fetched while the
@@ -214,7 +225,7 @@ __global__ void qk_norm_rope_d128_kernel(const TI* __restrict__ qkv, int splits,
     for (int i = 0; i < HPW; ++i) {
         v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (head0 + i >= n_heads) continue;
-        const TI* src = qkv + (size_t)t * n_heads * D + (size_t)(head0 + i) * D + d0;
+        const TI* src = qkv + (size_t)t * row_width + (size_t)(head0 + i) * D + d0;
         for (int s0 = 0; s0 < splits; s0 += 8) {             // eight partial sums in flight, added in order
             float4 u[8];
 #pragma unroll
@@ -230,6 +241,10 @@ __global__ void qk_norm_rope_d128_kernel(const TI* __restrict__ qkv, int splits,
         const int head = head0 + i;
         if (head >= n_heads) break;
         float4 x = make_float4(v[i].x * rs, v[i].y * rs, v[i].z * rs, v[i].w * rs);
+        if (head >= HQ + 2 * HKV) {
+            st4(gate_out + ((size_t)t * HQ + (head - HQ - 2 * HKV)) * D + d0, x);
+            continue;
+        }
         if (bias) {
             const float4 b = ld4(bias + (size_t)head * D + d0);
             x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w;
@@ -324,7 +339,8 @@ __global__ void qk_norm_rope_d128_wide_kernel(const TI* __restrict__ qkv, int sp
                                               const int32_t* __restrict__ slot_mapping, TQ* __restrict__ q_out,
                                               TKV* __restrict__ k_base, TKV* __restrict__ v_base, long long page_stride,
                                               int page_size, int HQ, int HKV, RowFactor rf, int interleaved,
-                                              float* __restrict__ v_first, const float* __restrict__ v_lambda, int v_mode) {
+                                              float* __restrict__ v_first, const float* __restrict__ v_lambda, int v_mode, long long row_width,
+                                              TQ* __restrict__ gate_out) {
     constexpr int D = 128;
     pdl_launch_dependents();
     pdl_wait();
@@ -333,7 +349,7 @@ __global__ void qk_norm_rope_d128_wide_kernel(const TI* __restrict__ qkv, int sp
     const int half = lane >> 4, l16 = lane & 15;
     const int head0 = (blockIdx.y * WARPS + warp) * 2 * ITERS + half;      // this half-warp's heads: head0, head0 + 2, ...
     const int t = blockIdx.x;
-    const int n_heads = HQ + 2 * HKV;
+    const int n_heads = HQ + 2 * HKV + (gate_out ? HQ : 0);
     const int d0 = l16 * 8;
     const float rs = row_factor(rf, t);
     F8 v[ITERS];
@@ -342,7 +358,7 @@ __global__ void qk_norm_rope_d128_wide_kernel(const TI* __restrict__ qkv, int sp
         v[i] = {make_float4(0.0f, 0.0f, 0.0f, 0.0f), make_float4(0.0f, 0.0f, 0.0f, 0.0f)};
         const int head = head0 + 2 * i;
         if (head >= n_heads) continue;
-        const TI* src = qkv + (size_t)t * n_heads * D + (size_t)head * D + d0;
+        const TI* src = qkv + (size_t)t * row_width + (size_t)head * D + d0;
         for (int s0 = 0; s0 < splits; ++s0) {
             const F8 u = ld8(src + (size_t)s0 * split_stride);
             add4(v[i].a, u.a);
@@ -372,7 +388,8 @@ __global__ void qk_norm_rope_d128_wide_kernel(const TI* __restrict__ qkv, int sp
         F8 x = v[i];
         x.a = make_float4(x.a.x * rs, x.a.y * rs, x.a.z * rs, x.a.w * rs);
         x.b = make_float4(x.b.x * rs, x.b.y * rs, x.b.z * rs, x.b.w * rs);
-        if (bias && live) {
+        const bool is_gate = head >= HQ + 2 * HKV;
+        if (bias && live && !is_gate) {
             const F8 b = ld8(bias + (size_t)head * D + d0);
             add4(x.a, b.a);
             add4(x.b, b.b);
@@ -396,6 +413,10 @@ __global__ void qk_norm_rope_d128_wide_kernel(const TI* __restrict__ qkv, int sp
         }
         const float4 oa = shfl4(y.a, 8), ob = shfl4(y.b, 8);
         if (!live) continue;
+        if (is_gate) {
+            st8(gate_out + ((size_t)t * HQ + (head - HQ - 2 * HKV)) * D + d0, x);
+            continue;
+        }
         if (!is_q && !is_k) {
             if (slot >= 0) {
                 const int h = head - HQ - HKV;
@@ -434,14 +455,16 @@ __global__ void qk_norm_rope_d128_wide_kernel(const TI* __restrict__ qkv, int sp
 
 }  // namespace
 
-PH_EXPORT int ph_qk_norm_rope_kv_write(const void* qkv, int qkv_dtype, int splits, long long split_stride,
-                                       const float* bias, const float* q_norm_w, const float* k_norm_w, float eps,
-                                       const float* cos_sin, int n_rot, int max_pos, const int32_t* positions,
-                                       const int32_t* slot_mapping, void* q_out, int q_dtype, void* k_base,
-                                       void* v_base, int kv_dtype, long long page_stride, int page_size, int T,
-                                       int HQ, int HKV, int D, int interleaved, const float* row_sumsq, int row_chunks,
-                                       int row_width, float row_eps, int DV, float* v_first, const float* v_lambda, int v_mode,
-                                       cudaStream_t stream) {
+// product_width: elements from one token's row of the product to the next's (0: [q | k | v] and nothing behind).  gate_out
+// [T, HQ * DV] in q's dtype, or null: the HQ * DV numbers behind v, added up, times the row's factor.
+PH_EXPORT int ph_qk_norm_rope_gate_kv_write(const void* qkv, int qkv_dtype, int splits, long long split_stride,
+                                            const float* bias, const float* q_norm_w, const float* k_norm_w, float eps,
+                                            const float* cos_sin, int n_rot, int max_pos, const int32_t* positions,
+                                            const int32_t* slot_mapping, void* q_out, int q_dtype, void* k_base,
+                                            void* v_base, int kv_dtype, long long page_stride, int page_size, int T,
+                                            int HQ, int HKV, int D, int interleaved, const float* row_sumsq, int row_chunks,
+                                            int row_width, float row_eps, int DV, float* v_first, const float* v_lambda, int v_mode,
+                                            long long product_width, void* gate_out, cudaStream_t stream) {
     if (!qkv || !positions || !q_out || T < 0 || HQ < 1 || HKV < 0 || D < 2 || splits < 1 || !valid_dtype(qkv_dtype) ||
         !valid_dtype(q_dtype) || !valid_dtype(kv_dtype))
         return fail(PH_ERR_ARG, "qk_norm_rope: bad arguments (T %d, HQ %d, HKV %d, D %d)", T, HQ, HKV, D);
@@ -455,13 +478,18 @@ PH_EXPORT int ph_qk_norm_rope_kv_write(const void* qkv, int qkv_dtype, int split
         return fail(PH_ERR_ARG, "qk_norm_rope: a cache write needs the pool and its page size");
     if (row_sumsq && (row_chunks < 1 || row_width < 1)) return fail(PH_ERR_ARG, "qk_norm_rope: a row factor needs its chunks and the row width");
     if (T == 0) return PH_OK;
+    const long long width = (long long)(HQ + HKV) * D + (long long)HKV * DV;
+    if (product_width <= 0) product_width = width;
+    if (product_width < width + (gate_out ? (long long)HQ * DV : 0))
+        return fail(PH_ERR_ARG, "qk_norm_rope: rows of %lld elements are too short", product_width);
     const RowFactor rf = {row_sumsq, row_chunks, row_width, row_eps};
-    dim3 grid(T, (HQ + 2 * HKV + WARPS - 1) / WARPS);
-    const bool fast = D == 128 && DV == D && (!cos_sin || n_rot == 128) && split_stride % 4 == 0 && (((uintptr_t)v_first) & 15) == 0 &&
+    const int n_heads = HQ + 2 * HKV + (gate_out ? HQ : 0);
+    dim3 grid(T, (n_heads + WARPS - 1) / WARPS);
+    const bool fast = D == 128 && DV == D && (!cos_sin || n_rot == 128) && split_stride % 4 == 0 && product_width % 8 == 0 &&
+                      (((uintptr_t)v_first | (uintptr_t)gate_out) & 15) == 0 &&
                       (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_base | (uintptr_t)v_base | (uintptr_t)bias |
                         (uintptr_t)q_norm_w | (uintptr_t)k_norm_w | (uintptr_t)cos_sin) & 15) == 0 && page_stride % 8 == 0;
     if (fast) {
-        const int n_heads = HQ + 2 * HKV;
         // enough tokens to fill the device with warps that walk three pairs of heads each: the wide kernel
         const bool many = (long long)T * n_heads >= 16384 && page_stride % 8 == 0 && split_stride % 8 == 0;
         const dim3 fgrid(T, many ? (n_heads + WARPS * 6 - 1) / (WARPS * 6) : (n_heads + WARPS - 1) / WARPS);
@@ -471,12 +499,12 @@ PH_EXPORT int ph_qk_norm_rope_kv_write(const void* qkv, int qkv_dtype, int split
             launch_overlapped(qk_norm_rope_d128_wide_kernel<TI, TQ, TKV, 3>, fgrid, dim3(WARPS * 32), 0, stream, (const TI*)qkv, \
                               splits, split_stride, bias, q_norm_w, k_norm_w, eps, cos_sin, max_pos, positions,     \
                               slot_mapping, (TQ*)q_out, (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, rf, \
-                              interleaved, v_first, v_lambda, v_mode);                                               \
+                              interleaved, v_first, v_lambda, v_mode, product_width, (TQ*)gate_out);                                               \
         else                                                                                                        \
             launch_overlapped(qk_norm_rope_d128_kernel<TI, TQ, TKV, 1>, fgrid, dim3(WARPS * 32), 0, stream, (const TI*)qkv, \
                               splits, split_stride, bias, q_norm_w, k_norm_w, eps, cos_sin, max_pos, positions,     \
                               slot_mapping, (TQ*)q_out, (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, rf, \
-                              interleaved, v_first, v_lambda, v_mode);                                               \
+                              interleaved, v_first, v_lambda, v_mode, product_width, (TQ*)gate_out);                                               \
     } while (0)
         PH_DISPATCH(qkv_dtype, TI, PH_DISPATCH(q_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, LAUNCH_FAST(TI, TQ, TKV))));
 #undef LAUNCH_FAST
@@ -486,8 +514,22 @@ PH_EXPORT int ph_qk_norm_rope_kv_write(const void* qkv, int qkv_dtype, int split
     qk_norm_rope_kernel<TI, TQ, TKV><<<grid, WARPS * 32, 0, stream>>>(                                            \
         (const TI*)qkv, splits, split_stride, bias, q_norm_w, k_norm_w, eps, cos_sin, n_rot, max_pos, positions,  \
         slot_mapping, (TQ*)q_out, (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, D, interleaved, rf, DV,     \
-        v_first, v_lambda, v_mode)
+        v_first, v_lambda, v_mode, product_width, (TQ*)gate_out)
     PH_DISPATCH(qkv_dtype, TI, PH_DISPATCH(q_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, LAUNCH(TI, TQ, TKV))));
 #undef LAUNCH
     return check_launch("qk_norm_rope");
+}
+
+PH_EXPORT int ph_qk_norm_rope_kv_write(const void* qkv, int qkv_dtype, int splits, long long split_stride,
+                                       const float* bias, const float* q_norm_w, const float* k_norm_w, float eps,
+                                       const float* cos_sin, int n_rot, int max_pos, const int32_t* positions,
+                                       const int32_t* slot_mapping, void* q_out, int q_dtype, void* k_base,
+                                       void* v_base, int kv_dtype, long long page_stride, int page_size, int T,
+                                       int HQ, int HKV, int D, int interleaved, const float* row_sumsq, int row_chunks,
+                                       int row_width, float row_eps, int DV, float* v_first, const float* v_lambda, int v_mode,
+                                       cudaStream_t stream) {
+    return ph_qk_norm_rope_gate_kv_write(qkv, qkv_dtype, splits, split_stride, bias, q_norm_w, k_norm_w, eps, cos_sin, n_rot, max_pos,
+                                         positions, slot_mapping, q_out, q_dtype, k_base, v_base, kv_dtype, page_stride, page_size, T, HQ,
+                                         HKV, D, interleaved, row_sumsq, row_chunks, row_width, row_eps, DV, v_first, v_lambda, v_mode, 0,
+                                         nullptr, stream);
 }

@@ -241,6 +241,41 @@ void context_from_layout(const StepLayout& lay, const CacheManager& cache, int p
     for (const auto& a : lay.extra) ctx.arrays[a.first] = StepArray{dev + a.second.first, a.second.second};
 }
 
+namespace {
+// What a residual of several lanes adds up to once the pending addend has entered (on the host, for dumps).
+void sum_of_lanes(const ResidualStream& stream, int T, int E, std::vector<float>& x) {
+    const int S = stream.n_lanes;
+    const bool first = !stream.lanes.defined();
+    const Tensor& held = first ? stream.x : stream.lanes;
+    std::vector<float> lanes((size_t)held.numel());
+    QE_CUDA(cudaMemcpy(lanes.data(), held.data, lanes.size() * 4, cudaMemcpyDeviceToHost));
+    // the lanes' sum behind the update: each old lane counts with its row of the mix, the addend with the sum of its factors
+    std::vector<double> weight(S, 1.0);
+    double addend = 0.0;
+    std::vector<float> add;
+    if (stream.has_pending) {
+        std::vector<float> mix((size_t)S * S), out(S);
+        QE_CUDA(cudaMemcpy(mix.data(), stream.lane_update.mix, mix.size() * 4, cudaMemcpyDeviceToHost));
+        QE_CUDA(cudaMemcpy(out.data(), stream.lane_update.out, out.size() * 4, cudaMemcpyDeviceToHost));
+        for (int s = 0; s < S; s++) {
+            weight[s] = 0.0;
+            for (int t = 0; t < S; t++) weight[s] += mix[(size_t)s * S + t];
+            addend += out[s];
+        }
+        if (stream.pending.tensor.dtype != DType::F32) throw Error(kInvalidState, "a dump reads float32 addends only");
+        add.resize((size_t)stream.pending.splits * T * E);
+        QE_CUDA(cudaMemcpy(add.data(), stream.pending.tensor.data, add.size() * 4, cudaMemcpyDeviceToHost));
+    }
+    for (int t = 0; t < T; t++)
+        for (int i = 0; i < E; i++) {
+            double v = 0.0;
+            for (int s = 0; s < S; s++) v += weight[s] * lanes[first ? (size_t)t * E + i : ((size_t)t * S + s) * E + i];
+            for (int p = 0; stream.has_pending && p < stream.pending.splits; p++) v += addend * add[((size_t)p * T + t) * E + i];
+            x[(size_t)t * E + i] = (float)v;
+        }
+}
+}  // namespace
+
 Tensor Engine::forward(StepContext& ctx, const int32_t* want_rows, int n_want) {
     if (LaunchProfile::get().on()) LaunchProfile::get().set_stream(stream_);
     if (!layer_dump_) return model_->forward(ctx, views_, want_rows, n_want);
@@ -248,6 +283,11 @@ Tensor Engine::forward(StepContext& ctx, const int32_t* want_rows, int n_want) {
         const int T = c.T, E = (int)stream.x.shape[1];
         std::vector<float> x((size_t)T * E);
         QE_CUDA(cudaStreamSynchronize(stream_));
+        if (stream.n_lanes) {                                     // the sum of the lanes, the pending addend folded in
+            sum_of_lanes(stream, T, E, x);
+            layer_dump_(entry, x.data(), T, E);
+            return;
+        }
         QE_CUDA(cudaMemcpy(x.data(), stream.x.data, x.size() * 4, cudaMemcpyDeviceToHost));
         if (stream.has_pending) {
             const Tensor& p = stream.pending.tensor;

@@ -178,7 +178,13 @@ const CoreKernels& core_kernels() {
     bind(h, "core", "ph_latent_prepare", g_core.latent_prepare);
     bind(h, "core", "ph_latent_absorb", g_core.latent_absorb);
     bind(h, "core", "ph_latent_expand", g_core.latent_expand);
-    bind(h, "core", "ph_attention_generic_sink", g_core.attention_generic_sink);
+    bind(h, "core", "ph_attention_generic_biased", g_core.attention_generic_biased);
+    bind(h, "core", "ph_qk_norm_rope_gate_kv_write", g_core.qk_norm_rope_gate_kv_write);
+    bind(h, "core", "ph_lanes_rmsnorm", g_core.lanes_rmsnorm);
+    bind(h, "core", "ph_ssd_scan", g_core.ssd_scan);
+    bind(h, "core", "ph_ssd_chunk", g_core.ssd_chunk);
+    bind(h, "core", "ph_ssd_chunk_supports", g_core.ssd_chunk_supports);
+    bind(h, "core", "ph_gate_rms", g_core.gate_rms);
     bind(h, "core", "ph_attention_talking", g_core.attention_talking);
     bind(h, "core", "ph_attention_talking_mma", g_core.attention_talking_mma);
     bind(h, "core", "ph_attention_talking_mma_supports", g_core.attention_talking_mma_supports);
@@ -202,8 +208,8 @@ const FlashKernels& flash_kernels() {
     bind(h, "flash", "ph_attention_decode", g_flash.decode);
     bind(h, "flash", "ph_attention_decode_bulk", g_flash.decode_bulk);
     bind(h, "flash", "ph_attention_prefill_tc5", g_flash.prefill_tc5);
-    bind(h, "flash", "ph_attention_decode_bulk_sink", g_flash.decode_bulk_sink);
-    bind(h, "flash", "ph_attention_prefill_tc5_sink", g_flash.prefill_tc5_sink);
+    bind(h, "flash", "ph_attention_decode_bulk_biased", g_flash.decode_bulk_biased);
+    bind(h, "flash", "ph_attention_prefill_tc5_biased", g_flash.prefill_tc5_biased);
     bind(h, "flash", "ph_flash_last_error", g_flash.last_error);
     g_flash_ok = true;
     return g_flash;

@@ -97,6 +97,11 @@ struct CoreKernels {
                                  const float*, int, int, const int32_t*, const int32_t*, void*, int, void*, void*, int,
                                  long long, int, int, int, int, int, int, const float*, int, int, float, int, float*,
                                  const float*, int, cudaStream_t);
+    // the same over rows that go on behind v, with the gate's logits there added up and stored
+    int (*qk_norm_rope_gate_kv_write)(const void*, int, int, long long, const float*, const float*, const float*, float,
+                                      const float*, int, int, const int32_t*, const int32_t*, void*, int, void*, void*, int,
+                                      long long, int, int, int, int, int, int, const float*, int, int, float, int, float*,
+                                      const float*, int, long long, void*, cudaStream_t);
     int (*add_weight_sumsq)(float*, const void*, int, int, long long, const float*, int, int, void*, int, float*, int, cudaStream_t);
     int (*attention_generic)(const void*, int, const void*, const void*, int, long long, int, const int32_t*, int,
                              const int32_t*, const int32_t*, void*, int, int, int, int, int, int, float, int, int, int, cudaStream_t);
@@ -151,15 +156,16 @@ struct CoreKernels {
     // attention through a latent: norms, rotation and the cache row; the key expansion folded into q; the value expansion
     int (*latent_prepare)(const void*, int, long long, int, int, int, const float*, const float*, float, const float*, int, int,
                           const int32_t*, const int32_t*, void*, int, void*, int, long long, int, int, cudaStream_t);
-    int (*latent_absorb)(const void*, int, const void*, int, const float*, int, int, const int32_t*, void*, int, int, int, int, int, int,
-                         cudaStream_t);
-    int (*latent_expand)(const void*, int, const void*, int, const void*, int, long long, void*, int, int, int, int, int, cudaStream_t);
+    int (*latent_absorb)(const void*, int, long long, const void*, int, const float*, int, int, const int32_t*, void*, int, int, int, int, int,
+                         int, cudaStream_t);
+    int (*latent_expand)(const void*, int, const void*, int, const void*, int, long long, int, void*, int, int, int, int, int, cudaStream_t);
     // attention with a sink in the softmax's denominator (the plain kernel); attention whose heads' scores are capped,
     // biased by the distance and mixed before the softmax, with the kernel that norms q and k over their whole width and
     // writes the cache rows in front of it
-    int (*attention_generic_sink)(const void*, int, const void*, const void*, int, long long, int, const int32_t*, int,
-                                  const int32_t*, const int32_t*, void*, int, int, int, int, int, int, float, int, int, int, const float*,
-                                  cudaStream_t);
+    // (the plain kernel: a sink, a distance bias and an output gate, each optional)
+    int (*attention_generic_biased)(const void*, int, const void*, const void*, int, long long, int, const int32_t*, int,
+                                    const int32_t*, const int32_t*, void*, int, int, int, int, int, int, float, int, int, int, const float*,
+                                    const float*, const void*, long long, cudaStream_t);
     int (*attention_talking)(const void*, int, const void*, const void*, int, long long, int, const int32_t*, int, const int32_t*,
                              const int32_t*, void*, int, int, int, int, int, int, int, int, float, float, const float*, const float*,
                              const float*, const float*, const void*, int, long long, cudaStream_t);
@@ -178,6 +184,16 @@ struct CoreKernels {
     // add_rmsnorm with a factor on the addend
     int (*add_scaled_rmsnorm)(float*, const void*, int, int, long long, const float*, float, const int32_t*, int, int, void*, int, int, float,
                               cudaStream_t);
+    // a residual of several lanes: the addend mixed in, the lanes read, the RMS norm of what was read
+    int (*lanes_rmsnorm)(const float*, long long, long long, float*, const void*, int, int, long long, const float*, const float*, const float*,
+                         const float*, float, const int32_t*, int, int, int, void*, int, cudaStream_t);
+    // the second Mamba form: the scan token by token, the scan in chunks on the tensor cores, the gated norm in parts
+    int (*ssd_scan)(const void*, const void*, int, long long, int, int, const float*, const float*, const float*, float*, long long,
+                    const int32_t*, const int32_t*, int, int, int, int, int, int, int, int, float*, cudaStream_t);
+    int (*ssd_chunk)(const void*, const void*, long long, int, int, const float*, const float*, const float*, float*, long long,
+                     const int32_t*, const int32_t*, int, int, int, int, int, int, int, int, float*, cudaStream_t);
+    int (*ssd_chunk_supports)(int, int, int);
+    int (*gate_rms)(const float*, const void*, int, long long, const float*, float, void*, int, int, int, int, cudaStream_t);
     // logits scaled and softly capped in place
     int (*scale_softcap)(float*, long long, float, float, cudaStream_t);
     const char* (*last_error)(void);
@@ -193,13 +209,13 @@ struct FlashKernels {
     int (*prefill_tc5)(const void*, int, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*,
                        const int32_t*, const int32_t*, const int32_t*, int, void*, int, int, int, int, int, float, int, float*,
                        float*, int*, cudaStream_t);
-    // the two kernels above with a sink ([HQ] float32) in the softmax's denominator
-    int (*decode_bulk_sink)(const void*, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*, int,
-                            const int32_t*, const int32_t*, float*, float*, void*, int, int, int, int, int, int, float, int, int*,
-                            const float*, cudaStream_t);
-    int (*prefill_tc5_sink)(const void*, int, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*,
-                            const int32_t*, const int32_t*, const int32_t*, int, void*, int, int, int, int, int, float, int, float*,
-                            float*, int*, const float*, cudaStream_t);
+    // the two kernels above with a sink in the softmax's denominator, a distance bias and an output gate, each optional
+    int (*decode_bulk_biased)(const void*, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*, int,
+                              const int32_t*, const int32_t*, float*, float*, void*, int, int, int, int, int, int, float, int, int*,
+                              const float*, const float*, const void*, long long, cudaStream_t);
+    int (*prefill_tc5_biased)(const void*, int, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*,
+                              const int32_t*, const int32_t*, const int32_t*, int, void*, int, int, int, int, int, float, int, float*,
+                              float*, int*, const float*, const float*, const void*, long long, cudaStream_t);
     const char* (*last_error)(void);
 };
 // attention over cached latent rows on the tensor cores (latent_attention_mma.cu)
@@ -208,8 +224,9 @@ struct LatentKernels {
     int (*attention)(const void*, const void*, long long, int, const int32_t*, int, const int32_t*, const int32_t*, const int32_t*,
                      const int32_t*, int, void*, float*, float*, int, int, int, int, float, int, cudaStream_t);
     // the products per head in front of and behind it
-    int (*latent_absorb)(const void*, const void*, const float*, int, int, const int32_t*, void*, int, int, int, int, int, cudaStream_t);
-    int (*latent_expand)(const void*, const void*, const void*, long long, void*, int, int, int, int, cudaStream_t);
+    int (*latent_absorb)(const void*, long long, const void*, const float*, int, int, const int32_t*, void*, int, int, int, int, int,
+                         cudaStream_t);
+    int (*latent_expand)(const void*, const void*, const void*, long long, int, void*, int, int, int, int, cudaStream_t);
     const char* (*last_error)(void);
 };
 struct GemmKernels {

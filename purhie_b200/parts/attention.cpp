@@ -13,7 +13,10 @@
 // and value mixing across layers ("value_mix": "first" | "blend"): the first such layer of a model leaves its v for
 // every token of the step, the later ones cache and attend over v <- (1 - lambda) v + lambda v_first, with lambda a
 // scalar tensor of their own ("value_mix_factor"); a sink (names.sink: one float32 number per query head that stands in
-// the softmax's denominator as exp(sink), without a key or a value).
+// the softmax's denominator as exp(sink), without a key or a value; "sink_value": the same with one constant for all
+// heads); norms of q and k without a weight ("qk_norm_weight": false); a distance bias ("distance_slopes": one number per
+// query head, taken off the scaled score times the distance); an output gate (names.gate_proj: the heads side by side
+// times sigmoid(Wg x), element by element, before Wo).
 //
 // K and V are written to pages before attention runs, and attention reads everything, the current step's keys
 // included, from pages: a whole prompt, a portion and a decoded token are one algorithm per kernel.
@@ -125,7 +128,8 @@ void add_tiles(StepPlan& plan, int rows, const std::string& name, bool single_ro
 // params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim (null: head_dim), qk_norm_eps (null: no q/k norm),
 // bias, position (a PartSpec as {kind, params}, or null), window (null: all positions), chunk (null: no block mask),
 // scale (null: 1/sqrt(head_dim)), value_mix (null | "first" | "blend"),
-// names{q_proj, k_proj, v_proj, o_proj, q_norm, k_norm, q_bias, k_bias, v_bias, value_mix_factor}.
+// qk_norm_weight (default true), distance_slopes (null, or a list of num_heads numbers), sink_value (null: none),
+// names{q_proj, k_proj, v_proj, o_proj, q_norm, k_norm, q_bias, k_bias, v_bias, value_mix_factor, sink, gate_proj}.
 class Attention : public Mixer {
 public:
     Attention(const Json& p, BuildContext& b) : Mixer(p, b) {
@@ -144,7 +148,20 @@ public:
         has_norm_ = eps && !eps->is_null();
         eps_ = has_norm_ ? eps->as_double() : 0.0;
         has_bias_ = p.get_bool("bias", false);
+        norm_weight_ = p.get_bool("qk_norm_weight", true);
         has_sink_ = names_.count("sink") != 0;
+        if (const Json* sv = p.find("sink_value"))
+            if (!sv->is_null()) {
+                if (has_sink_) throw ConfigError("attention: a sink is a stored number per head or one constant, not both");
+                has_sink_ = constant_sink_ = true;
+                sink_value_ = sv->as_double();
+            }
+        if (const Json* ds = p.find("distance_slopes"))
+            if (!ds->is_null()) {
+                if (!ds->is_array() || (int)ds->size() != heads_) throw ConfigError("attention: distance_slopes must list one number per query head");
+                for (const Json& v : ds->items()) slopes_host_.push_back((float)v.as_double());
+            }
+        has_gate_ = names_.count("gate_proj") != 0;
         window_ = (int)p.get_int("window", 0);
         chunk_ = (int)p.get_int("chunk", 0);
         if (chunk_ < 0) throw ConfigError("attention: a block mask holds at least one position");
@@ -166,6 +183,8 @@ public:
         kv_width_ = (int64_t)kv_heads_ * head_dim_;
         v_width_ = (int64_t)kv_heads_ * value_dim_;
         o_width_ = (int64_t)heads_ * value_dim_;
+        g_width_ = has_gate_ ? o_width_ : 0;
+        if (has_gate_ && has_bias_) throw ConfigError("attention: biases beside an output gate are not supported");
     }
 
     // ---- weights ----------------------------------------------------------------------------------------------
@@ -175,8 +194,9 @@ public:
                                      {name_of("v_proj"), {v_width_, hidden_}, Role::Matrix, Init::Normal},
                                      {name_of("o_proj"), {hidden_, o_width_}, Role::Matrix, Init::Normal}};
         if (value_mix_ == 2) s.push_back({name_of("value_mix_factor"), {}, Role::Vector, Init::Normal});
-        if (has_sink_) s.push_back({name_of("sink"), {heads_}, Role::Vector, Init::Normal});
-        if (has_norm_) {
+        if (has_sink_ && !constant_sink_) s.push_back({name_of("sink"), {heads_}, Role::Vector, Init::Normal});
+        if (has_gate_) s.push_back({name_of("gate_proj"), {g_width_, hidden_}, Role::Matrix, Init::Normal});
+        if (has_norm_ && norm_weight_) {
             s.push_back({name_of("q_norm"), {head_dim_}, Role::Vector, Init::Scale});
             s.push_back({name_of("k_norm"), {head_dim_}, Role::Vector, Init::Scale});
         }
@@ -189,11 +209,13 @@ public:
     }
 
     void bind(WeightSource& src) override {
-        // one matrix [q | k | v] so that the three projections are one product (a layout choice only)
-        Tensor parts[3] = {src.fetch(name_of("q_proj")), src.fetch(name_of("k_proj")), src.fetch(name_of("v_proj"))};
-        if (parts[0].dtype != parts[1].dtype || parts[0].dtype != parts[2].dtype)
-            throw WeightError(name_of("q_proj") + ", " + name_of("k_proj") + " and " + name_of("v_proj") + " are stored in different precisions");
-        Tensor qkv = src.arena().alloc(parts[0].dtype, {q_width_ + kv_width_ + v_width_, hidden_});
+        // one matrix [q | k | v | (g)] so that the projections are one product (a layout choice only)
+        std::vector<Tensor> parts = {src.fetch(name_of("q_proj")), src.fetch(name_of("k_proj")), src.fetch(name_of("v_proj"))};
+        if (has_gate_) parts.push_back(src.fetch(name_of("gate_proj")));
+        for (const Tensor& t : parts)
+            if (t.dtype != parts[0].dtype)
+                throw WeightError(name_of("q_proj") + ", " + name_of("k_proj") + " and " + name_of("v_proj") + " are stored in different precisions");
+        Tensor qkv = src.arena().alloc(parts[0].dtype, {q_width_ + kv_width_ + v_width_ + g_width_, hidden_});
         size_t off = 0;
         for (Tensor& t : parts) {
             QE_CUDA(cudaMemcpyAsync(static_cast<char*>(qkv.data) + off, t.data, t.bytes(), cudaMemcpyDeviceToDevice, src.stream()));
@@ -215,12 +237,22 @@ public:
         qkv_proj_ = Linear(qkv, "qkv_proj", gemm_);
         q_only_proj_ = Linear(qkv.rows(0, q_width_), "q_proj", gemm_);
         o_proj_ = Linear(src.fetch(name_of("o_proj")), "o_proj", gemm_);
-        if (has_norm_) {
+        auto constants = [&](const std::vector<float>& values) {
+            Tensor t = src.arena().alloc(DType::F32, {(int64_t)values.size()});
+            QE_CUDA(cudaMemcpyAsync(t.data, values.data(), values.size() * sizeof(float), cudaMemcpyHostToDevice, src.stream()));
+            QE_CUDA(cudaStreamSynchronize(src.stream()));
+            return t;
+        };
+        if (has_norm_ && norm_weight_) {
             q_norm_ = src.fetch(name_of("q_norm"));
             k_norm_ = src.fetch(name_of("k_norm"));
+        } else if (has_norm_) {
+            q_norm_ = k_norm_ = constants(std::vector<float>((size_t)head_dim_, 1.0f));
         }
         if (value_mix_ == 2) mix_factor_ = src.fetch(name_of("value_mix_factor"));
-        if (has_sink_) sink_ = src.fetch(name_of("sink"));
+        if (constant_sink_) sink_ = constants(std::vector<float>((size_t)heads_, (float)sink_value_));
+        else if (has_sink_) sink_ = src.fetch(name_of("sink"));
+        if (!slopes_host_.empty()) slopes_ = constants(slopes_host_);
         if (position_) {
             position_->bind(src);
             table_ = position_->rotation_table();
@@ -248,9 +280,9 @@ public:
     bool use_flash() const {
         if (compute_dtype != DType::BF16 || attention_ == "generic") return false;
         const int group = heads_ / kv_heads_;
-        // (of the tensor-core kernels the tcgen05 prompt kernel and the TMA decode kernel know sinks: heads of 128)
+        // (of the tensor-core kernels the tcgen05 prompt kernel and the TMA decode kernel know sinks, biases and gates: heads of 128)
         const bool ok = (head_dim_ == 64 || head_dim_ == 128) && value_dim_ == head_dim_ && group >= 1 && group <= 16 &&
-                        (!has_sink_ || head_dim_ == 128);
+                        (!extended() || head_dim_ == 128);
         if (!ok && attention_ == "flash")
             throw KernelError("the flash attention kernels do not take head_dim " + std::to_string(head_dim_) + " with " +
                               std::to_string(group) + " query heads per kv head");
@@ -260,14 +292,17 @@ public:
     // ---- cache and step metadata ------------------------------------------------------------------------------
     CacheNeed cache_need() const override { return CacheNeed::pages(kv_heads_, head_dim_, window_, value_dim_, chunk_); }
 
-    // attention with a sink in bfloat16 runs on the tensor-core kernel that knows sinks (a tile of 16 rows, all heads)
-    bool use_sink_kernel() const {
-        return has_sink_ && compute_dtype == DType::BF16 && attention_ != "generic" && !chunk_ &&
+    // a sink, a distance bias or a gate inside the attention kernel
+    bool extended() const { return has_sink_ || has_gate_ || !slopes_host_.empty(); }
+
+    // which in bfloat16 runs on the tensor-core kernel that knows them (a tile of 16 rows, all heads)
+    bool use_tile_kernel() const {
+        return extended() && compute_dtype == DType::BF16 && attention_ != "generic" && !chunk_ &&
                core_kernels().attention_talking_mma_supports(heads_, kv_heads_, head_dim_, value_dim_);
     }
 
     void prepare_step(StepPlan& plan) override {
-        if (use_sink_kernel()) add_tiles(plan, kTileAll, "attention.tiles16", true);
+        if (use_tile_kernel()) add_tiles(plan, kTileAll, "attention.tiles16", true);
         if (!use_flash()) return;
         bool portions = false;
         for (int n : plan.q_lens) portions |= n > 1;
@@ -298,7 +333,7 @@ public:
         const Linear& proj = cache.writable ? qkv_proj_ : q_only_proj_;
         // rows without their factor (RowScale): the product's epilogue applies it where it can, else the kernel behind it
         const bool scale_in_product = ctx.row_scale.defined() && proj.applies_row_scale(T, dt, false, true);
-        if (!cache.writable && value_mix_) throw Error(kInvalidState, "a layer that mixes values writes a cache of its own");
+        if (!cache.writable && (value_mix_ || has_gate_)) throw Error(kInvalidState, "a layer that mixes values or gates its heads writes a cache of its own");
         Addend qkv = proj(x, ctx, "qkv", dt, T, true, false, nullptr, scale_in_product ? &ctx.row_scale : nullptr);
         // the values of the first mixing layer, per token of the step: written by that layer, read by the later ones
         float* v_first = value_mix_ ? ws.get("attention.v_first", {T, v_width_}, DType::F32).as<float>() : nullptr;
@@ -307,19 +342,44 @@ public:
         Tensor q = ws.get("q", {T, heads_, head_dim_}, dt);
         const int column = position_ ? position_->position_column() : 0;
         const int32_t* positions = ctx.position_column(column);
+        const int64_t product_width = q_width_ + (int64_t)kv_heads_written * (head_dim_ + value_dim_) + g_width_;
+        // the gate's logits stay where the product left them, or, as partial sums or without their row's factor, are finished
+        // by the kernel that finishes q, k and v
+        Tensor gate_rows;
+        const void* gate = nullptr;
+        long long gate_stride = 0;
+        if (has_gate_) {
+            if (qkv.splits > 1 || later.defined() || qkv.tensor.dtype != dt) {
+                gate_rows = ws.get("attn_gate", {T, o_width_}, dt);
+                gate = gate_rows.data;
+                gate_stride = o_width_;
+            } else {
+                gate = static_cast<const char*>(qkv.tensor.data) + (size_t)(product_width - g_width_) * dtype_size(dt);
+                gate_stride = product_width;
+            }
+        }
         if (LaunchProfile::get().on()) {       // reads the product's rows (every split), writes q and the cache rows
-            const double row = (double)(q_width_ + (int64_t)kv_heads_written * (head_dim_ + value_dim_));
+            const double row = (double)(q_width_ + (int64_t)kv_heads_written * (head_dim_ + value_dim_) + (gate_rows.defined() ? g_width_ : 0));
             LaunchProfile::get().note_cost((double)T * row * (qkv.splits * dtype_size(qkv.tensor.dtype) + dtype_size(dt)), 0.0);
         }
-        QE_LAUNCH(core, core.qk_norm_rope_kv_write(
-            qkv.tensor.data, qkv.tensor.code(), qkv.splits, (long long)T * (q_width_ + (int64_t)kv_heads_written * (head_dim_ + value_dim_)),
-            bias_.defined() ? bias_.as<float>() : nullptr, has_norm_ ? q_norm_.as<float>() : nullptr,
-            has_norm_ ? k_norm_.as<float>() : nullptr, (float)eps_, table_.defined() ? table_.as<float>() : nullptr,
-            position_ ? position_->n_rot() : 0, table_.defined() ? (int)table_.shape[0] : 0, positions,
-            cache.writable ? g.slot_mapping : nullptr, q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype,
-            cache.page_stride, cache.page_size, T, heads_, kv_heads_written, head_dim_,
-            position_ && position_->interleaved() ? 1 : 0, later.sumsq, later.chunks, later.width, later.eps, value_dim_, v_first,
-            mix_factor_.defined() ? mix_factor_.as<float>() : nullptr, value_mix_, ctx.stream));
+        if (has_gate_)
+            QE_LAUNCH(core, core.qk_norm_rope_gate_kv_write(
+                qkv.tensor.data, qkv.tensor.code(), qkv.splits, (long long)T * product_width, nullptr, has_norm_ ? q_norm_.as<float>() : nullptr,
+                has_norm_ ? k_norm_.as<float>() : nullptr, (float)eps_, table_.defined() ? table_.as<float>() : nullptr,
+                position_ ? position_->n_rot() : 0, table_.defined() ? (int)table_.shape[0] : 0, positions, g.slot_mapping, q.data, q.code(),
+                cache.k_base, cache.v_base, (int)cache.kv_dtype, cache.page_stride, cache.page_size, T, heads_, kv_heads_written, head_dim_,
+                position_ && position_->interleaved() ? 1 : 0, later.sumsq, later.chunks, later.width, later.eps, value_dim_, v_first,
+                mix_factor_.defined() ? mix_factor_.as<float>() : nullptr, value_mix_, product_width, gate_rows.data, ctx.stream));
+        else
+            QE_LAUNCH(core, core.qk_norm_rope_kv_write(
+                qkv.tensor.data, qkv.tensor.code(), qkv.splits, (long long)T * (q_width_ + (int64_t)kv_heads_written * (head_dim_ + value_dim_)),
+                bias_.defined() ? bias_.as<float>() : nullptr, has_norm_ ? q_norm_.as<float>() : nullptr,
+                has_norm_ ? k_norm_.as<float>() : nullptr, (float)eps_, table_.defined() ? table_.as<float>() : nullptr,
+                position_ ? position_->n_rot() : 0, table_.defined() ? (int)table_.shape[0] : 0, positions,
+                cache.writable ? g.slot_mapping : nullptr, q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype,
+                cache.page_stride, cache.page_size, T, heads_, kv_heads_written, head_dim_,
+                position_ && position_->interleaved() ? 1 : 0, later.sumsq, later.chunks, later.width, later.eps, value_dim_, v_first,
+                mix_factor_.defined() ? mix_factor_.as<float>() : nullptr, value_mix_, ctx.stream));
         Tensor out = ws.get("attn_out", {T, o_width_}, dt);
         const int32_t* abs_positions = ctx.position_column(0);       // the mask always follows the index in the request
         if (LaunchProfile::get().on()) {
@@ -338,14 +398,15 @@ public:
                                            2.0 * seen * heads_ * (head_dim_ + value_dim_));
         }
         const StepArray t16 = ctx.array("attention.tiles16.seg"), t16f = ctx.array("attention.tiles16.first");
-        // a sink rides in the tcgen05 prompt kernel and the TMA decode kernel only: pages they take, and no other choice by option
+        // a sink, a bias and a gate ride in the tcgen05 prompt kernel and the TMA decode kernel only: pages they take, and no
+        // other choice by option
         const bool pages_ok = (cache.page_size == 8 || cache.page_size == 16 || cache.page_size == 32 || cache.page_size == 64) && cache.num_pages > 0;
-        const bool sink_ok = !has_sink_ || (pages_ok && ctx.option("prefill_kernel") != "mma_sync" && ctx.option("decode_kernel") != "cp_async" &&
-                                            ctx.option("sink_kernel") != "tile");
-        if (use_flash() && sink_ok) {
+        const bool extras_ok = !extended() || (pages_ok && ctx.option("prefill_kernel") != "mma_sync" && ctx.option("decode_kernel") != "cp_async" &&
+                                              ctx.option("sink_kernel") != "tile");
+        if (use_flash() && extras_ok) {
             if (cache.kv_dtype != DType::BF16) throw KernelError("attention_flash: the cache must be bfloat16");
-            flash(q, cache, g, ctx, out, abs_positions);
-        } else if (use_sink_kernel() && cache.kv_dtype == DType::BF16 && t16.count) {
+            flash(q, cache, g, ctx, out, abs_positions, gate, gate_stride);
+        } else if (use_tile_kernel() && cache.kv_dtype == DType::BF16 && t16.count) {
             int splits = (int)ctx.option_int("tile16_splits");
             if (splits < 1)
                 splits = tile16_splits(t16.count, std::max(ctx.decode_max_ctx, ctx.prefill_max_ctx), window_,
@@ -358,13 +419,13 @@ public:
             }
             QE_LAUNCH(core, core.attention_talking_mma(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, g.block_table,
                                                        g.table_width, ctx.seg_start, ctx.seg_ctx_len, t16.data, t16f.data, t16.count, out.data,
-                                                       heads_, kv_heads_, head_dim_, value_dim_, window_, 0, (float)scale_, 0.0f, nullptr,
-                                                       nullptr, nullptr, sink_.as<float>(), nullptr, 0, splits, T, part_o, part_ml, ctx.stream));
-        } else if (has_sink_) {
-            QE_LAUNCH(core, core.attention_generic_sink(q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype, cache.page_stride,
-                                                        cache.page_size, g.block_table, g.table_width, ctx.row_seg, abs_positions, out.data,
-                                                        out.code(), T, heads_, kv_heads_, head_dim_, window_, (float)scale_, value_dim_, chunk_, 0,
-                                                        sink_.as<float>(), ctx.stream));
+                                                       heads_, kv_heads_, head_dim_, value_dim_, window_, 0, (float)scale_, 0.0f, slopes(),
+                                                       nullptr, nullptr, sink(), gate, gate_stride, splits, T, part_o, part_ml, ctx.stream));
+        } else if (extended()) {
+            QE_LAUNCH(core, core.attention_generic_biased(q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype, cache.page_stride,
+                                                          cache.page_size, g.block_table, g.table_width, ctx.row_seg, abs_positions, out.data,
+                                                          out.code(), T, heads_, kv_heads_, head_dim_, window_, (float)scale_, value_dim_, chunk_, 0,
+                                                          sink(), slopes(), gate, gate_stride, ctx.stream));
         } else {
             QE_LAUNCH(core, core.attention_generic(q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype, cache.page_stride,
                                                    cache.page_size, g.block_table, g.table_width, ctx.row_seg, abs_positions, out.data,
@@ -376,7 +437,8 @@ public:
 
 private:
     // All rows of the step: q [T, HQ, D] bfloat16 -> out [T, HQ * D] bfloat16.
-    void flash(const Tensor& q, const CacheView& cache, const GroupStep& g, StepContext& ctx, Tensor& out, const int32_t* positions) {
+    void flash(const Tensor& q, const CacheView& cache, const GroupStep& g, StepContext& ctx, Tensor& out, const int32_t* positions,
+               const void* gate, long long gate_stride) {
         const FlashKernels& f = flash_kernels();
         Workspace& ws = *ctx.workspace;
         const int sms = sm_count();
@@ -391,18 +453,18 @@ private:
                 part_o = ws.get("attn_tile_part_o", {ctx.T, heads_, splits, head_dim_}, DType::F32).as<float>();
                 part_ml = ws.get("attn_tile_part_ml", {ctx.T, heads_, splits, 2}, DType::F32).as<float>();
             }
-            if (has_sink_)
-                QE_LAUNCH(f, f.prefill_tc5_sink(q.data, ctx.T, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages,
+            if (extended())
+                QE_LAUNCH(f, f.prefill_tc5_biased(q.data, ctx.T, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages,
                                                 g.block_table, g.table_width, ctx.seg_start, ctx.seg_ctx_len, t128.data, t128f.data, t128.count,
                                                 out.data, heads_, kv_heads_, head_dim_, window_, chunk_, (float)scale_, splits, part_o, part_ml,
-                                                ctx.attention_error, sink_.as<float>(), ctx.stream));
+                                                ctx.attention_error, sink(), slopes(), gate, gate_stride, ctx.stream));
             else
                 QE_LAUNCH(f, f.prefill_tc5(q.data, ctx.T, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages,
                                            g.block_table, g.table_width, ctx.seg_start, ctx.seg_ctx_len, t128.data, t128f.data, t128.count,
                                            out.data, heads_, kv_heads_, head_dim_, window_, chunk_, (float)scale_, splits, part_o, part_ml,
                                            ctx.attention_error, ctx.stream));
         } else if (t64.count) {
-            if (has_sink_) throw Error(kInvalidState, "attention: the tiled prompt kernel knows no sink");
+            if (extended()) throw Error(kInvalidState, "attention: the tiled prompt kernel knows no sink, bias or gate");
             QE_LAUNCH(f, f.prefill(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, g.block_table, g.table_width,
                                    ctx.seg_start, ctx.seg_ctx_len, t64.data, t64f.data, t64.count, out.data, heads_, kv_heads_,
                                    head_dim_, window_, chunk_, (float)scale_, ctx.stream));
@@ -420,31 +482,35 @@ private:
             part_o = ws.get("attn_part_o", {n, heads_, splits, head_dim_}, DType::F32).as<float>();
             part_ml = ws.get("attn_part_ml", {n, heads_, splits, 2}, DType::F32).as<float>();
         }
-        if (bulk && has_sink_)
-            QE_LAUNCH(f, f.decode_bulk_sink(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages, g.block_table,
+        if (bulk && extended())
+            QE_LAUNCH(f, f.decode_bulk_biased(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages, g.block_table,
                                             g.table_width, ctx.decode_rows, n, ctx.row_seg, positions, part_o, part_ml, out.data, heads_,
                                             kv_heads_, head_dim_, splits, window_, chunk_, (float)scale_, 0, ctx.attention_error,
-                                            sink_.as<float>(), ctx.stream));
+                                            sink(), slopes(), gate, gate_stride, ctx.stream));
         else if (bulk)
             QE_LAUNCH(f, f.decode_bulk(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages, g.block_table,
                                        g.table_width, ctx.decode_rows, n, ctx.row_seg, positions, part_o, part_ml, out.data, heads_,
                                        kv_heads_, head_dim_, splits, window_, chunk_, (float)scale_, 0, ctx.attention_error, ctx.stream));
-        else if (has_sink_)
-            throw Error(kInvalidState, "attention: the cp.async decode kernel knows no sink");
+        else if (extended())
+            throw Error(kInvalidState, "attention: the cp.async decode kernel knows no sink, bias or gate");
         else
             QE_LAUNCH(f, f.decode(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, g.block_table, g.table_width,
                                   ctx.decode_rows, n, ctx.row_seg, positions, part_o, part_ml, out.data, heads_, kv_heads_, head_dim_,
                                   splits, window_, chunk_, (float)scale_, ctx.stream));
     }
 
-    int64_t hidden_, q_width_, kv_width_, v_width_, o_width_;
+    const float* sink() const { return sink_.defined() ? sink_.as<float>() : nullptr; }
+    const float* slopes() const { return slopes_.defined() ? slopes_.as<float>() : nullptr; }
+
+    int64_t hidden_, q_width_, kv_width_, v_width_, o_width_, g_width_;
     int heads_, kv_heads_, head_dim_, value_dim_, window_, chunk_ = 0, value_mix_ = 0;
-    bool has_norm_, has_bias_, has_sink_ = false;
-    double eps_, scale_;
+    bool has_norm_, norm_weight_ = true, has_bias_, has_sink_ = false, constant_sink_ = false, has_gate_ = false;
+    double eps_, scale_, sink_value_ = 0.0;
+    std::vector<float> slopes_host_;
     std::string gemm_, attention_;
     std::shared_ptr<PositionEncoding> position_;
     Linear qkv_proj_, q_only_proj_, o_proj_;
-    Tensor q_norm_, k_norm_, bias_, table_, mix_factor_, sink_;
+    Tensor q_norm_, k_norm_, bias_, table_, mix_factor_, sink_, slopes_;
 };
 
 // Grouped-query attention whose heads talk to each other before the softmax.

@@ -21,6 +21,13 @@
 // keep_embedding_output), W [E, 2E], step [passes, E] and pass the run-order entry's LayerCall::pass.  It has no mixer,
 // keeps nothing in the cache, and stands in the run order in front of each round of a stretch of layers that runs
 // several times.  Layer params: hidden_size, passes, names{weight, step}.
+//
+// hyper_connection: the residual is `lanes` rows per token (ResidualStream::n_lanes), X[0 .. s-1], each what the embedding
+// gave at first.  A part f with vectors in, out [s] and a matrix mix [s, s] of its own reads u = sum_s in[s] X[s], gives
+// y = f(norm(u)), and X'[t] = sum_s mix[s][t] X[s] + out[t] y.  The update waits with the part's addend and the next
+// norm's kernel does update, read and norm in one pass over the lanes; the model's final norm reads the lanes' sum.
+// Sub-parts by name as in pre_norm (a layer may come without a feed-forward).  Layer params: lanes, mixer_names{in, out,
+// mix}, feed_forward_names{in, out, mix}.
 #include "linear.h"
 #include "parts.h"
 
@@ -236,6 +243,76 @@ private:
     std::shared_ptr<ReinjectWeights> weights_;
 };
 
+// One part's weights of a residual of several lanes, as a part so that the loader, the folder check and random weights see them.
+class LaneWeights : public Part {
+public:
+    LaneWeights(const Json& p, BuildContext& b) : Part(p, b), lanes_(p.at("lanes").as_int()) {
+        if (lanes_ < 1 || lanes_ > kMaxLanes) throw ConfigError("hyper_connection: 1 to " + std::to_string(kMaxLanes) + " lanes, not " + std::to_string(lanes_));
+    }
+    std::vector<TensorSpec> tensor_specs() const override {
+        return {{name_of("in"), {lanes_}, Role::Vector, Init::Scale}, {name_of("out"), {lanes_}, Role::Vector, Init::Scale},
+                {name_of("mix"), {lanes_, lanes_}, Role::Vector, Init::Normal}};
+    }
+    void bind(WeightSource& src) override {
+        in = src.fetch(name_of("in"));
+        out = src.fetch(name_of("out"));
+        mix = src.fetch(name_of("mix"));
+    }
+    LaneUpdate update() const {
+        LaneUpdate u;
+        u.mix = mix.as<float>(); u.out = out.as<float>();
+        return u;
+    }
+    static constexpr int64_t kMaxLanes = 32;
+    int64_t lanes_;
+    Tensor in, out, mix;
+};
+
+class HyperConnectionBlock : public Arrangement {
+public:
+    HyperConnectionBlock(const LayerSpec& layer, BuildContext& build) {
+        mixer_norm_ = make_part_as<Norm>("norm", layer.part("mixer_norm"), build);
+        mixer_ = make_part_as<Mixer>("mixer", layer.part("mixer"), build);
+        mixer_lanes_ = weights(layer, "mixer_names", build);
+        if (layer.has("feed_forward")) {
+            ff_norm_ = make_part_as<Norm>("norm", layer.part("feed_forward_norm"), build);
+            ff_ = make_part_as<FeedForward>("feed_forward", layer.part("feed_forward"), build);
+            ff_lanes_ = weights(layer, "feed_forward_names", build);
+        }
+    }
+    std::vector<Part*> parts() override {
+        std::vector<Part*> p = {mixer_norm_.get(), mixer_.get(), mixer_lanes_.get()};
+        if (ff_) { p.push_back(ff_norm_.get()); p.push_back(ff_.get()); p.push_back(ff_lanes_.get()); }
+        return p;
+    }
+    CacheNeed cache_need() const override { return mixer_->cache_need(); }
+    bool takes_lanes() const override { return true; }
+    void forward(ResidualStream& stream, StepContext& ctx, const CacheView& cache) override {
+        if (stream.n_lanes != (int)mixer_lanes_->lanes_) throw Error(kInvalidState, "hyper_connection: the residual does not have this layer's lanes");
+        // no product adds into the lanes itself, and no norm's work is handed to a product
+        ctx.residual = nullptr;
+        ctx.residual_width = 0;
+        ctx.row_scale = RowScale();
+        ctx.norm_ahead = NormAhead();
+        Tensor xn = mixer_norm_->forward_lanes(stream, ctx, mixer_lanes_->in.as<float>());
+        stream.add_to_lanes(mixer_->forward(xn, ctx, cache), mixer_lanes_->update());
+        if (!ff_) return;
+        xn = ff_norm_->forward_lanes(stream, ctx, ff_lanes_->in.as<float>());
+        stream.add_to_lanes(ff_->forward(xn, ctx), ff_lanes_->update());
+    }
+private:
+    static std::shared_ptr<LaneWeights> weights(const LayerSpec& layer, const char* names, BuildContext& build) {
+        Json p = Json::object();
+        p.set("lanes", layer.params.at("lanes"));
+        p.set("names", layer.params.at(names));
+        return std::make_shared<LaneWeights>(p, build);
+    }
+    std::shared_ptr<Norm> mixer_norm_, ff_norm_;
+    std::shared_ptr<Mixer> mixer_;
+    std::shared_ptr<FeedForward> ff_;
+    std::shared_ptr<LaneWeights> mixer_lanes_, ff_lanes_;
+};
+
 void register_norm_parts();
 void register_routed_parts();
 void register_state_space_parts();
@@ -269,6 +346,9 @@ void register_builtin_parts() {
     });
     register_arrangement("reinject", [](const LayerSpec& layer, BuildContext& build) {
         return std::unique_ptr<Arrangement>(new ReinjectBlock(layer, build));
+    });
+    register_arrangement("hyper_connection", [](const LayerSpec& layer, BuildContext& build) {
+        return std::unique_ptr<Arrangement>(new HyperConnectionBlock(layer, build));
     });
     register_arrangement("pre_norm", [](const LayerSpec& layer, BuildContext& build) {
         return std::unique_ptr<Arrangement>(new PreNormBlock(layer, build));

@@ -4,13 +4,15 @@
 //     [c' | r] = W_dkv h,  c = rmsnorm(c'; w_kv)            c: kv_rank wide, r: rot_dim wide, one rotated key part for all heads
 //     head a:  k = [W_uk_a c | rot(r)],  v = W_uv_a c,  score = (q_plain . k_plain + rot(q_rot) . rot(r)) * scale
 //     o_a = softmax over the visible positions (all earlier ones, or the last `window`) of the scores, times v
-//     y = W_o concat_a(o_a * sigmoid(W_g h)_a)              "gate": true; without it the heads' outputs go to W_o as they are
+//     y = W_o concat_a(o_a * sigmoid(W_g h)_a)              "gate": true (one logit per head) or "values" (one per value);
+//                                                           without it the heads' outputs go to W_o as they are
+// Without a query latent ("q_rank" null) q = W_q h (names.q_proj); "rot_dim" 0: no position enters at all.
 //
 // A token leaves only [c | rot(r)] in the cache: one row of kv_rank + rot_dim numbers and no value rows
 // (CacheNeed::rows).  Keys and values are never made: q_plain . (W_uk_a c) = (W_uk_a^T q_plain) . c and
 // sum_j p_j W_uv_a c_j = W_uv_a sum_j p_j c_j, so every head attends over the same cached rows with the query
 // [W_uk_a^T q_plain | rot(q_rot)], takes the weighted sum of the rows' first kv_rank numbers, and W_uv_a expands that.
-// The down projections W_dq, W_dkv and W_g are one product over the stacked matrices.  Norms, rotation, scores, softmax
+// The projections of h (W_dq or W_q, W_dkv, W_g) are one product over the stacked matrices.  Norms, rotation, scores, softmax
 // and the sums over the latent are float32 in every mode.
 //
 // In bfloat16 the attention runs on the tensor cores (latent_attention_mma.cu): the (token, head) pairs of a portion,
@@ -24,9 +26,10 @@
 
 namespace qe {
 
-// params: hidden_size, num_heads, head_dim (plain dimensions of a head), rot_dim (rotated ones), value_dim, q_rank, kv_rank,
-// norm_eps, scale, window (null: all positions), gate (default false), position (a PartSpec as {kind, params} whose n_rot is
-// at most rot_dim, or null), names{q_down, q_norm, q_up, kv_down, kv_norm, k_up, v_up, o_proj, gate (with "gate": true)}.
+// params: hidden_size, num_heads, head_dim (plain dimensions of a head), rot_dim (rotated ones), value_dim, q_rank (null: no
+// query latent), kv_rank, norm_eps, scale, window (null: all positions), gate (default false; true, or "values"), position (a PartSpec as {kind, params} whose n_rot is
+// at most rot_dim, or null), names{q_down, q_norm, q_up (or q_proj, without a query latent), kv_down, kv_norm, k_up,
+// v_up, o_proj, gate (with a gate)}.
 class LatentAttention : public Mixer {
 public:
     LatentAttention(const Json& p, BuildContext& b) : Mixer(p, b) {
@@ -35,13 +38,23 @@ public:
         dim_ = (int)p.at("head_dim").as_int();
         rot_ = (int)p.at("rot_dim").as_int();
         vdim_ = (int)p.at("value_dim").as_int();
-        q_rank_ = (int)p.at("q_rank").as_int();
+        const Json* qr = p.find("q_rank");
+        direct_q_ = !qr || qr->is_null();
+        q_cols_ = direct_q_ ? heads_ * (dim_ + rot_) : (int)qr->as_int();
         kv_rank_ = (int)p.at("kv_rank").as_int();
         eps_ = p.at("norm_eps").as_double();
         scale_ = p.at("scale").as_double();
         window_ = (int)p.get_int("window", 0);
-        gated_ = p.get_bool("gate", false);
-        if (heads_ < 1 || dim_ < 1 || rot_ < 0 || vdim_ < 1 || q_rank_ < 1 || kv_rank_ < 1 || window_ < 0)
+        if (const Json* gate = p.find("gate")) {
+            if (gate->is_string()) {
+                if (gate->as_string() != "values") throw ConfigError("latent_attention: gate is true, false or 'values', got '" + gate->as_string() + "'");
+                gate_cols_ = vdim_;
+            } else if (!gate->is_null() && p.get_bool("gate", false)) {
+                gate_cols_ = 1;
+            }
+        }
+        gated_ = gate_cols_ > 0;
+        if (heads_ < 1 || dim_ < 1 || rot_ < 0 || vdim_ < 1 || q_cols_ < 1 || kv_rank_ < 1 || window_ < 0)
             throw ConfigError("latent_attention: heads, head_dim, value_dim and the ranks must be positive");
         if (kv_rank_ + rot_ > kMaxRow)
             throw ConfigError("latent_attention: a cache row of " + std::to_string(kv_rank_ + rot_) + " numbers exceeds the supported " +
@@ -60,28 +73,32 @@ public:
         }
         gemm_ = b.options.get_string("gemm", "auto");
         attention_ = b.options.get_string("attention", "auto");
-        down_width_ = (int64_t)q_rank_ + kv_rank_ + rot_ + (gated_ ? heads_ : 0);
+        down_width_ = (int64_t)q_cols_ + kv_rank_ + rot_ + (int64_t)heads_ * gate_cols_;
     }
 
     std::vector<TensorSpec> tensor_specs() const override {
-        std::vector<TensorSpec> s = {{name_of("q_down"), {q_rank_, hidden_}, Role::Matrix, Init::Normal},
-                                     {name_of("q_norm"), {q_rank_}, Role::Vector, Init::Scale},
-                                     {name_of("q_up"), {(int64_t)heads_ * (dim_ + rot_), q_rank_}, Role::Matrix, Init::Normal},
-                                     {name_of("kv_down"), {(int64_t)kv_rank_ + rot_, hidden_}, Role::Matrix, Init::Normal},
-                                     {name_of("kv_norm"), {kv_rank_}, Role::Vector, Init::Scale},
-                                     {name_of("k_up"), {(int64_t)heads_ * dim_, kv_rank_}, Role::Matrix, Init::Normal},
-                                     {name_of("v_up"), {(int64_t)heads_ * vdim_, kv_rank_}, Role::Matrix, Init::Normal},
-                                     {name_of("o_proj"), {hidden_, (int64_t)heads_ * vdim_}, Role::Matrix, Init::Normal}};
-        if (gated_) s.push_back({name_of("gate"), {heads_, hidden_}, Role::Matrix, Init::Normal});
+        std::vector<TensorSpec> s;
+        if (direct_q_) s = {{name_of("q_proj"), {q_cols_, hidden_}, Role::Matrix, Init::Normal}};
+        else s = {{name_of("q_down"), {q_cols_, hidden_}, Role::Matrix, Init::Normal},
+                  {name_of("q_norm"), {q_cols_}, Role::Vector, Init::Scale},
+                  {name_of("q_up"), {(int64_t)heads_ * (dim_ + rot_), q_cols_}, Role::Matrix, Init::Normal}};
+        for (const TensorSpec& t : {TensorSpec{name_of("kv_down"), {(int64_t)kv_rank_ + rot_, hidden_}, Role::Matrix, Init::Normal},
+                                    TensorSpec{name_of("kv_norm"), {kv_rank_}, Role::Vector, Init::Scale},
+                                    TensorSpec{name_of("k_up"), {(int64_t)heads_ * dim_, kv_rank_}, Role::Matrix, Init::Normal},
+                                    TensorSpec{name_of("v_up"), {(int64_t)heads_ * vdim_, kv_rank_}, Role::Matrix, Init::Normal},
+                                    TensorSpec{name_of("o_proj"), {hidden_, (int64_t)heads_ * vdim_}, Role::Matrix, Init::Normal}})
+            s.push_back(t);
+        if (gated_) s.push_back({name_of("gate"), {(int64_t)heads_ * gate_cols_, hidden_}, Role::Matrix, Init::Normal});
         return s;
     }
 
     void bind(WeightSource& src) override {
-        // one matrix [q_down | kv_down | gate]: the projections of h are one product (a layout choice only)
-        std::vector<Tensor> parts = {src.fetch(name_of("q_down")), src.fetch(name_of("kv_down"))};
+        // one matrix [q_down or q_proj | kv_down | gate]: the projections of h are one product (a layout choice only)
+        const std::string& q_first = name_of(direct_q_ ? "q_proj" : "q_down");
+        std::vector<Tensor> parts = {src.fetch(q_first), src.fetch(name_of("kv_down"))};
         if (gated_) parts.push_back(src.fetch(name_of("gate")));
         for (Tensor& t : parts)
-            if (t.dtype != parts[0].dtype) throw WeightError("the down projections of " + name_of("q_down") + "'s mixer are stored in different precisions");
+            if (t.dtype != parts[0].dtype) throw WeightError("the projections of " + q_first + "'s mixer are stored in different precisions");
         Tensor all = src.arena().alloc(parts[0].dtype, {down_width_, hidden_});
         size_t off = 0;
         for (Tensor& t : parts) {
@@ -91,8 +108,10 @@ public:
         QE_CUDA(cudaStreamSynchronize(src.stream()));
         for (Tensor& t : parts) src.release(t);
         down_proj_ = Linear(all, "latent_down", gemm_);
-        q_up_ = Linear(src.fetch(name_of("q_up")), "q_up", gemm_);
-        q_norm_ = src.fetch(name_of("q_norm"));
+        if (!direct_q_) {
+            q_up_ = Linear(src.fetch(name_of("q_up")), "q_up", gemm_);
+            q_norm_ = src.fetch(name_of("q_norm"));
+        }
         kv_norm_ = src.fetch(name_of("kv_norm"));
         k_up_ = src.fetch(name_of("k_up"));
         v_up_ = src.fetch(name_of("v_up"));
@@ -162,22 +181,26 @@ public:
         const int max_pos = table_.defined() ? (int)table_.shape[0] : 0;
         const size_t es = dtype_size(dt);
 
-        Tensor down = down_proj_(x, ctx, "la_down", dt, T).tensor;                            // [T, c_q' | c' | r | gate logits]
-        Tensor cq = ws.get("la_cq", {T, q_rank_}, dt);
-        if (LaunchProfile::get().on()) LaunchProfile::get().note_cost((double)T * (down_width_ + q_rank_ + row) * es, 0.0);
-        QE_LAUNCH(k, k.latent_prepare(down.data, down.code(), down_width_, q_rank_, kv_rank_, rot_, q_norm_.as<float>(), kv_norm_.as<float>(),
-                                      (float)eps_, table, n_rot, max_pos, positions, g.slot_mapping, cq.data, cq.code(), cache.k_base,
-                                      (int)cache.kv_dtype, cache.page_stride, cache.page_size, T, ctx.stream));
-        Tensor q = q_up_(cq, ctx, "la_q", dt, T).tensor;                                      // [T, heads, plain | rotated]
+        Tensor down = down_proj_(x, ctx, "la_down", dt, T).tensor;                            // [T, c_q' or q | c' | r | gate logits]
+        Tensor cq;
+        if (!direct_q_) cq = ws.get("la_cq", {T, q_cols_}, dt);
+        if (LaunchProfile::get().on())
+            LaunchProfile::get().note_cost((double)T * (direct_q_ ? 2.0 * row : (double)(q_cols_ + row) * 2.0) * es, 0.0);
+        QE_LAUNCH(k, k.latent_prepare(down.data, down.code(), down_width_, q_cols_, kv_rank_, rot_, direct_q_ ? nullptr : q_norm_.as<float>(),
+                                      kv_norm_.as<float>(), (float)eps_, table, n_rot, max_pos, positions, g.slot_mapping, cq.data, (int)dt,
+                                      cache.k_base, (int)cache.kv_dtype, cache.page_stride, cache.page_size, T, ctx.stream));
+        // [T, heads, plain | rotated]: the up product's rows, or the first columns of the stacked product's
+        Tensor q = direct_q_ ? down : q_up_(cq, ctx, "la_q", dt, T).tensor;
+        const long long q_stride = direct_q_ ? down_width_ : (long long)heads_ * (dim_ + rot_);
         Tensor q_lat = ws.get("la_q_lat", {T, heads_, row}, dt);
         if (LaunchProfile::get().on())
             LaunchProfile::get().note_cost((double)T * heads_ * (dim_ + rot_ + row) * es + (double)k_up_.bytes(), 2.0 * T * heads_ * dim_ * kv_rank_);
         const bool tc_products = products_on_tensor_cores() && dt == DType::BF16;
         if (tc_products) {
             const LatentKernels& lk = latent_kernels();
-            QE_LAUNCH(lk, lk.latent_absorb(q.data, k_up_.data, table, n_rot, max_pos, positions, q_lat.data, T, heads_, dim_, rot_, kv_rank_, ctx.stream));
+            QE_LAUNCH(lk, lk.latent_absorb(q.data, q_stride, k_up_.data, table, n_rot, max_pos, positions, q_lat.data, T, heads_, dim_, rot_, kv_rank_, ctx.stream));
         } else
-        QE_LAUNCH(k, k.latent_absorb(q.data, q.code(), k_up_.data, k_up_.code(), table, n_rot, max_pos, positions, q_lat.data, q_lat.code(), T,
+        QE_LAUNCH(k, k.latent_absorb(q.data, q.code(), q_stride, k_up_.data, k_up_.code(), table, n_rot, max_pos, positions, q_lat.data, q_lat.code(), T,
                                      heads_, dim_, rot_, kv_rank_, ctx.stream));
         // every head reads the one cached row per position: keys the whole row, values its first kv_rank numbers
         Tensor o_lat = ws.get("la_o_lat", {T, heads_, kv_rank_}, DType::F32);
@@ -214,13 +237,13 @@ public:
                                          T, heads_, 1, row, window_, (float)scale_, kv_rank_, 0, row, ctx.stream));
         Tensor out = ws.get("la_heads", {T, (int64_t)heads_ * vdim_}, dt);
         if (LaunchProfile::get().on())
-            LaunchProfile::get().note_cost((double)T * heads_ * (kv_rank_ * 4.0 + vdim_ * es) + (double)v_up_.bytes(), 2.0 * T * heads_ * vdim_ * kv_rank_);
-        const char* gate = gated_ ? static_cast<const char*>(down.data) + (size_t)(q_rank_ + row) * es : nullptr;
+            LaunchProfile::get().note_cost((double)T * heads_ * (kv_rank_ * 4.0 + (vdim_ + gate_cols_) * es) + (double)v_up_.bytes(), 2.0 * T * heads_ * vdim_ * kv_rank_);
+        const char* gate = gated_ ? static_cast<const char*>(down.data) + (size_t)(q_cols_ + row) * es : nullptr;
         if (tc_products && T > kFewRows) {               // few rows: more CTAs with a warp per value column
             const LatentKernels& lk = latent_kernels();
-            QE_LAUNCH(lk, lk.latent_expand(o_lat.data, v_up_.data, gate, down_width_, out.data, T, heads_, kv_rank_, vdim_, ctx.stream));
+            QE_LAUNCH(lk, lk.latent_expand(o_lat.data, v_up_.data, gate, down_width_, gate_cols_, out.data, T, heads_, kv_rank_, vdim_, ctx.stream));
         } else
-        QE_LAUNCH(k, k.latent_expand(o_lat.data, o_lat.code(), v_up_.data, v_up_.code(), gate, down.code(), down_width_, out.data, out.code(), T,
+        QE_LAUNCH(k, k.latent_expand(o_lat.data, o_lat.code(), v_up_.data, v_up_.code(), gate, down.code(), down_width_, gate_cols_, out.data, out.code(), T,
                                      heads_, kv_rank_, vdim_, ctx.stream));
         return o_proj_(out, ctx, "la_out", DType::F32, T, true, false, ctx.residual, nullptr, &ctx.norm_ahead);
     }
@@ -246,8 +269,8 @@ private:
     static constexpr int kTileRows = 64;         // (token, head) pairs of a tile of the tensor-core kernel
     static constexpr int kMaxRow = 640;          // the widest cache row the attention kernel holds a query for
     int64_t hidden_, down_width_;
-    int heads_, dim_, rot_, vdim_, q_rank_, kv_rank_, window_;
-    bool gated_;
+    int heads_, dim_, rot_, vdim_, q_cols_, kv_rank_, window_, gate_cols_ = 0;      // q_cols_: columns in front of c' in the stacked product
+    bool gated_, direct_q_;
     double eps_, scale_;
     std::string gemm_, attention_;
     std::shared_ptr<PositionEncoding> position_;

@@ -10,7 +10,11 @@ DecoderModel::DecoderModel(ModelSpec spec, DType compute_dtype, Json options)
     register_builtin_parts();
     spec_.validate();
     embedding_ = make_part_as<Embedding>("embedding", spec_.embedding, build_);
-    for (const LayerSpec& layer : spec_.layers) layers_.push_back(make_arrangement(layer, build_));
+    for (const LayerSpec& layer : spec_.layers) {
+        layers_.push_back(make_arrangement(layer, build_));
+        if (layers_.back()->takes_lanes() != (spec_.residual_lanes > 0))
+            throw ConfigError("layers of kind '" + layer.arrangement + "' do not fit a residual of " + std::to_string(spec_.residual_lanes) + " lanes");
+    }
     final_norm_ = make_part_as<Norm>("norm", spec_.final_norm, build_);
     head_ = make_part_as<Head>("head", spec_.head, build_);
 }
@@ -91,6 +95,7 @@ Tensor DecoderModel::forward(StepContext& ctx, const std::vector<CacheView>& vie
                              const std::function<void(int, ResidualStream&, StepContext&)>& after_entry) {
     ResidualStream stream;
     stream.x = embedding_->forward(ctx);
+    stream.n_lanes = spec_.residual_lanes;
     ctx.embedding_output = nullptr;
     if (spec_.keep_embedding_output) {
         // the stream is rewritten in place from here on: what the embedding gave is kept beside it
@@ -108,7 +113,8 @@ Tensor DecoderModel::forward(StepContext& ctx, const std::vector<CacheView>& vie
     ctx.next_layer_norm = NormAhead();
     ctx.pass = 0;
     if (n_want == 0) return Tensor();
-    Tensor xn = final_norm_->forward(stream, ctx, want_rows, n_want);
+    Tensor xn = stream.n_lanes ? final_norm_->forward_lanes(stream, ctx, nullptr, want_rows, n_want)
+                               : final_norm_->forward(stream, ctx, want_rows, n_want);
     return head_->forward(xn, ctx, n_want);
 }
 

@@ -61,6 +61,39 @@ void fold_all_addends(ResidualStream& stream, StepContext& ctx) {
     stream.clear();
 }
 
+namespace {
+// One launch over a residual of several lanes: the pending addend enters the lanes, u = sum_s in[s] X[s], and u normed with
+// `weight` (null: u itself) goes to `out`.  Rows are gathered or all of them; gathered rows leave the stream as it was.
+void lanes_pass(ResidualStream& stream, StepContext& ctx, const float* in, const float* weight, float eps, const int32_t* rows, int n, Tensor& out) {
+    const int64_t E = stream.x.shape[1];
+    const int S = stream.n_lanes;
+    const CoreKernels& k = core_kernels();
+    const Addend* a = stream.has_pending ? &stream.pending : nullptr;
+    const bool first = !stream.lanes.defined();              // every lane is x
+    const float* src = first ? stream.x.as<float>() : stream.lanes.as<float>();
+    Tensor dst;
+    if (a && !rows) dst = first ? ctx.workspace->get("residual_lanes", {ctx.T, S, E}, DType::F32) : stream.lanes;
+    if (LaunchProfile::get().on()) {
+        double bytes = 4.0 * n * E * (first ? 1 : S) + (double)n * E * dtype_size(out.dtype);
+        if (a) bytes += (double)a->splits * n * E * dtype_size(a->tensor.dtype) + (dst.defined() ? 4.0 * n * E * S : 0.0);
+        LaunchProfile::get().note_cost(bytes, 0.0);
+    }
+    QE_LAUNCH(k, k.lanes_rmsnorm(src, first ? E : S * E, first ? 0 : E, dst.defined() ? dst.as<float>() : nullptr, a ? a->tensor.data : nullptr,
+                                 a ? a->tensor.code() : 0, a ? a->splits : 1, a ? (long long)ctx.T * E : 0, a ? stream.lane_update.mix : nullptr,
+                                 a ? stream.lane_update.out : nullptr, in, weight, eps, rows, n, (int)E, S, out.data, out.code(), ctx.stream));
+    if (rows) return;
+    if (dst.defined()) stream.lanes = dst;
+    stream.clear();
+}
+}  // namespace
+
+Tensor Norm::forward_lanes(ResidualStream& stream, StepContext& ctx, const float* in, const int32_t* rows, int n_rows) {
+    ResidualStream read;
+    read.x = ctx.workspace->get("lanes_read", {ctx.T, stream.x.shape[1]}, DType::F32);
+    lanes_pass(stream, ctx, in, nullptr, 0.0f, nullptr, ctx.T, read.x);
+    return forward(read, ctx, rows, n_rows);
+}
+
 // params: size, eps, names{weight}.
 class RMSNorm : public Norm {
 public:
@@ -117,6 +150,13 @@ public:
                                         (int)size_, out.data, out.code(), sumsq.as<float>(), chunks, ctx.stream));
         stream.clear();
         scale->sumsq = sumsq.as<float>(); scale->chunks = chunks; scale->width = (int)size_; scale->eps = (float)eps_;
+        return out;
+    }
+
+    Tensor forward_lanes(ResidualStream& stream, StepContext& ctx, const float* in, const int32_t* rows, int n_rows) override {
+        const int n = rows ? n_rows : ctx.T;
+        Tensor out = ctx.workspace->get(rows ? "normed_rows" : "normed", {n, size_}, compute_dtype);
+        lanes_pass(stream, ctx, in, weight_.as<float>(), (float)eps_, rows, n, out);
         return out;
     }
 

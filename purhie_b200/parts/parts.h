@@ -141,6 +141,7 @@ struct ModelSpec {
     int64_t hidden_size = 0, vocab_size = 0, max_position = 0;
     int position_columns = 1;    // columns of positions a step carries per row (column 0: the index in the request)
     PartSpec embedding, final_norm, head;
+    int residual_lanes = 0;               // rows per token of the residual stream (0: the ordinary single one; see ResidualStream)
     bool keep_embedding_output = false;   // the rows the embedding gave stay readable for the whole step (StepContext::embedding_output)
     std::vector<LayerSpec> layers;
     std::vector<LayerCall> schedule;
@@ -276,10 +277,25 @@ struct StepPlan {
     void add(const std::string& name, std::vector<int32_t> values) { arrays.emplace_back(name, std::move(values)); }
 };
 
+// How a pending addend y enters a residual of several lanes: X'[t] = sum_s mix[s][t] X[s] + out[t] y, all lanes at once
+// from the old ones.
+struct LaneUpdate {
+    const float* mix = nullptr;              // [lanes, lanes] float32 on the device, indexed [from][to]
+    const float* out = nullptr;              // [lanes]
+};
+
 // The float32 residual [T, E] plus an addend that the next norm folds in (x += addend, then norm), so that the
 // sum and the normalisation are one pass over the row.
+//
+// A residual may be several lanes wide (n_lanes > 0): n_lanes rows of E numbers per token that start as copies of what
+// the embedding gave and are mixed with each other at every addition.  Then `lanes` holds them [T, n_lanes, E] once an
+// addition has made them differ; until then (lanes undefined) every lane is x.  The pending addend waits with the
+// LaneUpdate that says how it enters, and Norm::forward_lanes() folds it in.
 struct ResidualStream {
     Tensor x;
+    int n_lanes = 0;
+    Tensor lanes;
+    LaneUpdate lane_update;                  // of the pending addend (n_lanes > 0)
     Addend pending;
     bool has_pending = false;
     Addend also;                             // a second addend (a layer whose two parts read the same rows), without a transform
@@ -299,6 +315,12 @@ struct ResidualStream {
     }
     // after add(): what the part's last product did for the norm ahead (nothing, if it did nothing)
     void prepare(const NormAhead& ahead) { prepared = (!has_pending && !has_also && ahead.done()) ? ahead : NormAhead(); }
+    // the pending addend of a residual of several lanes
+    void add_to_lanes(Addend a, const LaneUpdate& how) {
+        if (!a.tensor.defined() || a.transform.defined()) throw Error(kInvalidState, "a part of a layer with several lanes returns a plain addend");
+        lane_update = how;
+        add(std::move(a));
+    }
     void clear() { has_pending = false; pending = Addend(); has_also = false; also = Addend(); prepared = NormAhead(); }
 };
 
@@ -352,6 +374,10 @@ public:
     // What a product in front may do of this norm's work (NormAhead), if forward_unscaled() would pick it up from
     // stream.prepared; a norm that has no such form offers nothing.
     virtual NormAhead offer(const StepContext&) const { return NormAhead(); }
+    // For a residual of several lanes: the pending addend is folded into the lanes (for good unless rows are gathered, as
+    // in forward()), the lanes are read as u = sum_s in[s] X[s] (in [n_lanes] float32 on the device; null: their sum), and
+    // the normed u comes back.  A norm without a kernel of its own for this norms u in a second pass.
+    virtual Tensor forward_lanes(ResidualStream& stream, StepContext& ctx, const float* in, const int32_t* rows = nullptr, int n_rows = 0);
     // This norm as a transform of an addend (AddendTransform) with the given factor, for a layer that norms what a
     // part gives before adding it; a norm that has no such form throws.
     virtual AddendTransform as_transform(float factor) const;
@@ -411,6 +437,7 @@ public:
     virtual ~Arrangement() = default;
     virtual std::vector<Part*> parts() = 0;
     virtual CacheNeed cache_need() const = 0;            // of the layer's mixer
+    virtual bool takes_lanes() const { return false; }   // the layer works on a residual of several lanes (ResidualStream)
     virtual void forward(ResidualStream& stream, StepContext& ctx, const CacheView& cache) = 0;
     // The offer of the layer's first norm, if in this step it would take rows prepared by the layer in front (the
     // model hands it to that layer as ctx.next_layer_norm).
@@ -437,8 +464,8 @@ template <typename T> std::shared_ptr<T> make_part_as(const std::string& family,
 }
 
 // Registers the parts this library brings (rmsnorm, layernorm, none, dyntanh, rope_neox, attention, talking_attention,
-// latent_attention, mamba1, gated_linear_attention, lightning_attention, min_gru, side_by_side, swiglu, mlp, routed_glu, embedding, lm_head,
-// pre_norm, sandwich_norm, parallel, reinject).
+// latent_attention, mamba1, mamba2, gated_linear_attention, lightning_attention, min_gru, side_by_side, swiglu, mlp, routed_glu, embedding, lm_head,
+// pre_norm, sandwich_norm, parallel, reinject, hyper_connection).
 QE_API void register_builtin_parts();
 
 }  // namespace qe
