@@ -449,3 +449,54 @@ def add_scaled_rmsnorm(x, add, weight, eps, y, add_scale, *, add_splits=1, write
     call("core", "ph_add_scaled_rmsnorm", _ptr(x), _ptr(add), _code(add.dtype), add_splits, T * E, _ptr(weight), float(eps), None, T, E,
          _ptr(y), _code(y.dtype), 1 if write_x else 0, float(add_scale), _stream())
     return y
+
+
+# ---- a residual of several lanes, and the second Mamba form -----------------------------------------------------------
+register_signatures("core", {
+    "ph_lanes_rmsnorm": [c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_void_p,
+                         c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
+    "ph_ssd_scan": [c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
+                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "ph_ssd_chunk": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
+                     c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "ph_ssd_chunk_supports": [c_int, c_int, c_int],
+    "ph_gate_rms": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+})
+
+
+def lanes_rmsnorm(src, lanes, dst, add, mix, out, in_, weight, eps, y, *, rows=None) -> torch.Tensor:
+    """src [T, S, E] (or [T, E]: every lane is that row); add [splits, T, E] or None enters by mix [S, S] and out [S]; the
+    lanes afterwards go to dst [T, S, E] (or None); y = rms(sum_s in[s] X[s]) * weight (None: the sum itself)."""
+    _need(src, "src", torch.float32); _need(y, "y")
+    T, E = src.shape[0], src.shape[-1]
+    one = src.dim() == 2
+    n = T if rows is None else rows.numel()
+    call("core", "ph_lanes_rmsnorm", _ptr(src), E if one else lanes * E, 0 if one else E, _ptr(dst), _ptr(add),
+         _code(add.dtype) if add is not None else 0, add.shape[0] if add is not None else 1, T * E, _ptr(mix), _ptr(out), _ptr(in_), _ptr(weight),
+         float(eps), _ptr(rows), n, E, lanes, _ptr(y), _code(y.dtype), _stream())
+    return y
+
+
+def ssd_chunk_supports(value_dim: int, state: int, groups: int) -> bool:
+    f, _ = _fn("core", "ph_ssd_chunk_supports")
+    return bool(f(value_dim, state, groups))
+
+
+def ssd(kind, xbc, rows, dt_col, conv_col, dt_bias, a, d, state, seg_start, seg_slot, y, *, heads, value_dim, states, groups, taps,
+        rows_from=0, rows_to=0) -> torch.Tensor:
+    """The recurrence of the second Mamba form, ``kind`` "scan" (token by token) or "chunk" (on the tensor cores): xbc [T, x | B |
+    C], rows [T, in-projection], state [slots, floats] float32 (updated in place), y [T, heads * value_dim] float32."""
+    _need(xbc, "xbc"); _need(rows, "rows", xbc.dtype); _need(state, "state", torch.float32); _need(y, "y", torch.float32)
+    head = [_ptr(xbc), _ptr(rows)] + ([_code(xbc.dtype)] if kind == "scan" else [])
+    call("core", f"ph_ssd_{kind}", *head, rows.shape[-1], dt_col, conv_col, _ptr(dt_bias), _ptr(a), _ptr(d), _ptr(state), state.shape[-1],
+         _ptr(seg_start), _ptr(seg_slot), seg_slot.numel(), heads, value_dim, states, groups, taps, rows_from, rows_to, _ptr(y), _stream())
+    return y
+
+
+def gate_rms(y, z, weight, eps, out, *, parts) -> torch.Tensor:
+    """out = rms in ``parts`` equal parts of (y * silu(z)), times weight; z [T, stride] with its first columns read."""
+    _need(y, "y", torch.float32); _need(z, "z"); _need(out, "out")
+    T, inner = y.shape
+    call("core", "ph_gate_rms", _ptr(y), _ptr(z), _code(z.dtype), z.shape[-1], _ptr(weight), float(eps), _ptr(out), _code(out.dtype), T, inner,
+         parts, _stream())
+    return out
