@@ -21,6 +21,8 @@
 // nothing before its own block).  Pages past the tile's last token
 // come from an out-of-range coordinate (zeros), scores of invisible keys are replaced by -inf and value rows
 // after the last token inside its page are zeroed before P V, so unwritten page slots may hold anything.
+// Keys and values may also lie densely, a row per token with the heads side by side (made for the step from something
+// smaller that the cache holds): then a request's rows start at dense_base[segment] and a box is 64 rows of one head's half.
 // A distance bias (a slope per head) takes slope_h * (row - key) off the scaled scores before the softmax; a gate (rows of
 // logits, a number per output element) multiplies the output by its sigmoid where the row is stored or merged.
 // Every mbarrier wait is bounded and reports through an error word; TMEM is freed on every path.
@@ -79,6 +81,7 @@ struct Tc5Params {
     const float* sink;             // [HQ] float32 or null: exp(sink) joins each head's denominator, once per row
     const float* slopes;           // [HQ] float32 or null: taken off the scores per position of distance
     const __nv_bfloat16* gate; long long gate_stride;      // rows of HQ * D logits, or null
+    const int32_t* dense_base;     // [S] or null: keys and values are dense rows, the request's first one
 };
 
 __device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
@@ -289,10 +292,15 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
             if (lane < ppb * 2) {
                 const int pj = lane >> 1, half = lane & 1;
                 const int pos = lo_page + (b_first + b) * BN + (pj << psh);
-                int row = p.total_rows;                       // past the tile's last token: zeros
-                if (pos <= z_last) row = (int)((long long)table[pos >> psh] * p.rows_per_page + (long long)g * p.page_size);
+                int row = p.total_rows, col = half * 64;      // past the tile's last token: zeros
+                if (p.dense_base) {
+                    col += g * D;
+                    if (pos <= z_last) row = p.dense_base[seg] + pos;
+                } else if (pos <= z_last) {
+                    row = (int)((long long)table[pos >> psh] * p.rows_per_page + (long long)g * p.page_size);
+                }
                 unsigned char* dst = (is_v ? v_ring : k_ring) + stage * KV_BYTES + half * HALF_KV + (pj << psh) * 128;
-                tma_load_2d(dst, is_v ? &map_v : &map_k, full, half * 64, row);
+                tma_load_2d(dst, is_v ? &map_v : &map_k, full, col, row);
             }
         };
         for (int b = 0; b <= n_blocks && ok; ++b) {
@@ -581,7 +589,7 @@ EncodeTiledFn encode_fn() {
 bool encode(CUtensorMap* out, const void* base, int rank, const cuuint64_t* dims, const cuuint64_t* strides, const cuuint32_t* box) {
     static std::mutex mu;
     static std::map<std::tuple<const void*, int, cuuint64_t, cuuint64_t, cuuint64_t, cuuint32_t>, CUtensorMap> cache;
-    const auto key = std::make_tuple(base, rank, dims[1], strides[0], rank > 3 ? dims[3] : 0, box[1]);
+    const auto key = std::make_tuple(base, rank, dims[1], strides[0], rank > 3 ? dims[3] : dims[0], box[1]);
     std::lock_guard<std::mutex> lock(mu);
     auto it = cache.find(key);
     if (it != cache.end()) { *out = it->second; return true; }
@@ -603,6 +611,72 @@ bool encode(CUtensorMap* out, const void* base, int rank, const cuuint64_t* dims
 
 PH_DEFINE_LAST_ERROR(ph_flash5)
 
+namespace {
+// Where keys and values are: pages of the cache, or dense rows.
+struct KvPlace {
+    const void* k; const void* v;
+    long long page_stride; int page_size, num_pages;         // pages
+    const int32_t* block_table; int table_stride;
+    const int32_t* dense_base; long long row_width; int rows;      // dense rows, row_width elements apart (dense_base not null)
+};
+
+int launch_tc5(const void* q, long long q_stride, int T, const KvPlace& kv, const int32_t* seg_start, const int32_t* seg_ctx_len,
+               const int32_t* tile_seg, const int32_t* tile_first, int n_tiles, void* out, int HQ, int HKV, int head_dim, int window, int chunk,
+               float scale, int splits, float* part_o, float* part_ml, int* error_flag, const float* sink, const float* slopes,
+               const void* gate, long long gate_stride, cudaStream_t stream) {
+    const bool dense = kv.dense_base != nullptr;
+    if (!q || !kv.k || !kv.v || !seg_start || !seg_ctx_len || !tile_seg || !tile_first || !out || !error_flag || T < 1 || n_tiles < 0 || HQ < 1 ||
+        HKV < 1 || HQ % HKV || window < 0 || chunk < 0 || !(scale > 0.0f) || q_stride < (long long)HQ * D ||
+        (dense ? kv.rows < 1 || kv.row_width < (long long)HKV * D : !kv.block_table || kv.num_pages < 1))
+        return fail(PH_ERR_ARG, "attention_prefill_tc5: bad arguments (tiles %d, HQ %d, HKV %d)", n_tiles, HQ, HKV);
+    if (head_dim != D) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: head_dim %d is not %d", head_dim, D);
+    const int page_size = dense ? BN : kv.page_size;
+    if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64)
+        return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: pages of %d tokens (8, 16, 32 or 64 are taken)", page_size);
+    if ((dense ? kv.row_width % 8 : kv.page_stride % D) || q_stride % 8 || (((uintptr_t)q | (uintptr_t)kv.k | (uintptr_t)kv.v | (uintptr_t)out) & 15))
+        return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: tensors must be 16-byte aligned, pages whole rows");
+    if (n_tiles > 65535) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: %d tiles exceed the grid", n_tiles);
+    if (splits < 1 || splits > MERGE_MAX || (splits > 1 && (!part_o || !part_ml || (((uintptr_t)part_o) & 15))))
+        return fail(PH_ERR_ARG, "attention_prefill_tc5: %d splits need 16-byte aligned scratch for the partial results", splits);
+    if (gate && (gate_stride % 8 || ((uintptr_t)gate & 15))) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: the gate's rows must be 16-byte aligned");
+    if (n_tiles == 0) return PH_OK;
+    const long long rows_per_page = dense ? 0 : kv.page_stride / D;
+    const long long rows = dense ? kv.rows : (long long)(kv.num_pages - 1) * rows_per_page + (long long)HKV * page_size;
+    if (rows >= 0x7fffffffLL) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: the pool has too many rows");
+    CUtensorMap mq, mk, mv;
+    // Q: {64 elements, T tokens (q_stride elements apart), 2 halves (128 bytes apart), HQ heads (D * 2 bytes apart)}
+    const cuuint64_t qdims[4] = {64, (cuuint64_t)T, 2, (cuuint64_t)HQ};
+    const cuuint64_t qstrides[3] = {(cuuint64_t)q_stride * 2, 128, (cuuint64_t)D * 2};
+    const cuuint32_t qbox[4] = {64, BM, 2, 1};
+    // K, V: [rows, D] from the entry's first element (dense: [rows, HKV * D]); a box is one 64-element half of one page of one kv head
+    const cuuint64_t kdims[2] = {(cuuint64_t)(dense ? HKV * D : D), (cuuint64_t)rows};
+    const cuuint64_t kstrides[1] = {(cuuint64_t)(dense ? kv.row_width : D) * 2};
+    const cuuint32_t kbox[2] = {64, (cuuint32_t)page_size};
+    if (!encode(&mq, q, 4, qdims, qstrides, qbox) || !encode(&mk, kv.k, 2, kdims, kstrides, kbox) ||
+        !encode(&mv, kv.v, 2, kdims, kstrides, kbox))
+        return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: cuTensorMapEncodeTiled refused the layout");
+    Tc5Params p;
+    p.rows_per_page = rows_per_page; p.total_rows = (int)rows; p.page_size = page_size; p.page_shift = page_size == 8 ? 3 : page_size == 16 ? 4 : page_size == 32 ? 5 : 6;
+    p.block_table = kv.block_table; p.table_stride = kv.table_stride; p.seg_start = seg_start; p.seg_ctx_len = seg_ctx_len;
+    p.tile_seg = tile_seg; p.tile_first = tile_first; p.n_tiles = n_tiles; p.out = (__nv_bfloat16*)out;
+    p.HQ = HQ; p.HKV = HKV; p.window = window; p.chunk = chunk; p.scale_log2 = scale * LOG2E; p.error_flag = error_flag;
+    p.splits = splits; p.part_o = part_o; p.part_ml = part_ml; p.sink = sink;
+    p.slopes = slopes; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride; p.dense_base = kv.dense_base;
+    static bool configured = false;
+    if (!configured) {
+        if (cudaFuncSetAttribute(attention_prefill_tc5_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(attention_prefill_tc5_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess)
+            return fail(PH_ERR_LAUNCH, "attention_prefill_tc5: cannot reserve %d bytes of shared memory", SMEM_BYTES);
+        configured = true;
+    }
+    launch_overlapped(slopes ? attention_prefill_tc5_kernel<true> : attention_prefill_tc5_kernel<false>, dim3(HQ, n_tiles, splits), dim3(THREADS), (size_t)SMEM_BYTES, stream, mq, mk, mv, p);
+    if (splits > 1)
+        launch_overlapped(attention_prefill_tc5_combine_kernel, dim3(n_tiles, HQ, BM / 4), dim3(128), 0, stream,
+                          (const float*)part_o, (const float*)part_ml, seg_start, tile_seg, tile_first, (__nv_bfloat16*)out, HQ, splits, sink, p.gate, gate_stride);
+    return check_launch("attention_prefill_tc5");
+}
+}  // namespace
+
 // q [T, HQ, 128] bfloat16 -> out [T, HQ * 128].  splits > 1: that many CTAs share the keys of every tile and leave
 // partial results in part_o [T][HQ][splits][128] and part_ml [T][HQ][splits][2] (float32), which a second kernel merges;
 // for few tiles that look far back.  tile_seg / tile_first: the step's prompt portions cut into tiles
@@ -616,53 +690,26 @@ PH_EXPORT int ph_attention_prefill_tc5_biased(const void* q, int T, const void* 
                                               int window, int chunk, float scale, int splits, float* part_o, float* part_ml,
                                               int* error_flag, const float* sink, const float* slopes, const void* gate,
                                               long long gate_stride, cudaStream_t stream) {
-    if (!q || !k_base || !v_base || !block_table || !seg_start || !seg_ctx_len || !tile_seg || !tile_first || !out ||
-        !error_flag || T < 1 || n_tiles < 0 || HQ < 1 || HKV < 1 || HQ % HKV || num_pages < 1 || window < 0 || chunk < 0 || !(scale > 0.0f))
-        return fail(PH_ERR_ARG, "attention_prefill_tc5: bad arguments (tiles %d, HQ %d, HKV %d)", n_tiles, HQ, HKV);
-    if (head_dim != D) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: head_dim %d is not %d", head_dim, D);
-    if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64)
-        return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: pages of %d tokens (8, 16, 32 or 64 are taken)", page_size);
-    if (page_stride % D || (((uintptr_t)q | (uintptr_t)k_base | (uintptr_t)v_base | (uintptr_t)out) & 15))
-        return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: tensors must be 16-byte aligned, pages whole rows");
-    if (n_tiles > 65535) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: %d tiles exceed the grid", n_tiles);
-    if (splits < 1 || splits > MERGE_MAX || (splits > 1 && (!part_o || !part_ml || (((uintptr_t)part_o) & 15))))
-        return fail(PH_ERR_ARG, "attention_prefill_tc5: %d splits need 16-byte aligned scratch for the partial results", splits);
-    if (gate && (gate_stride % 8 || ((uintptr_t)gate & 15))) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: the gate's rows must be 16-byte aligned");
-    if (n_tiles == 0) return PH_OK;
-    const long long rows_per_page = page_stride / D;
-    const long long rows = (long long)(num_pages - 1) * rows_per_page + (long long)HKV * page_size;
-    if (rows >= 0x7fffffffLL) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: the pool has too many rows");
-    CUtensorMap mq, mk, mv;
-    // Q: {64 elements, T tokens (HQ * D * 2 bytes apart), 2 halves (128 bytes apart), HQ heads (D * 2 bytes apart)}
-    const cuuint64_t qdims[4] = {64, (cuuint64_t)T, 2, (cuuint64_t)HQ};
-    const cuuint64_t qstrides[3] = {(cuuint64_t)HQ * D * 2, 128, (cuuint64_t)D * 2};
-    const cuuint32_t qbox[4] = {64, BM, 2, 1};
-    // K, V: [rows, D] from the entry's first element; a box is one 64-element half of one page of one kv head
-    const cuuint64_t kdims[2] = {(cuuint64_t)D, (cuuint64_t)rows};
-    const cuuint64_t kstrides[1] = {(cuuint64_t)D * 2};
-    const cuuint32_t kbox[2] = {64, (cuuint32_t)page_size};
-    if (!encode(&mq, q, 4, qdims, qstrides, qbox) || !encode(&mk, k_base, 2, kdims, kstrides, kbox) ||
-        !encode(&mv, v_base, 2, kdims, kstrides, kbox))
-        return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: cuTensorMapEncodeTiled refused the layout");
-    Tc5Params p;
-    p.rows_per_page = rows_per_page; p.total_rows = (int)rows; p.page_size = page_size; p.page_shift = page_size == 8 ? 3 : page_size == 16 ? 4 : page_size == 32 ? 5 : 6;
-    p.block_table = block_table; p.table_stride = table_stride; p.seg_start = seg_start; p.seg_ctx_len = seg_ctx_len;
-    p.tile_seg = tile_seg; p.tile_first = tile_first; p.n_tiles = n_tiles; p.out = (__nv_bfloat16*)out;
-    p.HQ = HQ; p.HKV = HKV; p.window = window; p.chunk = chunk; p.scale_log2 = scale * LOG2E; p.error_flag = error_flag;
-    p.splits = splits; p.part_o = part_o; p.part_ml = part_ml; p.sink = sink;
-    p.slopes = slopes; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride;
-    static bool configured = false;
-    if (!configured) {
-        if (cudaFuncSetAttribute(attention_prefill_tc5_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess ||
-            cudaFuncSetAttribute(attention_prefill_tc5_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess)
-            return fail(PH_ERR_LAUNCH, "attention_prefill_tc5: cannot reserve %d bytes of shared memory", SMEM_BYTES);
-        configured = true;
-    }
-    launch_overlapped(slopes ? attention_prefill_tc5_kernel<true> : attention_prefill_tc5_kernel<false>, dim3(HQ, n_tiles, splits), dim3(THREADS), (size_t)SMEM_BYTES, stream, mq, mk, mv, p);
-    if (splits > 1)
-        launch_overlapped(attention_prefill_tc5_combine_kernel, dim3(n_tiles, HQ, BM / 4), dim3(128), 0, stream,
-                          (const float*)part_o, (const float*)part_ml, seg_start, tile_seg, tile_first, (__nv_bfloat16*)out, HQ, splits, sink, p.gate, gate_stride);
-    return check_launch("attention_prefill_tc5");
+    KvPlace kv = {};
+    kv.k = k_base; kv.v = v_base; kv.page_stride = page_stride; kv.page_size = page_size; kv.num_pages = num_pages;
+    kv.block_table = block_table; kv.table_stride = table_stride;
+    return launch_tc5(q, (long long)HQ * D, T, kv, seg_start, seg_ctx_len, tile_seg, tile_first, n_tiles, out, HQ, HKV, head_dim, window, chunk,
+                      scale, splits, part_o, part_ml, error_flag, sink, slopes, gate, gate_stride, stream);
+}
+
+// The same over keys and values that lie densely: k and v [rows, H * 128] bfloat16, row_width elements from a token's row to
+// the next one's, the rows of segment s from dense_base[s] on (one per position of the request); q's tokens q_stride elements
+// apart; every query head has a key head of its own.
+PH_EXPORT int ph_attention_prefill_tc5_dense(const void* q, long long q_stride, int T, const void* k, const void* v, long long row_width,
+                                             int rows, const int32_t* dense_base, const int32_t* seg_start, const int32_t* seg_ctx_len,
+                                             const int32_t* tile_seg, const int32_t* tile_first, int n_tiles, void* out, int H, int head_dim,
+                                             float scale, int splits, float* part_o, float* part_ml, int* error_flag, const void* gate,
+                                             long long gate_stride, cudaStream_t stream) {
+    KvPlace kv = {};
+    kv.k = k; kv.v = v; kv.dense_base = dense_base; kv.row_width = row_width; kv.rows = rows;
+    if (!dense_base) return fail(PH_ERR_ARG, "attention_prefill_tc5_dense: no first rows");
+    return launch_tc5(q, q_stride, T, kv, seg_start, seg_ctx_len, tile_seg, tile_first, n_tiles, out, H, H, head_dim, 0, 0, scale, splits, part_o,
+                      part_ml, error_flag, nullptr, nullptr, gate, gate_stride, stream);
 }
 
 PH_EXPORT int ph_attention_prefill_tc5_sink(const void* q, int T, const void* k_base, const void* v_base, long long page_stride,

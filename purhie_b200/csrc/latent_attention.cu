@@ -10,6 +10,8 @@
 //                    latent (for the up product), the RMS norm of the kv latent and the rotation of r into the token's
 //                    cache row.
 //   latent_absorb    q_lat[t, h] = [Wuk_h^T q_plain[t, h] | rotate(q_rot[t, h])]
+//   latent_gather    the cached latents of whole requests as dense rows, for a portion long enough that making the heads' keys
+//                    and values once costs less than attending over the latents
 //   latent_expand    out[t, h] = (Wuv_h o_lat[t, h]) * sigmoid(gate[t, h]), or with a gate per value, * sigmoid(gate[t, h, v])
 // The attention itself is attention_generic (values read out of the key rows) or the tensor-core kernels of
 // latent_attention_mma.cu.  Sums here are float32 with the contraction index ascending, whatever else is in the batch.
@@ -64,6 +66,26 @@ __global__ void latent_prepare_kernel(const TD* __restrict__ down, long long dow
         if (i < half) v = turn_u(v, to_float<TD>(r[i + half]), cs[i], cs[half + i]);
         else if (i < n_rot) v = turn_v(to_float<TD>(r[i - half]), v, cs[i - half], cs[i]);
         dst[C + i] = from_float<TKV>(v);
+    }
+}
+
+// dense[base[seg] + pos] = the cache row at pos, for the requests listed and pos < their length; a warp per row
+template <typename T>
+__global__ void latent_gather_kernel(const T* __restrict__ k_base, long long page_stride, int page_size, const int32_t* __restrict__ block_table,
+                                     int table_stride, const int32_t* __restrict__ segs, const int32_t* __restrict__ base,
+                                     const int32_t* __restrict__ seg_ctx_len, T* __restrict__ dense, int C, int row) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int seg = segs[blockIdx.y], len = seg_ctx_len[seg];
+    const int pos = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (pos >= len) return;
+    const T* src = k_base + (size_t)block_table[(size_t)seg * table_stride + pos / page_size] * page_stride + (size_t)(pos % page_size) * row;
+    T* dst = dense + (size_t)(base[seg] + pos) * C;
+    constexpr int V = 16 / sizeof(T);
+    if (C % V == 0 && row % V == 0 && (((uintptr_t)k_base | (uintptr_t)dense) & 15) == 0 && page_stride % V == 0) {
+        for (int i = lane; i < C / V; i += 32) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+    } else {
+        for (int i = lane; i < C; i += 32) dst[i] = src[i];
     }
 }
 
@@ -173,6 +195,22 @@ PH_EXPORT int ph_latent_prepare(const void* down, int down_dtype, long long down
     PH_DISPATCH(down_dtype, TD, PH_DISPATCH(cq_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, LAUNCH(TD, TQ, TKV))));
 #undef LAUNCH
     return check_launch("latent_prepare");
+}
+
+// The first C numbers of the cache rows (row numbers each) of the n_segs requests listed in segs, one per position below
+// seg_ctx_len, into dense [*, C] from base[segment] on; max_len: the longest of them.
+PH_EXPORT int ph_latent_gather(const void* k_base, int dtype, long long page_stride, int page_size, const int32_t* block_table,
+                               int table_stride, const int32_t* segs, int n_segs, const int32_t* base, const int32_t* seg_ctx_len,
+                               int max_len, void* dense, int C, int row, cudaStream_t stream) {
+    if (!k_base || !block_table || !segs || !base || !seg_ctx_len || !dense || n_segs < 0 || max_len < 0 || C < 1 || row < C || page_size < 1 ||
+        !valid_dtype(dtype))
+        return fail(PH_ERR_ARG, "latent_gather: bad arguments (requests %d, C %d of %d)", n_segs, C, row);
+    if (n_segs > 65535) return fail(PH_ERR_UNSUPPORTED, "latent_gather: %d requests exceed the grid", n_segs);
+    if (n_segs == 0 || max_len == 0) return PH_OK;
+    const dim3 grid((unsigned)((max_len + 7) / 8), (unsigned)n_segs);
+    PH_DISPATCH(dtype, T, launch_overlapped(latent_gather_kernel<T>, grid, dim3(256), 0, stream, (const T*)k_base, page_stride, page_size,
+                                            block_table, table_stride, segs, base, seg_ctx_len, (T*)dense, C, row));
+    return check_launch("latent_gather");
 }
 
 // q [T, H, D + R] with the tokens' rows q_stride elements apart, wuk [H * D, C] -> q_lat [T, H, C + R].

@@ -11,7 +11,9 @@
 //   ssd_scan    token by token: a group of lanes holds four rows (p) of S, N spread over the lanes; a token costs a
 //               multiply-add per state element and a butterfly per row.  Decoding, short portions, float32.
 //   ssd_chunk   chunks of 64 tokens on the tensor cores (bfloat16 in, float32 sums), a block per (request, head, 32 of its P
-//               columns) that walks the request's chunks in order with S in registers.  With cum_i the sum of a dt over the
+//               columns) that walks the request's chunks in order.  Four of its warps make the chunk's outputs while the four
+//               others fetch the next chunk, work out its step sizes and carry S, which they hold in registers, over the
+//               current one.  With cum_i the sum of a dt over the
 //               chunk's tokens up to i:
 //                   y_i = sum_(j <= i) (C_i . B_j) exp(cum_i - cum_j) dt_j x_j + exp(cum_i) C_i^T S + d x_i
 //                   S   = exp(cum_last) S + sum_j exp(cum_last - cum_j) dt_j B_j x_j^T
@@ -45,13 +47,13 @@ struct SsdParams {
 };
 
 // The last K - 1 inputs of the convolution, oldest first: from this step's rows, or moved up from what was kept.  The
-// channels are spread over the `blocks` blocks that work on a request.
+// channels are spread over the `blocks` groups of `threads` threads that work on a request.
 template <typename TX>
-__device__ __forceinline__ void move_conv_inputs(const SsdParams& p, float* st, int row0, int n, int block, int blocks) {
+__device__ __forceinline__ void move_conv_inputs(const SsdParams& p, float* st, int row0, int n, int block, int blocks, int thread, int threads) {
     const int CH = p.H * p.P + 2 * p.G * p.N;
     float* past = st + (size_t)p.H * p.P * p.N;
     const TX* src = static_cast<const TX*>(p.in) + p.conv_col;
-    for (int c = block * blockDim.x + threadIdx.x; c < CH; c += blocks * blockDim.x)
+    for (int c = block * threads + thread; c < CH; c += blocks * threads)
         for (int k = 0; k < p.K - 1; ++k) {
             const int i = n - (p.K - 1) + k;
             past[(size_t)k * CH + c] = i >= 0 ? to_float<TX>(src[(size_t)(row0 + i) * p.in_stride + c]) : past[(size_t)(k + n) * CH + c];
@@ -138,23 +140,24 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssd_scan_kernel(const SsdParams 
             if constexpr (V == 4) store4(S0 + (size_t)(p0 + r) * N + n, &S[r][i * V]);
             else S0[(size_t)(p0 + r) * N + n] = S[r][i];
         }
-    move_conv_inputs<TX>(p, st, row0, n_rows, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
+    move_conv_inputs<TX>(p, st, row0, n_rows, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y, threadIdx.x, SCAN_THREADS);
 }
 
 // ---- chunks on the tensor cores ------------------------------------------------------------------------------------
 constexpr int CQ = 64;                 // tokens of a chunk
 constexpr int CP = 32;                 // columns (p) of a block
-constexpr int CTHREADS = 128;          // four warps: warp w owns the rows 16 w .. 16 w + 15 of the chunk
+constexpr int CWARPS = 4;              // warps 0 .. 3: outputs, 16 rows of the chunk each; warps 4 .. 7: the next chunk and S
+constexpr int CTHREADS = 2 * CWARPS * 32;
 constexpr int XPITCH = CP * 2 + 16;    // bytes of a row of the x tile
 
 __host__ __device__ constexpr int ssd_pitch(int NP) { return NP * 2 + 16; }
-__host__ __device__ constexpr int ssd_smem(int NP) { return 4 * CQ * ssd_pitch(NP) + 2 * CQ * XPITCH + 2 * CP * ssd_pitch(NP) + 4 * 3 * CQ * 4; }
+// B, C and x of two chunks, S as two bfloat16 tiles, and (cum, dt, w) of two chunks
+__host__ __device__ constexpr int ssd_smem(int NP) { return 4 * CQ * ssd_pitch(NP) + 2 * CQ * XPITCH + 2 * CP * ssd_pitch(NP) + 2 * 3 * CQ * 4; }
 
 // v = hi + lo with both in bfloat16 (hi the rounded value, lo the rounded rest), two values at a time
 __device__ __forceinline__ void split2(float u, float v, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(u, v);
-    const float2 back = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&hi));
-    lo = pack_bf16(u - back.x, v - back.y);
+    lo = pack_bf16(u - __uint_as_float(hi << 16), v - __uint_as_float(hi & 0xffff0000u));
 }
 
 // NP: N rounded up to 16.  NTW: tiles of 16 states that a warp holds of S (tile w + 4 k).
@@ -164,49 +167,175 @@ __global__ void __launch_bounds__(CTHREADS, NTW <= 2 ? 2 : 1) ssd_chunk_kernel(c
     pdl_launch_dependents();
     const int seg = blockIdx.z, h = blockIdx.y, pt0 = blockIdx.x * CP;
     const int row0 = p.seg_start[seg], n_rows = p.seg_start[seg + 1] - row0;
-    const float bias = p.dt_bias[h], a = p.a[h], skip = p.d[h];
     if (n_rows < p.rows_from || n_rows > p.rows_to) { pdl_wait(); return; }
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = (threadIdx.x >> 5) & (CWARPS - 1), lane = threadIdx.x & 31;
+    const bool outputs = threadIdx.x < CWARPS * 32;
     const int P = p.P, N = p.N, inner = p.H * P, CH = inner + 2 * p.G * N;
     const int g = h / (p.H / p.G), pitch = ssd_pitch(NP), ntiles = NP / 16;
     const uint32_t b_tiles = smem_u32(smem), c_tiles = b_tiles + 2 * CQ * pitch, x_tiles = c_tiles + 2 * CQ * pitch;
     const uint32_t s_hi = x_tiles + 2 * CQ * XPITCH, s_lo = s_hi + CP * pitch;
-    uint8_t* s_hi_ptr = smem + (s_hi - b_tiles);
-    uint8_t* s_lo_ptr = smem + (s_lo - b_tiles);
-    float* cum = reinterpret_cast<float*>(smem + (s_lo - b_tiles) + CP * pitch) + warp * 3 * CQ;      // this warp's copy: cum, dt, w
-    float* dts = cum + CQ;
-    float* wts = dts + CQ;
-    float* st = p.state + (size_t)p.seg_slot[seg] * p.state_stride;
-    float* S0 = st + (size_t)h * P * N;
-    const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(p.xbc) + (size_t)row0 * CH;
-    const __nv_bfloat16* dt_in = static_cast<const __nv_bfloat16*>(p.in) + (size_t)row0 * p.in_stride + p.dt_col + h;
+    float* sums = reinterpret_cast<float*>(smem + (s_lo - b_tiles) + CP * pitch);      // [2][cum | dt | w][CQ]
+    const int chunks = (n_rows + CQ - 1) / CQ;
+    const int nc = (lane & 3) * 2;
     pdl_wait();
 
-    auto load_chunk = [&](int c, int buf) {
-        const int first = c * CQ, bc = NP / 8;                          // 16-byte pieces of a row of B or C
-        for (int i = threadIdx.x; i < CQ * 2 * bc; i += CTHREADS) {
-            const int r = i / (2 * bc), q = i % (2 * bc), piece = q % bc;
-            const bool is_c = q >= bc, valid = first + r < n_rows && piece * 8 < N;
-            const __nv_bfloat16* src = xbc + (valid ? (size_t)(first + r) * CH + inner + (size_t)((is_c ? p.G : 0) + g) * N + piece * 8 : 0);
-            cp_async16((is_c ? c_tiles : b_tiles) + (buf * CQ + r) * pitch + piece * 16, src, valid);
+    if (outputs) {
+        // ---- y of the rows 16 warp .. 16 warp + 15 of every chunk
+        const float skip = p.d[h];
+        const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;
+        float* y_out = p.y + (size_t)row0 * inner + (size_t)h * P;
+        for (int c = 0; c < chunks; ++c) {
+            const int buf = c & 1;
+            const uint32_t bt = b_tiles + buf * CQ * pitch, ct = c_tiles + buf * CQ * pitch, xt = x_tiles + buf * CQ * XPITCH;
+            const float* cum = sums + buf * 3 * CQ;
+            const float* dts = cum + CQ;
+            asm volatile("bar.sync 2, %0;" ::"n"(CTHREADS) : "memory");                             // the chunk, its sums and the S it starts from are there
+            // C_i . B_j for this warp's rows and the keys up to their last, and C_i^T S
+            float s[CQ / 8][4], y[CP / 8][4], rest[CP / 8][4];
+#pragma unroll
+            for (int nt = 0; nt < CQ / 8; ++nt)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) s[nt][i] = 0.0f;
+#pragma unroll
+            for (int nt = 0; nt < CP / 8; ++nt)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) y[nt][i] = rest[nt][i] = 0.0f;
+            for (int ks = 0; ks < ntiles; ++ks) {
+                uint32_t a0, a1, a2, a3;
+                ldmatrix_x4(ct + (warp * 16 + (lane & 15)) * pitch + (ks * 2 + (lane >> 4)) * 16, a0, a1, a2, a3);
+                const int col = (ks * 2 + ((lane >> 3) & 1)) * 16, row = (lane & 7) + ((lane >> 4) << 3);
+#pragma unroll
+                for (int nt = 0; nt < CP / 8; nt += 2) {
+                    uint32_t b0, b1, b2, b3;
+                    const int at = (nt * 8 + row) * pitch + col;
+                    ldmatrix_x4(s_hi + at, b0, b1, b2, b3);
+                    mma_bf16(y[nt], a0, a1, a2, a3, b0, b1);
+                    mma_bf16(y[nt + 1], a0, a1, a2, a3, b2, b3);
+                    ldmatrix_x4(s_lo + at, b0, b1, b2, b3);
+                    mma_bf16(rest[nt], a0, a1, a2, a3, b0, b1);
+                    mma_bf16(rest[nt + 1], a0, a1, a2, a3, b2, b3);
+                }
+#pragma unroll
+                for (int nt = 0; nt < CQ / 8; nt += 2) {
+                    if (nt > 2 * warp) continue;         // keys behind every row of this warp
+                    uint32_t b0, b1, b2, b3;
+                    ldmatrix_x4(bt + (nt * 8 + row) * pitch + col, b0, b1, b2, b3);
+                    mma_bf16(s[nt], a0, a1, a2, a3, b0, b1);
+                    mma_bf16(s[nt + 1], a0, a1, a2, a3, b2, b3);
+                }
+            }
+            asm volatile("bar.arrive 1, %0;" ::"n"(CTHREADS) : "memory");      // S is read: it may be written for the next chunk
+            const float cum0 = cum[r0], cum1 = cum[r1];
+            const float e0 = __expf(cum0), e1 = __expf(cum1);
+#pragma unroll
+            for (int nt = 0; nt < CP / 8; ++nt) {
+                y[nt][0] = (y[nt][0] + rest[nt][0]) * e0; y[nt][1] = (y[nt][1] + rest[nt][1]) * e0;
+                y[nt][2] = (y[nt][2] + rest[nt][2]) * e1; y[nt][3] = (y[nt][3] + rest[nt][3]) * e1;
+            }
+            // the weights of the chunk's own tokens (the skip sits on the diagonal), times x
+#pragma unroll
+            for (int kt = 0; kt < CQ / 16; ++kt) {
+                if (kt > warp) continue;
+                uint32_t hi[4], lo[4];
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int nt = 2 * kt + half, j = nt * 8 + nc;
+                    const float2 cj = *reinterpret_cast<const float2*>(cum + j), dj = *reinterpret_cast<const float2*>(dts + j);
+                    float w[4] = {s[nt][0] * (__expf(cum0 - cj.x) * dj.x), s[nt][1] * (__expf(cum0 - cj.y) * dj.y),
+                                  s[nt][2] * (__expf(cum1 - cj.x) * dj.x), s[nt][3] * (__expf(cum1 - cj.y) * dj.y)};
+                    if (kt == warp) {                    // the tile on the diagonal
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const int row = i < 2 ? r0 : r1, key = j + (i & 1);
+                            w[i] = key > row ? 0.0f : key == row ? w[i] + skip : w[i];
+                        }
+                    }
+                    split2(w[0], w[1], hi[2 * half], lo[2 * half]);
+                    split2(w[2], w[3], hi[2 * half + 1], lo[2 * half + 1]);
+                }
+                const int row = kt * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
+#pragma unroll
+                for (int nt = 0; nt < CP / 8; nt += 2) {
+                    uint32_t b0, b1, b2, b3;
+                    ldmatrix_x4_trans(xt + row * XPITCH + (nt + (lane >> 4)) * 16, b0, b1, b2, b3);
+                    mma_bf16(y[nt], hi[0], hi[1], hi[2], hi[3], b0, b1);
+                    mma_bf16(y[nt + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
+                    mma_bf16(y[nt], lo[0], lo[1], lo[2], lo[3], b0, b1);
+                    mma_bf16(y[nt + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
+                }
+            }
+#pragma unroll
+            for (int nt = 0; nt < CP / 8; ++nt) {
+                const int col = pt0 + nt * 8 + nc;
+                if (col >= P) continue;                  // P is even: a pair is inside or outside
+                const int t0 = c * CQ + r0, t1 = c * CQ + r1;
+                if (t0 < n_rows) *reinterpret_cast<float2*>(y_out + (size_t)t0 * inner + col) = make_float2(y[nt][0], y[nt][1]);
+                if (t1 < n_rows) *reinterpret_cast<float2*>(y_out + (size_t)t1 * inner + col) = make_float2(y[nt][2], y[nt][3]);
+            }
         }
-        for (int i = threadIdx.x; i < CQ * (CP / 8); i += CTHREADS) {
-            const int r = i / (CP / 8), piece = i % (CP / 8), col = pt0 + piece * 8;
-            const bool valid = first + r < n_rows && col < P;
-            cp_async16(x_tiles + (buf * CQ + r) * XPITCH + piece * 16, xbc + (valid ? (size_t)(first + r) * CH + (size_t)h * P + col : 0), valid);
+        return;
+    }
+
+    // ---- the chunks' rows, their step sizes, and S
+    const float bias = p.dt_bias[h], a = p.a[h];
+    float* st = p.state + (size_t)p.seg_slot[seg] * p.state_stride;
+    float* S0 = st + (size_t)h * P * N;
+    uint8_t* s_hi_ptr = smem + (s_hi - b_tiles);
+    uint8_t* s_lo_ptr = smem + (s_lo - b_tiles);
+    const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(p.xbc) + (size_t)row0 * CH;
+    const __nv_bfloat16* dt_in = static_cast<const __nv_bfloat16*>(p.in) + (size_t)row0 * p.in_stride + p.dt_col + h;
+    const int pieces = NP / 8;                               // 16-byte pieces of a row of B or C
+    auto load_chunk = [&](int c) {
+        const int buf = c & 1, first = c * CQ;
+        for (int r = warp; r < CQ; r += CWARPS) {            // a row of B and of C by a warp
+            const bool there = first + r < n_rows;
+            const __nv_bfloat16* src = xbc + (there ? (size_t)(first + r) * CH : 0) + inner + (size_t)g * N;
+            for (int q = lane; q < 2 * pieces; q += 32) {
+                const bool is_c = q >= pieces;
+                const int piece = is_c ? q - pieces : q;
+                cp_async16((is_c ? c_tiles : b_tiles) + (buf * CQ + r) * pitch + piece * 16,
+                           src + (is_c ? (size_t)p.G * N : 0) + (piece * 8 < N ? piece * 8 : 0), there && piece * 8 < N);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < CQ * (CP / 8) / (CWARPS * 32); ++i) {
+            const int at = i * CWARPS * 32 + warp * 32 + lane, r = at / (CP / 8), piece = at % (CP / 8), col = pt0 + piece * 8;
+            const bool there = first + r < n_rows && col < P;
+            cp_async16(x_tiles + (buf * CQ + r) * XPITCH + piece * 16, xbc + (there ? (size_t)(first + r) * CH + (size_t)h * P + col : 0), there);
         }
         cp_async_commit();
     };
-    // the step logits of this lane's two tokens of a chunk
+    // step sizes, the running sums of a dt, and what each token's outer product is worth at the chunk's end (by one warp; a
+    // lane has two neighbouring tokens)
+    auto make_sums = [&](int c, float u, float v) {
+        const int t = c * CQ + 2 * lane;
+        const float d0 = t < n_rows ? softplus(u + bias) : 0.0f, d1 = t + 1 < n_rows ? softplus(v + bias) : 0.0f;
+        const float l0 = a * d0, l1 = a * d1;
+        float run = l0 + l1;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float up = __shfl_up_sync(0xffffffffu, run, o);
+            if (lane >= o) run += up;
+        }
+        const float last = __shfl_sync(0xffffffffu, run, 31), before = __shfl_up_sync(0xffffffffu, run, 1);
+        const float c0 = (lane ? before : 0.0f) + l0;
+        float* to = sums + (c & 1) * 3 * CQ + 2 * lane;
+        *reinterpret_cast<float2*>(to) = make_float2(c0, run);
+        *reinterpret_cast<float2*>(to + CQ) = make_float2(d0, d1);
+        *reinterpret_cast<float2*>(to + 2 * CQ) = make_float2(__expf(last - c0) * d0, __expf(last - run) * d1);
+    };
     auto load_dt = [&](int c, float& u, float& v) {
         const int t = c * CQ + 2 * lane;
         u = t < n_rows ? __bfloat162float(dt_in[(size_t)t * p.in_stride]) : 0.0f;
         v = t + 1 < n_rows ? __bfloat162float(dt_in[(size_t)(t + 1) * p.in_stride]) : 0.0f;
     };
 
+    load_chunk(0);
+    float u, v;
+    if (warp == 0) load_dt(0, u, v);
     // S: rows p = mt * 16 + lane / 4 (+ 8), columns n = 16 tile + nt * 8 + 2 (lane % 4) (+ 1)
     float S[NTW][2][2][4];
-    const int pr = lane >> 2, nc = (lane & 3) * 2;
+    const int pr = lane >> 2;
 #pragma unroll
     for (int k = 0; k < NTW; ++k)
 #pragma unroll
@@ -214,9 +343,11 @@ __global__ void __launch_bounds__(CTHREADS, NTW <= 2 ? 2 : 1) ssd_chunk_kernel(c
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const int pp = pt0 + mt * 16 + pr + (i >> 1) * 8, n = (warp + 4 * k) * 16 + nt * 8 + nc + (i & 1);
-                    S[k][mt][nt][i] = pp < P && n < N ? S0[(size_t)pp * N + n] : 0.0f;
+                for (int half = 0; half < 2; ++half) {
+                    const int pp = pt0 + mt * 16 + pr + half * 8, n = (warp + 4 * k) * 16 + nt * 8 + nc;      // N is even
+                    const float2 v2 = pp < P && n < N ? *reinterpret_cast<const float2*>(S0 + (size_t)pp * N + n) : make_float2(0.0f, 0.0f);
+                    S[k][mt][nt][2 * half] = v2.x;
+                    S[k][mt][nt][2 * half + 1] = v2.y;
                 }
     auto put_state = [&]() {
 #pragma unroll
@@ -237,123 +368,18 @@ __global__ void __launch_bounds__(CTHREADS, NTW <= 2 ? 2 : 1) ssd_chunk_kernel(c
         }
     };
     put_state();
-    const int chunks = (n_rows + CQ - 1) / CQ;
-    float u_next, v_next;
-    load_chunk(0, 0);
-    load_dt(0, u_next, v_next);
-    const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;
+    if (warp == 0) make_sums(0, u, v);
+    cp_async_wait<0>();
     for (int c = 0; c < chunks; ++c) {
         const int buf = c & 1;
-        const uint32_t bt = b_tiles + buf * CQ * pitch, ct = c_tiles + buf * CQ * pitch, xt = x_tiles + buf * CQ * XPITCH;
-        const float u = u_next, v = v_next;
-        cp_async_wait<0>();
-        __syncthreads();                             // the chunk and S are there; everyone is done with the other buffer
-        if (c + 1 < chunks) {
-            load_chunk(c + 1, buf ^ 1);
-            load_dt(c + 1, u_next, v_next);
-        }
-        // step sizes, the running sums of a dt, and what each token's outer product is worth at the chunk's end
-        {
-            const int t = c * CQ + 2 * lane;
-            const float d0 = t < n_rows ? softplus(u + bias) : 0.0f, d1 = t + 1 < n_rows ? softplus(v + bias) : 0.0f;
-            const float l0 = a * d0, l1 = a * d1;
-            float run = l0 + l1;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float up = __shfl_up_sync(0xffffffffu, run, o);
-                if (lane >= o) run += up;
-            }
-            const float last = __shfl_sync(0xffffffffu, run, 31);
-            const float before = __shfl_up_sync(0xffffffffu, run, 1);
-            const float c0 = (lane ? before : 0.0f) + l0;
-            *reinterpret_cast<float2*>(cum + 2 * lane) = make_float2(c0, run);
-            *reinterpret_cast<float2*>(dts + 2 * lane) = make_float2(d0, d1);
-            *reinterpret_cast<float2*>(wts + 2 * lane) = make_float2(__expf(last - c0) * d0, __expf(last - run) * d1);
-            __syncwarp();
-        }
-        const float cum0 = cum[r0], cum1 = cum[r1];
-        // C_i . B_j for this warp's 16 rows and the keys up to their last, and C_i^T S
-        float s[CQ / 8][4], from_state[CP / 8][4];
-#pragma unroll
-        for (int nt = 0; nt < CQ / 8; ++nt)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) s[nt][i] = 0.0f;
-#pragma unroll
-        for (int nt = 0; nt < CP / 8; ++nt)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) from_state[nt][i] = 0.0f;
-        for (int ks = 0; ks < ntiles; ++ks) {
-            uint32_t a0, a1, a2, a3;
-            ldmatrix_x4(ct + (warp * 16 + (lane & 15)) * pitch + (ks * 2 + (lane >> 4)) * 16, a0, a1, a2, a3);
-#pragma unroll
-            for (int nt = 0; nt < CQ / 8; nt += 2) {
-                if (nt > 2 * warp) continue;         // keys behind every row of this warp
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4(bt + (nt * 8 + (lane & 7) + ((lane >> 4) << 3)) * pitch + (ks * 2 + ((lane >> 3) & 1)) * 16, b0, b1, b2, b3);
-                mma_bf16(s[nt], a0, a1, a2, a3, b0, b1);
-                mma_bf16(s[nt + 1], a0, a1, a2, a3, b2, b3);
-            }
-#pragma unroll
-            for (int nt = 0; nt < CP / 8; nt += 2) {
-                uint32_t b0, b1, b2, b3;
-                const int at = (nt * 8 + (lane & 7) + ((lane >> 4) << 3)) * pitch + (ks * 2 + ((lane >> 3) & 1)) * 16;
-                ldmatrix_x4(s_hi + at, b0, b1, b2, b3);
-                mma_bf16(from_state[nt], a0, a1, a2, a3, b0, b1);
-                mma_bf16(from_state[nt + 1], a0, a1, a2, a3, b2, b3);
-                ldmatrix_x4(s_lo + at, b0, b1, b2, b3);
-                mma_bf16(from_state[nt], a0, a1, a2, a3, b0, b1);
-                mma_bf16(from_state[nt + 1], a0, a1, a2, a3, b2, b3);
-            }
-        }
-        // the weights of the chunk's own tokens, and what the state gives; the skip sits on the diagonal
-        float y[CP / 8][4];
-        const float e0 = __expf(cum0), e1 = __expf(cum1);
-#pragma unroll
-        for (int nt = 0; nt < CP / 8; ++nt) {
-            y[nt][0] = from_state[nt][0] * e0; y[nt][1] = from_state[nt][1] * e0;
-            y[nt][2] = from_state[nt][2] * e1; y[nt][3] = from_state[nt][3] * e1;
-        }
-#pragma unroll
-        for (int nt = 0; nt < CQ / 8; ++nt) {
-            if (nt > 2 * warp + 1) continue;
-            const int j = nt * 8 + nc;
-            const float2 cj = *reinterpret_cast<const float2*>(cum + j), dj = *reinterpret_cast<const float2*>(dts + j);
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int row = i < 2 ? r0 : r1, key = j + (i & 1);
-                const float w = (i & 1) ? __expf((i < 2 ? cum0 : cum1) - cj.y) * dj.y : __expf((i < 2 ? cum0 : cum1) - cj.x) * dj.x;
-                s[nt][i] = key > row ? 0.0f : s[nt][i] * w + (key == row ? skip : 0.0f);
-            }
-        }
-#pragma unroll
-        for (int kt = 0; kt < CQ / 16; ++kt) {
-            if (kt > warp) continue;
-            uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
-            split2(s[2 * kt][0], s[2 * kt][1], h0, l0);
-            split2(s[2 * kt][2], s[2 * kt][3], h1, l1);
-            split2(s[2 * kt + 1][0], s[2 * kt + 1][1], h2, l2);
-            split2(s[2 * kt + 1][2], s[2 * kt + 1][3], h3, l3);
-            const int row = kt * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
-#pragma unroll
-            for (int nt = 0; nt < CP / 8; nt += 2) {
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4_trans(xt + row * XPITCH + (nt + (lane >> 4)) * 16, b0, b1, b2, b3);
-                mma_bf16(y[nt], h0, h1, h2, h3, b0, b1);
-                mma_bf16(y[nt + 1], h0, h1, h2, h3, b2, b3);
-                mma_bf16(y[nt], l0, l1, l2, l3, b0, b1);
-                mma_bf16(y[nt + 1], l0, l1, l2, l3, b2, b3);
-            }
-        }
-#pragma unroll
-        for (int nt = 0; nt < CP / 8; ++nt) {
-            const int col = pt0 + nt * 8 + nc;
-            if (col >= P) continue;                  // P is even: a pair is inside or outside
-#pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int t = c * CQ + (half ? r1 : r0);
-                if (t < n_rows)
-                    *reinterpret_cast<float2*>(p.y + (size_t)(row0 + t) * inner + (size_t)h * P + col) = make_float2(y[nt][2 * half], y[nt][2 * half + 1]);
-            }
+        const uint32_t bt = b_tiles + buf * CQ * pitch, xt = x_tiles + buf * CQ * XPITCH;
+        const float* cum = sums + buf * 3 * CQ;
+        const float* wts = cum + 2 * CQ;
+        asm volatile("bar.sync 2, %0;" ::"n"(CTHREADS) : "memory");                                 // everyone is done with the other buffer
+        const bool more = c + 1 < chunks;
+        if (more) {
+            load_chunk(c + 1);
+            if (warp == 0) load_dt(c + 1, u, v);
         }
         // S <- exp(cum_last) S + sum_j w_j x_j B_j^T: rows p, contraction over the tokens
         const float keep = __expf(cum[CQ - 1]);
@@ -377,9 +403,8 @@ __global__ void __launch_bounds__(CTHREADS, NTW <= 2 ? 2 : 1) ssd_chunk_kernel(c
                 ldmatrix_x4_trans(xt + (kt * 16 + (lane & 7) + ((lane >> 4) << 3)) * XPITCH + (mt * 2 + ((lane >> 3) & 1)) * 16, x[0], x[1], x[2], x[3]);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const float2 f = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&x[i]));
                     const float2 w = i < 2 ? w0 : w1;
-                    split2(f.x * w.x, f.y * w.y, hi[mt][i], lo[mt][i]);
+                    split2(__uint_as_float(x[i] << 16) * w.x, __uint_as_float(x[i] & 0xffff0000u) * w.y, hi[mt][i], lo[mt][i]);
                 }
             }
 #pragma unroll
@@ -397,9 +422,11 @@ __global__ void __launch_bounds__(CTHREADS, NTW <= 2 ? 2 : 1) ssd_chunk_kernel(c
                 }
             }
         }
-        if (c + 1 < chunks) {
-            __syncthreads();                         // everyone has read the S that this chunk started from
+        if (more && warp == 0) make_sums(c + 1, u, v);
+        asm volatile("bar.sync 1, %0;" ::"n"(CTHREADS) : "memory");      // the outputs' warps have read the S of this chunk
+        if (more) {
             put_state();
+            cp_async_wait<0>();
         }
     }
 #pragma unroll
@@ -410,10 +437,10 @@ __global__ void __launch_bounds__(CTHREADS, NTW <= 2 ? 2 : 1) ssd_chunk_kernel(c
             for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {
-                    const int pp = pt0 + mt * 16 + pr + half * 8, n = (warp + 4 * k) * 16 + nt * 8 + nc;      // N is even
+                    const int pp = pt0 + mt * 16 + pr + half * 8, n = (warp + 4 * k) * 16 + nt * 8 + nc;
                     if (pp < P && n < N) *reinterpret_cast<float2*>(S0 + (size_t)pp * N + n) = make_float2(S[k][mt][nt][2 * half], S[k][mt][nt][2 * half + 1]);
                 }
-    move_conv_inputs<__nv_bfloat16>(p, st, row0, n_rows, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
+    move_conv_inputs<__nv_bfloat16>(p, st, row0, n_rows, (blockIdx.y * gridDim.x + blockIdx.x) * CWARPS + warp, gridDim.x * gridDim.y * CWARPS, lane, 32);
 }
 
 // One block per (token, part).

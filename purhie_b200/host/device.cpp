@@ -178,6 +178,7 @@ const CoreKernels& core_kernels() {
     bind(h, "core", "ph_latent_prepare", g_core.latent_prepare);
     bind(h, "core", "ph_latent_absorb", g_core.latent_absorb);
     bind(h, "core", "ph_latent_expand", g_core.latent_expand);
+    bind(h, "core", "ph_latent_gather", g_core.latent_gather);
     bind(h, "core", "ph_attention_generic_biased", g_core.attention_generic_biased);
     bind(h, "core", "ph_qk_norm_rope_gate_kv_write", g_core.qk_norm_rope_gate_kv_write);
     bind(h, "core", "ph_lanes_rmsnorm", g_core.lanes_rmsnorm);
@@ -210,6 +211,7 @@ const FlashKernels& flash_kernels() {
     bind(h, "flash", "ph_attention_prefill_tc5", g_flash.prefill_tc5);
     bind(h, "flash", "ph_attention_decode_bulk_biased", g_flash.decode_bulk_biased);
     bind(h, "flash", "ph_attention_prefill_tc5_biased", g_flash.prefill_tc5_biased);
+    bind(h, "flash", "ph_attention_prefill_tc5_dense", g_flash.prefill_tc5_dense);
     bind(h, "flash", "ph_flash_last_error", g_flash.last_error);
     g_flash_ok = true;
     return g_flash;

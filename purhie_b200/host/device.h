@@ -159,6 +159,8 @@ struct CoreKernels {
     int (*latent_absorb)(const void*, int, long long, const void*, int, const float*, int, int, const int32_t*, void*, int, int, int, int, int,
                          int, cudaStream_t);
     int (*latent_expand)(const void*, int, const void*, int, const void*, int, long long, int, void*, int, int, int, int, int, cudaStream_t);
+    int (*latent_gather)(const void*, int, long long, int, const int32_t*, int, const int32_t*, int, const int32_t*, const int32_t*, int, void*,
+                         int, int, cudaStream_t);
     // attention with a sink in the softmax's denominator (the plain kernel); attention whose heads' scores are capped,
     // biased by the distance and mixed before the softmax, with the kernel that norms q and k over their whole width and
     // writes the cache rows in front of it
@@ -216,6 +218,10 @@ struct FlashKernels {
     int (*prefill_tc5_biased)(const void*, int, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*,
                               const int32_t*, const int32_t*, const int32_t*, int, void*, int, int, int, int, int, float, int, float*,
                               float*, int*, const float*, const float*, const void*, long long, cudaStream_t);
+    // the prompt kernel over dense keys and values, a row per token with the heads side by side
+    int (*prefill_tc5_dense)(const void*, long long, int, const void*, const void*, long long, int, const int32_t*, const int32_t*,
+                             const int32_t*, const int32_t*, const int32_t*, int, void*, int, int, float, int, float*, float*, int*, const void*,
+                             long long, cudaStream_t);
     const char* (*last_error)(void);
 };
 // attention over cached latent rows on the tensor cores (latent_attention_mma.cu)

@@ -18,6 +18,11 @@
 // In bfloat16 the attention runs on the tensor cores (latent_attention_mma.cu): the (token, head) pairs of a portion,
 // heads side by side, are cut into tiles of 64 that prepare_step() lists, and when there are few tiles the keys of
 // each are split over several CTAs.  Rows that kernel does not take, and float32, go through attention_generic.
+//
+// A long portion of a request (kDenseRows rows or more) in bfloat16, without a rotated part or a window and with heads of
+// 128 / 128, goes the other way: the request's latents are gathered from the cache, one product makes every head's keys and
+// values from them, and the tcgen05 prompt kernel attends over those rows, q as the stacked product left it and the gate in
+// its epilogue.  That is a quarter of the flops of attending over latents of 512, and the making is paid once per portion.
 #include <algorithm>
 #include <cmath>
 
@@ -113,8 +118,21 @@ public:
             q_norm_ = src.fetch(name_of("q_norm"));
         }
         kv_norm_ = src.fetch(name_of("kv_norm"));
-        k_up_ = src.fetch(name_of("k_up"));
-        v_up_ = src.fetch(name_of("v_up"));
+        // [k_up | v_up] in one matrix: one product makes the heads' keys and values where they are made at all
+        Tensor up[2] = {src.fetch(name_of("k_up")), src.fetch(name_of("v_up"))};
+        if (up[0].dtype == up[1].dtype) {
+            Tensor both = src.arena().alloc(up[0].dtype, {(int64_t)heads_ * (dim_ + vdim_), kv_rank_});
+            QE_CUDA(cudaMemcpyAsync(both.data, up[0].data, up[0].bytes(), cudaMemcpyDeviceToDevice, src.stream()));
+            QE_CUDA(cudaMemcpyAsync(static_cast<char*>(both.data) + up[0].bytes(), up[1].data, up[1].bytes(), cudaMemcpyDeviceToDevice, src.stream()));
+            QE_CUDA(cudaStreamSynchronize(src.stream()));
+            for (Tensor& t : up) src.release(t);
+            kv_up_ = Linear(both, "kv_up", gemm_);
+            k_up_ = both.rows(0, (int64_t)heads_ * dim_);
+            v_up_ = both.rows((int64_t)heads_ * dim_, (int64_t)heads_ * vdim_);
+        } else {
+            k_up_ = up[0];
+            v_up_ = up[1];
+        }
         o_proj_ = Linear(src.fetch(name_of("o_proj")), "o_proj", gemm_);
         if (position_) {
             position_->bind(src);
@@ -126,6 +144,7 @@ public:
         std::vector<std::string> libs = {"core"};
         if (down_proj_.fast() || q_up_.fast() || o_proj_.fast()) libs.push_back("gemm100");
         if (products_on_tensor_cores()) libs.push_back("latent");
+        if (may_go_dense()) libs.push_back("flash");
         return libs;
     }
 
@@ -140,15 +159,53 @@ public:
         return compute_dtype == DType::BF16 && attention_ != "generic" && kv_rank_ % 8 == 0 && rot_ % 8 == 0 && kv_rank_ <= 512 && rot_ <= 64;
     }
 
+    // a portion long enough may attend over keys and values made for it (see above)
+    bool may_go_dense() const {
+        return compute_dtype == DType::BF16 && (attention_ == "auto" || attention_ == "flash") && rot_ == 0 && window_ == 0 && dim_ == 128 && vdim_ == 128 &&
+               kv_up_.fast() && down_proj_.fast() && direct_q_;
+    }
+    // the segments of a step that do: long portions, as long as their rows fit the scratch
+    void add_dense(StepPlan& plan) const {
+        if (plan.has("latent.dense.base")) return;
+        struct Tile { int seg, first, reach; };
+        std::vector<Tile> tiles;
+        std::vector<int32_t> segs, base((size_t)plan.S, -1);
+        int rows = 0;
+        for (int s = 0; s < plan.S; s++) {
+            const int n = plan.q_lens[s], len = plan.ctx_lens[s];
+            if (n < kDenseRows || rows + len > kDenseMax) continue;
+            segs.push_back(s);
+            base[s] = rows;
+            rows += len;
+            for (int first = 0; first < n; first += kDenseTile) tiles.push_back({s, first, len - n + std::min(first + kDenseTile, n)});
+        }
+        std::stable_sort(tiles.begin(), tiles.end(), [](const Tile& a, const Tile& b) { return a.reach > b.reach; });
+        std::vector<int32_t> tile_seg, tile_first;
+        for (const Tile& t : tiles) { tile_seg.push_back(t.seg); tile_first.push_back(t.first); }
+        if (!segs.empty()) {
+            plan.add("latent.dense.segs", std::move(segs));
+            plan.add("latent.dense.tile_seg", std::move(tile_seg));
+            plan.add("latent.dense.tile_first", std::move(tile_first));
+        }
+        plan.add("latent.dense.base", std::move(base));
+    }
+
     // tiles of kTileRows (token, head) pairs per segment: the segment and the first pair of each, the tiles that look
     // furthest back first
     void prepare_step(StepPlan& plan) override {
+        const bool dense = may_go_dense();
+        if (dense) add_dense(plan);
         if (!on_tensor_cores()) return;
+        const std::vector<int32_t>* base = nullptr;
+        if (dense)
+            for (const auto& a : plan.arrays)
+                if (a.first == "latent.dense.base") base = &a.second;
         const std::string name = tiles_name();
         if (plan.has(name + ".seg")) return;
         struct Tile { int seg, first, reach; };
         std::vector<Tile> tiles;
         for (int s = 0; s < plan.S; s++) {
+            if (base && (*base)[s] >= 0) continue;                   // attends over keys and values of its own
             const int n = plan.q_lens[s] * heads_, start = plan.ctx_lens[s] - plan.q_lens[s];
             for (int first = 0; first < n; first += kTileRows) {
                 const int last_token = (std::min(first + kTileRows, n) - 1) / heads_;
@@ -192,59 +249,66 @@ public:
         // [T, heads, plain | rotated]: the up product's rows, or the first columns of the stacked product's
         Tensor q = direct_q_ ? down : q_up_(cq, ctx, "la_q", dt, T).tensor;
         const long long q_stride = direct_q_ ? down_width_ : (long long)heads_ * (dim_ + rot_);
-        Tensor q_lat = ws.get("la_q_lat", {T, heads_, row}, dt);
-        if (LaunchProfile::get().on())
-            LaunchProfile::get().note_cost((double)T * heads_ * (dim_ + rot_ + row) * es + (double)k_up_.bytes(), 2.0 * T * heads_ * dim_ * kv_rank_);
-        const bool tc_products = products_on_tensor_cores() && dt == DType::BF16;
-        if (tc_products) {
-            const LatentKernels& lk = latent_kernels();
-            QE_LAUNCH(lk, lk.latent_absorb(q.data, q_stride, k_up_.data, table, n_rot, max_pos, positions, q_lat.data, T, heads_, dim_, rot_, kv_rank_, ctx.stream));
-        } else
-        QE_LAUNCH(k, k.latent_absorb(q.data, q.code(), q_stride, k_up_.data, k_up_.code(), table, n_rot, max_pos, positions, q_lat.data, q_lat.code(), T,
-                                     heads_, dim_, rot_, kv_rank_, ctx.stream));
-        // every head reads the one cached row per position: keys the whole row, values its first kv_rank numbers
-        Tensor o_lat = ws.get("la_o_lat", {T, heads_, kv_rank_}, DType::F32);
-        const int32_t* abs_positions = ctx.position_column(0);
-        if (LaunchProfile::get().on()) {
-            double seen = 0.0, read = 0.0;
-            for (size_t i = 0; i < ctx.q_lens.size(); i++) {
-                const double n = ctx.q_lens[i], len = ctx.ctx_lens[i];
-                read += window_ ? std::min<double>(len, window_ + n) : len;
-                seen += window_ ? n * std::min<double>(len, window_) : n * (len - n) + n * (n + 1) / 2.0;
-            }
-            LaunchProfile::get().note_cost(read * row * dtype_size(cache.kv_dtype) + (double)T * heads_ * (row * es + kv_rank_ * 4.0),
-                                           2.0 * seen * heads_ * (row + kv_rank_));
-        }
+        Tensor out = ws.get("la_heads", {T, (int64_t)heads_ * vdim_}, dt);
+        const char* gate = gated_ ? static_cast<const char*>(down.data) + (size_t)(q_cols_ + row) * es : nullptr;
         // 16-byte copies: the rows of this entry start on such a boundary in every page (other entries of the group may not)
         const bool aligned = reinterpret_cast<uintptr_t>(cache.k_base) % 16 == 0 && cache.page_stride % 8 == 0;
-        if (on_tensor_cores() && cache.kv_dtype == DType::BF16 && aligned) {
-            const LatentKernels& lk = latent_kernels();
-            const StepArray tiles = ctx.array(tiles_name() + ".seg"), firsts = ctx.array(tiles_name() + ".first");
-            if (!tiles.count) throw Error(kInvalidState, "latent_attention: the step carries no tiles for this mixer");
-            int splits = (int)ctx.option_int("latent_splits");           // a test's choice, else what fills the device
-            if (splits < 1) splits = key_splits(tiles.count, std::max(ctx.decode_max_ctx, ctx.prefill_max_ctx), sm_count());
-            float *part_o = nullptr, *part_ml = nullptr;
-            if (splits > 1) {
-                part_o = ws.get("la_part_o", {tiles.count, splits, kTileRows, kv_rank_}, DType::F32).as<float>();
-                part_ml = ws.get("la_part_ml", {tiles.count, splits, kTileRows, 2}, DType::F32).as<float>();
+        const bool tiled = on_tensor_cores() && cache.kv_dtype == DType::BF16 && aligned;
+        const StepArray tiles = ctx.array(tiles_name() + ".seg"), firsts = ctx.array(tiles_name() + ".first");
+        const int n_dense = may_go_dense() && cache.kv_dtype == DType::BF16 ? ctx.array("latent.dense.segs").count : 0;
+        // rows that attend over the latents themselves: every row of the step, unless its long portions go the other way (a
+        // mixed step's long rows pass through here too and are overwritten)
+        if (n_dense < ctx.S) {
+            Tensor q_lat = ws.get("la_q_lat", {T, heads_, row}, dt);
+            if (LaunchProfile::get().on())
+                LaunchProfile::get().note_cost((double)T * heads_ * (dim_ + rot_ + row) * es + (double)k_up_.bytes(), 2.0 * T * heads_ * dim_ * kv_rank_);
+            const bool tc_products = products_on_tensor_cores() && dt == DType::BF16;
+            if (tc_products) {
+                const LatentKernels& lk = latent_kernels();
+                QE_LAUNCH(lk, lk.latent_absorb(q.data, q_stride, k_up_.data, table, n_rot, max_pos, positions, q_lat.data, T, heads_, dim_, rot_, kv_rank_, ctx.stream));
+            } else
+            QE_LAUNCH(k, k.latent_absorb(q.data, q.code(), q_stride, k_up_.data, k_up_.code(), table, n_rot, max_pos, positions, q_lat.data, q_lat.code(), T,
+                                         heads_, dim_, rot_, kv_rank_, ctx.stream));
+            // every head reads the one cached row per position: keys the whole row, values its first kv_rank numbers
+            Tensor o_lat = ws.get("la_o_lat", {T, heads_, kv_rank_}, DType::F32);
+            const int32_t* abs_positions = ctx.position_column(0);
+            if (LaunchProfile::get().on()) {
+                double seen = 0.0, read = 0.0;
+                for (size_t i = 0; i < ctx.q_lens.size(); i++) {
+                    const double n = ctx.q_lens[i], len = ctx.ctx_lens[i];
+                    read += window_ ? std::min<double>(len, window_ + n) : len;
+                    seen += window_ ? n * std::min<double>(len, window_) : n * (len - n) + n * (n + 1) / 2.0;
+                }
+                LaunchProfile::get().note_cost(read * row * dtype_size(cache.kv_dtype) + (double)T * heads_ * (row * es + kv_rank_ * 4.0),
+                                               2.0 * seen * heads_ * (row + kv_rank_));
             }
-            QE_LAUNCH(lk, lk.attention(q_lat.data, cache.k_base, cache.page_stride, cache.page_size, g.block_table, g.table_width, ctx.seg_start,
-                                       ctx.seg_ctx_len, tiles.data, firsts.data, tiles.count, o_lat.data, part_o, part_ml, heads_, kv_rank_,
-                                       rot_, window_, (float)scale_, splits, ctx.stream));
-        } else
-        QE_LAUNCH(k, k.attention_generic(q_lat.data, q_lat.code(), cache.k_base, cache.k_base, (int)cache.kv_dtype, cache.page_stride,
-                                         cache.page_size, g.block_table, g.table_width, ctx.row_seg, abs_positions, o_lat.data, o_lat.code(),
-                                         T, heads_, 1, row, window_, (float)scale_, kv_rank_, 0, row, ctx.stream));
-        Tensor out = ws.get("la_heads", {T, (int64_t)heads_ * vdim_}, dt);
-        if (LaunchProfile::get().on())
-            LaunchProfile::get().note_cost((double)T * heads_ * (kv_rank_ * 4.0 + (vdim_ + gate_cols_) * es) + (double)v_up_.bytes(), 2.0 * T * heads_ * vdim_ * kv_rank_);
-        const char* gate = gated_ ? static_cast<const char*>(down.data) + (size_t)(q_cols_ + row) * es : nullptr;
-        if (tc_products && T > kFewRows) {               // few rows: more CTAs with a warp per value column
-            const LatentKernels& lk = latent_kernels();
-            QE_LAUNCH(lk, lk.latent_expand(o_lat.data, v_up_.data, gate, down_width_, gate_cols_, out.data, T, heads_, kv_rank_, vdim_, ctx.stream));
-        } else
-        QE_LAUNCH(k, k.latent_expand(o_lat.data, o_lat.code(), v_up_.data, v_up_.code(), gate, down.code(), down_width_, gate_cols_, out.data, out.code(), T,
-                                     heads_, kv_rank_, vdim_, ctx.stream));
+            if (tiled) {
+                const LatentKernels& lk = latent_kernels();
+                if (!tiles.count) throw Error(kInvalidState, "latent_attention: the step carries no tiles for this mixer");
+                int splits = (int)ctx.option_int("latent_splits");           // a test's choice, else what fills the device
+                if (splits < 1) splits = key_splits(tiles.count, std::max(ctx.decode_max_ctx, ctx.prefill_max_ctx), sm_count());
+                float *part_o = nullptr, *part_ml = nullptr;
+                if (splits > 1) {
+                    part_o = ws.get("la_part_o", {tiles.count, splits, kTileRows, kv_rank_}, DType::F32).as<float>();
+                    part_ml = ws.get("la_part_ml", {tiles.count, splits, kTileRows, 2}, DType::F32).as<float>();
+                }
+                QE_LAUNCH(lk, lk.attention(q_lat.data, cache.k_base, cache.page_stride, cache.page_size, g.block_table, g.table_width, ctx.seg_start,
+                                           ctx.seg_ctx_len, tiles.data, firsts.data, tiles.count, o_lat.data, part_o, part_ml, heads_, kv_rank_,
+                                           rot_, window_, (float)scale_, splits, ctx.stream));
+            } else
+            QE_LAUNCH(k, k.attention_generic(q_lat.data, q_lat.code(), cache.k_base, cache.k_base, (int)cache.kv_dtype, cache.page_stride,
+                                             cache.page_size, g.block_table, g.table_width, ctx.row_seg, abs_positions, o_lat.data, o_lat.code(),
+                                             T, heads_, 1, row, window_, (float)scale_, kv_rank_, 0, row, ctx.stream));
+            if (LaunchProfile::get().on())
+                LaunchProfile::get().note_cost((double)T * heads_ * (kv_rank_ * 4.0 + (vdim_ + gate_cols_) * es) + (double)v_up_.bytes(), 2.0 * T * heads_ * vdim_ * kv_rank_);
+            if (tc_products && T > kFewRows) {               // few rows: more CTAs with a warp per value column
+                const LatentKernels& lk = latent_kernels();
+                QE_LAUNCH(lk, lk.latent_expand(o_lat.data, v_up_.data, gate, down_width_, gate_cols_, out.data, T, heads_, kv_rank_, vdim_, ctx.stream));
+            } else
+            QE_LAUNCH(k, k.latent_expand(o_lat.data, o_lat.code(), v_up_.data, v_up_.code(), gate, down.code(), down_width_, gate_cols_, out.data, out.code(), T,
+                                         heads_, kv_rank_, vdim_, ctx.stream));
+        }
+        if (n_dense) forward_dense(down, out, ctx, cache, g, gate);
         return o_proj_(out, ctx, "la_out", DType::F32, T, true, false, ctx.residual, nullptr, &ctx.norm_ahead);
     }
 
@@ -263,8 +327,58 @@ private:
         }
         return best;
     }
-    std::string tiles_name() const { return "latent.tiles.h" + std::to_string(heads_) + (window_ ? ".w" + std::to_string(window_) : ""); }
+    std::string tiles_name() const {
+        return "latent.tiles.h" + std::to_string(heads_) + (window_ ? ".w" + std::to_string(window_) : "") + (may_go_dense() ? ".rest" : "");
+    }
 
+    // The step's long portions: the heads' keys and values from the requests' latents, and attention over them into `out`.
+    void forward_dense(const Tensor& down, Tensor& out, StepContext& ctx, const CacheView& cache, const GroupStep& g, const char* gate) {
+        const StepArray segs = ctx.array("latent.dense.segs"), base = ctx.array("latent.dense.base");
+        const StepArray tile_seg = ctx.array("latent.dense.tile_seg"), tile_first = ctx.array("latent.dense.tile_first");
+        const CoreKernels& k = core_kernels();
+        const FlashKernels& f = flash_kernels();
+        Workspace& ws = *ctx.workspace;
+        int rows = 0, longest = 0;
+        double seen = 0.0, queries = 0.0;
+        for (size_t i = 0; i < ctx.q_lens.size(); i++) {
+            const int n = ctx.q_lens[i], len = ctx.ctx_lens[i];
+            if (n < kDenseRows || rows + len > kDenseMax) continue;      // as add_dense() chose
+            rows += len;
+            longest = std::max(longest, len);
+            queries += n;
+            seen += (double)n * (len - n) + (double)n * (n + 1) / 2.0;
+        }
+        const size_t es = dtype_size(DType::BF16);
+        Tensor latents = ws.get("la_dense_rows", {rows, kv_rank_}, DType::BF16);
+        if (LaunchProfile::get().on()) LaunchProfile::get().note_cost(2.0 * rows * kv_rank_ * es, 0.0);
+        QE_LAUNCH(k, k.latent_gather(cache.k_base, (int)cache.kv_dtype, cache.page_stride, cache.page_size, g.block_table, g.table_width, segs.data,
+                                     segs.count, base.data, ctx.seg_ctx_len, longest, latents.data, kv_rank_, kv_rank_ + rot_, ctx.stream));
+        const int64_t width = (int64_t)heads_ * (dim_ + vdim_);
+        Tensor kv = kv_up_(latents, ctx, "la_dense_kv", DType::BF16, rows).tensor;                // [rows, keys of all heads | values]
+        const char* values = static_cast<const char*>(kv.data) + (size_t)heads_ * dim_ * es;
+        int splits = (int)ctx.option_int("prefill_splits");
+        if (!splits) splits = dense_splits(tile_seg.count, longest);
+        float *part_o = nullptr, *part_ml = nullptr;
+        if (splits > 1) {
+            part_o = ws.get("attn_tile_part_o", {ctx.T, heads_, splits, dim_}, DType::F32).as<float>();
+            part_ml = ws.get("attn_tile_part_ml", {ctx.T, heads_, splits, 2}, DType::F32).as<float>();
+        }
+        if (LaunchProfile::get().on())
+            LaunchProfile::get().note_cost((double)rows * width * es + queries * heads_ * (dim_ + 2.0 * vdim_) * es, 2.0 * seen * heads_ * (dim_ + vdim_));
+        QE_LAUNCH(f, f.prefill_tc5_dense(down.data, down_width_, ctx.T, kv.data, values, width, rows, base.data, ctx.seg_start, ctx.seg_ctx_len,
+                                         tile_seg.data, tile_first.data, tile_seg.count, out.data, heads_, dim_, (float)scale_, splits, part_o, part_ml,
+                                         ctx.attention_error, gate, down_width_, ctx.stream));
+    }
+    // CTAs per tile when there are few tiles: enough to fill the device about once
+    int dense_splits(int n_tiles, int longest) const {
+        const int ctas = n_tiles * heads_, places = 2 * sm_count();
+        if (2 * ctas > places) return 1;
+        return std::max(1, std::min({places / std::max(ctas, 1), (longest + 63) / 64 / 4, 8}));
+    }
+
+    static constexpr int kDenseRows = 128;       // the shortest portion whose keys and values are made for it
+    static constexpr int kDenseMax = 16384;      // rows of a step that they may be made for
+    static constexpr int kDenseTile = 128;       // rows of a tile of the tcgen05 prompt kernel
     static constexpr int kFewRows = 16;
     static constexpr int kTileRows = 64;         // (token, head) pairs of a tile of the tensor-core kernel
     static constexpr int kMaxRow = 640;          // the widest cache row the attention kernel holds a query for
@@ -274,7 +388,7 @@ private:
     double eps_, scale_;
     std::string gemm_, attention_;
     std::shared_ptr<PositionEncoding> position_;
-    Linear down_proj_, q_up_, o_proj_;
+    Linear down_proj_, q_up_, kv_up_, o_proj_;
     Tensor q_norm_, kv_norm_, k_up_, v_up_, table_;
 };
 

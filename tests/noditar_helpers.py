@@ -55,10 +55,11 @@ CONFIG_C = config(128, 200, 3, [
     (latent(6, 48, 32, 160, 0.15), dense(96, 0.8)),
 ], eps=1e-6)
 
-# heads of 128, which take the tcgen05 prompt kernel and the TMA decode kernel; one stream; a latent of 512 and of 264
+# heads of 128, which take the tcgen05 prompt kernel and the TMA decode kernel; one stream; a latent of 512 whose heads of
+# 128 / 128 get keys and values of their own for long portions, and one of 264 whose heads do not
 CONFIG_D = config(96, 60, 1, [
     (biased(4, 2, 128, 128, 0.09), dense(64, 1.3)),
-    (latent(2, 128, 64, 512, 0.09), None),
+    (latent(2, 128, 128, 512, 0.09), None),
     (biased(2, 2, 128, 128, 0.07), None),
     (latent(3, 64, 128, 264, 0.1), dense(48, 2.0)),
 ], eps=1e-5)

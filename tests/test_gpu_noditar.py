@@ -244,13 +244,25 @@ def whole_cut_decoded_and_batched(p, x, ref, tol):
     again = p.mixer_step([(4, 2), (3, 1)], np.concatenate([x[90:92], x[151:152]]))
     close(np.concatenate([a, both[:1], again[2:]]), ref[:152], tol)
     close(np.concatenate([both[1:], again[:2]]), ref[:92], tol)
+    # a long portion late in a request beside a decode row, a short portion, and another long one
+    p.release(3); p.release(4)
+    for r in (5, 6, 7):
+        p.add_request(r)
+    first = p.mixer_step([(5, 40), (6, 33)], np.concatenate([x[:40], x[:33]]))
+    mixed = p.mixer_step([(6, 1), (5, 140), (7, 129)], np.concatenate([x[33:34], x[40:180], x[:129]]))
+    last = p.mixer_step([(7, 3), (5, 2), (6, 1)], np.concatenate([x[129:132], x[180:182], x[34:35]]))
+    close(np.concatenate([first[:40], mixed[1:141], last[3:5]]), ref[:182], tol)
+    close(np.concatenate([first[40:], mixed[:1], last[5:]]), ref[:35], tol)
+    close(np.concatenate([mixed[141:], last[:3]]), ref[:132], tol)
+    for r in (5, 6, 7):
+        p.release(r)
 
 
 # latents of 12 to 512: every width of the tensor-core kernel, and 12 and 20, which go the plain way; one head alone
 LATENTS = {
     "r12": (latent(4, 16, 20, 12, 2.0), 64), "r20": (latent(3, 24, 8, 20, 1.5), 40), "r64": (latent(8, 32, 48, 64, 1.0), 72),
     "r136": (latent(5, 48, 40, 136, 0.7), 64), "r256": (latent(1, 64, 64, 256, 0.5), 48), "r264": (latent(6, 40, 24, 264, 0.6), 64),
-    "r512": (latent(2, 128, 128, 512, 0.4), 64),
+    "r512": (latent(2, 128, 128, 512, 0.4), 64), "r72": (latent(3, 128, 128, 72, 0.3), 40),      # long portions: keys and values of their own
 }
 
 
