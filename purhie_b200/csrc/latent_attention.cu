@@ -143,27 +143,67 @@ constexpr int EX_TOK = 8, EX_WARPS = 8;
 // lanes walk c, 32 apart, for EX_TOK tokens at once, and add up with a butterfly.
 template <typename TI, typename TW, typename TG, typename TO>
 __global__ void latent_expand_kernel(const TI* __restrict__ o_lat, const TW* __restrict__ wuv, const TG* __restrict__ gate,
-                                     long long gate_stride, int gate_cols, TO* __restrict__ out, int T, int H, int C, int DV) {
-    extern __shared__ float os[];      // [EX_TOK][C]
+                                     long long gate_stride, int gate_cols, TO* __restrict__ out, int T, int H, int C, int DV, int vec) {
+    extern __shared__ __align__(16) float os[];      // [EX_TOK][C]
     pdl_launch_dependents();
-    pdl_wait();
     const int h = blockIdx.y, t0 = blockIdx.z * EX_TOK;
-    for (int i = threadIdx.x; i < EX_TOK * C; i += blockDim.x) {
-        const int tt = i / C, c = i % C;
-        os[i] = t0 + tt < T ? to_float<TI>(o_lat[((size_t)(t0 + tt) * H + h) * C + c]) : 0.0f;
-    }
-    __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int v = blockIdx.x * EX_WARPS + warp;
-    if (v >= DV) return;
-    const TW* w = wuv + ((size_t)h * DV + v) * C;
+    const TW* w = wuv + ((size_t)h * DV + min(v, DV - 1)) * C;
     float acc[EX_TOK];
 #pragma unroll
     for (int i = 0; i < EX_TOK; ++i) acc[i] = 0.0f;
-    for (int c = lane; c < C; c += 32) {
-        const float wv = to_float<TW>(w[c]);
+    if (vec) {
+        // rows of a multiple of eight numbers: 16-byte accesses, and the weights (which no kernel of the step writes) are on
+        // their way while the kernel in front still runs
+        constexpr int AHEAD = 2;
+        float wv[AHEAD][8];
 #pragma unroll
-        for (int i = 0; i < EX_TOK; ++i) acc[i] = fmaf(os[i * C + c], wv, acc[i]);
+        for (int j = 0; j < AHEAD; ++j)
+            if ((j * 32 + lane) * 8 < C) load8(w + (j * 32 + lane) * 8, wv[j]);
+        pdl_wait();
+#pragma unroll
+        for (int tt = 0; tt < EX_TOK; ++tt)
+            for (int c = threadIdx.x * 4; c < C; c += EX_WARPS * 32 * 4) {
+                const float4 u = t0 + tt < T ? load4(o_lat + ((size_t)(t0 + tt) * H + h) * C + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                *reinterpret_cast<float4*>(os + tt * C + c) = u;
+            }
+        __syncthreads();
+        if (v >= DV) return;
+        for (int c0 = 0, j = 0; c0 < C; c0 += 256, ++j) {
+            const int c = c0 + lane * 8;
+            if (c >= C) break;
+            float ww[8];
+            if (j == 0) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ww[e] = wv[0][e];
+            } else if (j == 1) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ww[e] = wv[1][e];
+            } else {
+                load8(w + c, ww);
+            }
+#pragma unroll
+            for (int i = 0; i < EX_TOK; ++i) {
+                const float4 x = *reinterpret_cast<const float4*>(os + i * C + c), y = *reinterpret_cast<const float4*>(os + i * C + c + 4);
+                acc[i] = fmaf(x.x, ww[0], acc[i]); acc[i] = fmaf(x.y, ww[1], acc[i]); acc[i] = fmaf(x.z, ww[2], acc[i]); acc[i] = fmaf(x.w, ww[3], acc[i]);
+                acc[i] = fmaf(y.x, ww[4], acc[i]); acc[i] = fmaf(y.y, ww[5], acc[i]); acc[i] = fmaf(y.z, ww[6], acc[i]); acc[i] = fmaf(y.w, ww[7], acc[i]);
+            }
+        }
+        __syncwarp();                                  // lanes that had nothing to add join for the sums
+    } else {
+        pdl_wait();
+        for (int i = threadIdx.x; i < EX_TOK * C; i += blockDim.x) {
+            const int tt = i / C, c = i % C;
+            os[i] = t0 + tt < T ? to_float<TI>(o_lat[((size_t)(t0 + tt) * H + h) * C + c]) : 0.0f;
+        }
+        __syncthreads();
+        if (v >= DV) return;
+        for (int c = lane; c < C; c += 32) {
+            const float wv = to_float<TW>(w[c]);
+#pragma unroll
+            for (int i = 0; i < EX_TOK; ++i) acc[i] = fmaf(os[i * C + c], wv, acc[i]);
+        }
     }
 #pragma unroll
     for (int i = 0; i < EX_TOK; ++i) {
@@ -244,10 +284,11 @@ PH_EXPORT int ph_latent_expand(const void* o_lat, int in_dtype, const void* wuv,
     if (T == 0) return PH_OK;
     const size_t smem = (size_t)EX_TOK * C * sizeof(float);
     if (smem > 48 * 1024) return fail(PH_ERR_UNSUPPORTED, "latent_expand: a latent of %d does not fit", C);
+    const int vec = C % 8 == 0 && (((uintptr_t)o_lat | (uintptr_t)wuv) & 15) == 0;
     const dim3 grid((unsigned)((DV + EX_WARPS - 1) / EX_WARPS), (unsigned)H, (unsigned)((T + EX_TOK - 1) / EX_TOK));
 #define LAUNCH(TI, TW, TG, TO)                                                                                                   \
     launch_overlapped(latent_expand_kernel<TI, TW, TG, TO>, grid, dim3(EX_WARPS * 32), smem, stream, (const TI*)o_lat, (const TW*)wuv, \
-                      (const TG*)gate, gate_stride, gate_cols, (TO*)out, T, H, C, DV)
+                      (const TG*)gate, gate_stride, gate_cols, (TO*)out, T, H, C, DV, vec)
     PH_DISPATCH(in_dtype, TI, PH_DISPATCH(w_dtype, TW, PH_DISPATCH(gate_dtype, TG, PH_DISPATCH(out_dtype, TO, LAUNCH(TI, TW, TG, TO)))));
 #undef LAUNCH
     return check_launch("latent_expand");

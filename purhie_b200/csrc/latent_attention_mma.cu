@@ -22,6 +22,7 @@ using namespace ph_attn;
 
 constexpr int LA_ROWS = 64;        // query rows of a tile
 constexpr int LA_THREADS = 256;
+constexpr int MAX_SPLITS = 64;     // CTAs that may share a tile's keys
 
 template <int CP, int RP> struct LatentShape {
     static constexpr int DK = CP + RP;
@@ -221,22 +222,44 @@ __global__ void latent_attention_combine_kernel(const float* __restrict__ part_o
     const int row0 = seg_start[seg], q_len = seg_start[seg + 1] - row0;
     if (r >= q_len * H - first) return;
     const size_t part = (size_t)tile * splits * LA_ROWS + r;
-    float top = -INFINITY;
-    for (int s = 0; s < splits; ++s) top = fmaxf(top, part_ml[(part + (size_t)s * LA_ROWS) * 2]);
-    float sum = 0.0f;
-    for (int s = 0; s < splits; ++s) {
-        const float* ml = part_ml + (part + (size_t)s * LA_ROWS) * 2;
-        if (ml[1] > 0.0f) sum += exp2f(ml[0] - top) * ml[1];
-    }
-    const float inv = sum > 0.0f ? 1.0f / sum : 0.0f;
-    float* dst = out + ((size_t)row0 * H + first + r) * C;
-    for (int d = threadIdx.x; d < C; d += blockDim.x) {
-        float acc = 0.0f;
-        for (int s = 0; s < splits; ++s) {
-            const float* ml = part_ml + (part + (size_t)s * LA_ROWS) * 2;
-            if (ml[1] > 0.0f) acc += exp2f(ml[0] - top) * part_o[(part + (size_t)s * LA_ROWS) * C + d];
+    // the weights of all splits at once, by the first warp (its lanes take the splits 32 apart; the sum runs in their order)
+    __shared__ float weight[MAX_SPLITS];
+    __shared__ float inv_sum;
+    if (threadIdx.x < 32) {
+        const int lane = threadIdx.x;
+        float top = -INFINITY;
+        for (int s = lane; s < splits; s += 32) top = fmaxf(top, part_ml[(part + (size_t)s * LA_ROWS) * 2]);
+        top = warp_max(top);
+        float sum = 0.0f;
+        for (int s0 = 0; s0 < splits; s0 += 32) {
+            const int s = s0 + lane;
+            const float2 ml = s < splits ? *(const float2*)(part_ml + (part + (size_t)s * LA_ROWS) * 2) : make_float2(-INFINITY, 0.0f);
+            const float w = ml.y > 0.0f ? exp2f(ml.x - top) : 0.0f;
+            if (s < splits) weight[s] = w;
+            sum += warp_sum(w * ml.y);
         }
-        dst[d] = acc * inv;
+        if (lane == 0) inv_sum = sum > 0.0f ? 1.0f / sum : 0.0f;
+    }
+    __syncthreads();
+    float* dst = out + ((size_t)row0 * H + first + r) * C;
+    const float* src = part_o + part * C;
+    const size_t step = (size_t)LA_ROWS * C;
+    for (int d = threadIdx.x * 4; d < C; d += blockDim.x * 4) {      // C is a multiple of 8
+        float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (int s0 = 0; s0 < splits; s0 += 8) {
+            float4 u[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+                u[j] = s0 + j < splits && weight[s0 + j] > 0.0f ? load4(src + (s0 + j) * step + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+                if (s0 + j < splits) {
+                    const float w = weight[s0 + j];
+                    acc.x = fmaf(w, u[j].x, acc.x); acc.y = fmaf(w, u[j].y, acc.y); acc.z = fmaf(w, u[j].z, acc.z); acc.w = fmaf(w, u[j].w, acc.w);
+                }
+        }
+        const float inv = inv_sum, v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+        store4(dst + d, v);
     }
 }
 
@@ -441,7 +464,7 @@ PH_EXPORT int ph_latent_attention(const void* q, const void* k_base, long long p
                                   const int32_t* tile_first, int n_tiles, void* out, float* part_o, float* part_ml, int H, int C, int R,
                                   int window, float scale, int splits, cudaStream_t stream) {
     if (!q || !k_base || !block_table || !seg_start || !seg_ctx_len || !tile_seg || !tile_first || !out || n_tiles < 0 || H < 1 ||
-        page_size < 1 || window < 0 || splits < 1 || (splits > 1 && (!part_o || !part_ml)))
+        page_size < 1 || window < 0 || splits < 1 || splits > MAX_SPLITS || (splits > 1 && (!part_o || !part_ml)))
         return fail(PH_ERR_ARG, "latent_attention: bad arguments (tiles %d, H %d, splits %d)", n_tiles, H, splits);
     if (!ph_latent_attention_supports(C, R))
         return fail(PH_ERR_UNSUPPORTED, "latent_attention: rows of %d + %d numbers are not taken (multiples of 8, at most 512 + 64)", C, R);
