@@ -317,7 +317,7 @@ def test_attention_with_a_distance_bias_a_sink_and_a_gate_alone(tmp_path, which,
 
 # states, groups, taps and norm parts of every kind; r32, r64 and r72 run long portions in chunks on the tensor cores
 MAMBAS = {
-    "r32": (mamba2(4, 32, 48, 2, 4, 2), 64), "r64": (mamba2(2, 64, 128, 1, 3, 4), 48), "r72": (mamba2(3, 72, 8, 3, 2, 1), 40), "r5": (mamba2(6, 5, 7, 2, 5, 10), 32),
+    "r32": (mamba2(6, 32, 40, 2, 4, 3), 64), "r64": (mamba2(2, 64, 128, 1, 3, 4), 48), "r72": (mamba2(3, 72, 8, 3, 2, 1), 40), "r5": (mamba2(6, 5, 7, 2, 5, 10), 32),
     "r16": (mamba2(1, 16, 200, 1, 1, 1), 24), "r8": (mamba2(8, 8, 16, 8, 4, 16), 56), "r40": (mamba2(2, 40, 256, 2, 4, 2), 32),
 }
 
@@ -362,7 +362,7 @@ def test_chunks_and_single_steps_of_the_scan_agree_wherever_a_prompt_is_cut(tmp_
 def test_the_first_token_still_shows_hundreds_of_tokens_later_in_a_state_that_hardly_forgets(tmp_path):
     for dtype in ("float32", "bfloat16"):
         cfg, w, folder, width = mamba_case(tmp_path / dtype, "r32", dtype)
-        w["l0.mix.A_log"] = np.full(4, -7.0, dtype=np.float32)                # a decay of about 1/1000 per unit of dt
+        w["l0.mix.A_log"] = np.full(6, -7.0, dtype=np.float32)                # a decay of about 1/1000 per unit of dt
         folder = make_folder(tmp_path / dtype, cfg, w, "F32" if dtype == "float32" else "BF16")
         m, eps, wd = cfg["layers"][0]["mixer"], cfg["norm"]["eps"], f64(w)
         x = inputs(400, width, 4, dtype)

@@ -15,7 +15,7 @@ def i32(x):
 
 # ---- the residual of several lanes -----------------------------------------------------------------------------------
 # clusters for few rows, a block per row for many; one to nine lanes; widths that no vector access fits
-@pytest.mark.parametrize("S,E,T,splits", [(3, 256, 5, 1), (4, 4096, 8, 9), (4, 4096, 200, 1), (2, 2048, 70, 3), (1, 512, 3, 2), (5, 1000, 66, 1),
+@pytest.mark.parametrize("S,E,T,splits", [(3, 320, 5, 1), (4, 4096, 8, 9), (4, 4096, 200, 1), (2, 2048, 70, 3), (1, 512, 3, 2), (5, 1000, 66, 1),
                                           (8, 8192, 2, 4), (7, 50, 9, 3), (9, 128, 4, 2), (3, 12000, 3, 1), (3, 4, 65, 1)])
 @pytest.mark.parametrize("out_dtype", [torch.float32, torch.bfloat16])
 def test_lanes_rmsnorm(S, E, T, splits, out_dtype):
@@ -110,7 +110,7 @@ def run_ssd(case, kind, **limits):
 
 
 # states of 1 to 300 with and without whole quads, one lane group and several per lane; values that end inside a block
-@pytest.mark.parametrize("H,P,N,G,K", [(4, 32, 48, 2, 4), (6, 10, 6, 3, 1), (2, 64, 128, 1, 4), (3, 5, 33, 3, 6), (2, 72, 300, 2, 3), (1, 7, 1, 1, 2),
+@pytest.mark.parametrize("H,P,N,G,K", [(6, 32, 40, 2, 4), (6, 10, 6, 3, 1), (2, 64, 128, 1, 4), (3, 5, 33, 3, 6), (2, 72, 300, 2, 3), (1, 7, 1, 1, 2),
                                        (2, 16, 250, 1, 2)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_ssd_scan_token_by_token(H, P, N, G, K, dtype):
@@ -120,7 +120,7 @@ def test_ssd_scan_token_by_token(H, P, N, G, K, dtype):
 
 
 # chunks full and cut, states of 8 to 256, values that end inside a block of 32 and beyond it; decays of a few tokens' reach
-@pytest.mark.parametrize("H,P,N,G,K,fast", [(4, 32, 48, 2, 4, False), (2, 64, 128, 1, 4, False), (2, 64, 128, 2, 4, True), (3, 40, 8, 3, 2, False),
+@pytest.mark.parametrize("H,P,N,G,K,fast", [(6, 32, 40, 2, 4, False), (2, 64, 128, 1, 4, False), (2, 64, 128, 2, 4, True), (3, 40, 8, 3, 2, False),
                                             (2, 72, 144, 1, 1, False), (1, 8, 256, 1, 3, False), (2, 96, 64, 2, 4, True)])
 def test_ssd_chunks_on_the_tensor_cores(H, P, N, G, K, fast):
     from purhie_b200.csrc import ops
@@ -158,7 +158,7 @@ def test_gate_rms_in_parts(T, inner, parts, extra, dtype):
 
 
 # ---- a bias linear in the distance -----------------------------------------------------------------------------------
-@pytest.mark.parametrize("dtype,HQ,HKV,D", [(torch.float32, 5, 1, 24), (torch.bfloat16, 4, 2, 48), (torch.bfloat16, 20, 4, 32)])
+@pytest.mark.parametrize("dtype,HQ,HKV,D", [(torch.float32, 5, 1, 24), (torch.bfloat16, 6, 2, 48), (torch.bfloat16, 20, 4, 32)])
 def test_a_bias_linear_in_the_distance_in_the_plain_and_the_tile_kernel(dtype, HQ, HKV, D):
     from purhie_b200.csrc import ops
     segs = [(1, 1), (64, 64), (200, 130), (300, 1), (65, 2)]
