@@ -282,9 +282,6 @@ def main():
                     help="instead of the headline workload: prefill and decode of this design at real layer sizes beside four "
                          "Qwen3 layers of equal size, with the time and roofline fraction of every kernel class")
     ap.add_argument("--size", default="4k", choices=sorted(DESIGN_SIZES), help="with --design: the layer sizes")
-    ap.add_argument("--leave-out", default="", metavar="NAMES",
-                    help="with --phase decode: launchers (comma separated, e.g. add_rmsnorm,decode_bulk) that the timed steps "
-                         "skip; the difference to a run without shows what they cost inside the graph (no benchmark value)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -366,12 +363,6 @@ def main():
         bytes_step = weight_bytes + batch * (ctx0 + steps / 2.0) * kv_bytes_per_token
         return ms, launches, bytes_step
 
-    if args.leave_out:
-        if args.phase != "decode":
-            print("bench.py: --leave-out goes with --phase decode")
-            return 2
-        from purhie_b200 import native
-        native.lib().qe_profile_leave_out(args.leave_out.encode())     # the graphs are captured after this
     from purhie_b200 import native as _native
     if _native.profile_enabled():
         _native.profile_report(True)                 # what came before the timed steps does not count
@@ -403,8 +394,7 @@ def main():
         from purhie_b200 import native
         if native.profile_enabled():             # PURHIE_PROFILE=1: every launch between events, graphs off
             sys.stderr.write(native.format_profile(native.profile_report(), f"decode, batch {args.batch}, {args.layers} layers") + "\n")
-        print(json.dumps({"phase": "decode", "batch": args.batch, "ms_per_step": ms_step, "layers": args.layers,
-                          "left_out": args.leave_out or None}))
+        print(json.dumps({"phase": "decode", "batch": args.batch, "ms_per_step": ms_step, "layers": args.layers}))
         return 0
 
     # ---- end to end through the Python entry point ------------------------------------------------------

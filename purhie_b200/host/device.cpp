@@ -272,23 +272,6 @@ std::string LaunchProfile::launcher_name(const char* call_text) {
     if (dot != std::string::npos) name = name.substr(dot + 1);
     return name;
 }
-void LaunchProfile::leave_out(const char* names) {
-    left_out_.clear();
-    std::string all(names ? names : "");
-    size_t at = 0;
-    while (at <= all.size()) {
-        size_t comma = all.find(',', at);
-        if (comma == std::string::npos) comma = all.size();
-        if (comma > at) left_out_.push_back(all.substr(at, comma - at));
-        at = comma + 1;
-    }
-}
-bool LaunchProfile::is_left_out(const char* call_text) const {
-    const std::string name = launcher_name(call_text);
-    for (const std::string& n : left_out_)
-        if (n == name) return true;
-    return false;
-}
 void LaunchProfile::begin(const char* call_text) {
     Record r;
     r.name = launcher_name(call_text);
