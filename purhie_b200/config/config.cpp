@@ -337,6 +337,7 @@ void register_sizizen_architecture();
 void register_zerusun_architecture();
 void register_vokepel_architecture();
 void register_noditar_architecture();
+void register_defapel_architecture();
 
 void register_builtin_architectures() {
     static std::once_flag once;
@@ -347,6 +348,7 @@ void register_builtin_architectures() {
         register_zerusun_architecture();
         register_vokepel_architecture();
         register_noditar_architecture();
+        register_defapel_architecture();
     });
 }
 

@@ -55,6 +55,7 @@ struct BulkParams {
     int* error_flag;
     const float* sink;             // [HQ] float32 or null: exp(sink) joins each head's denominator, once per row
     const float* slopes;           // [HQ] float32 or null: taken off the scores per position of distance
+    float to_cap, cap_log2;        // KIND 2: scale / cap and cap * log2(e)
     const __nv_bfloat16* gate; long long gate_stride;      // rows of HQ * D logits (by token row), or null
 };
 
@@ -106,7 +107,8 @@ __host__ __device__ constexpr int bulk_smem_bytes(int D, int G, int stages) {
            (2 * stages + 4) * 8 + PAGE_CACHE * 4;
 }
 
-template <int D, int STAGES, int CTAS, bool BIAS>
+// KIND: what happens to a scaled score in front of the softmax: 0 nothing, 1 a distance bias, 2 a cap.
+template <int D, int STAGES, int CTAS, int KIND>
 __global__ void __launch_bounds__(BULK_THREADS, CTAS)
 attention_decode_bulk_kernel(const __grid_constant__ CUtensorMap map_kv, const BulkParams p) {
     constexpr int HALVES = D / 64;
@@ -291,17 +293,26 @@ attention_decode_bulk_kernel(const __grid_constant__ CUtensorMap map_kv, const B
 #pragma unroll
                 for (int i = 0; i < 4; ++i) o[dt][i] = 0.0f;
 
-            const float slope0 = BIAS ? p.slopes[it.g * G + min(r0, G - 1)] * LOG2E : 0.0f;
-            const float slope1 = BIAS ? p.slopes[it.g * G + min(r1, G - 1)] * LOG2E : 0.0f;
-            const float scale_log2 = BIAS ? 1.0f : p.scale_log2;
-            // (BIAS) the scores in log2 units, each row's share of the distance taken off
+            const float slope0 = KIND == 1 ? p.slopes[it.g * G + min(r0, G - 1)] * LOG2E : 0.0f;
+            const float slope1 = KIND == 1 ? p.slopes[it.g * G + min(r1, G - 1)] * LOG2E : 0.0f;
+            const float scale_log2 = KIND ? 1.0f : p.scale_log2;
+            // the scores in log2 units, each row's share of the distance taken off, or bent by the cap
             auto bias = [&](float (&s)[2][4], int key0) {
-                if constexpr (BIAS) {
+                if constexpr (KIND == 1) {
 #pragma unroll
                     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
                         for (int i = 0; i < 4; ++i)
                             s[nt][i] = fmaf(s[nt][i], p.scale_log2, (i < 2 ? slope0 : slope1) * (float)(key0 + nt * 8 + (lane & 3) * 2 + (i & 1) - it.z));
+                }
+                if constexpr (KIND == 2) {
+#pragma unroll
+                    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const float e = __expf(-2.0f * fabsf(s[nt][i] * p.to_cap));
+                            s[nt][i] = copysignf(__fdividef(1.0f - e, 1.0f + e), s[nt][i]) * p.cap_log2;
+                        }
                 }
             };
             // The scores of block j + 1 are computed in the same straight-line code as the softmax and P V of
@@ -501,10 +512,10 @@ bool make_page_map(CUtensorMap* out, const void* k_base, long long kv_stride_byt
     return true;
 }
 
-template <int D, int STAGES, int CTAS, bool BIAS>
+template <int D, int STAGES, int CTAS, int KIND>
 int launch_config(const CUtensorMap& mkv, const BulkParams& p, int bytes, int max_ctas, cudaStream_t stream) {
     static int configured = 0;
-    auto kernel = attention_decode_bulk_kernel<D, STAGES, CTAS, BIAS>;
+    auto kernel = attention_decode_bulk_kernel<D, STAGES, CTAS, KIND>;
     if (configured < bytes) {
         if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) != cudaSuccess)
             return fail(PH_ERR_LAUNCH, "attention_decode_bulk: cannot reserve %d bytes of shared memory", bytes);
@@ -524,30 +535,32 @@ int launch_config(const CUtensorMap& mkv, const BulkParams& p, int bytes, int ma
 // Two CTAs per SM with three stages each when that fits the SM's shared memory, else two stages each, else one
 // CTA with four stages: what counts is warps per SM (the consumers wait on dependent tensor-core instructions)
 // and enough copies in flight.
-template <int D, bool BIAS> int launch_bulk(const CUtensorMap& mkv, const BulkParams& p, int max_ctas, cudaStream_t stream) {
+template <int D, int KIND> int launch_bulk(const CUtensorMap& mkv, const BulkParams& p, int max_ctas, cudaStream_t stream) {
     const int G = p.HQ / p.HKV;
     constexpr int SM_BYTES = 227 * 1024;
     const int b3 = bulk_smem_bytes(D, G, 3), b2 = bulk_smem_bytes(D, G, 2), b4 = bulk_smem_bytes(D, G, 4);
-    if (2 * (b3 + 1024) <= SM_BYTES) return launch_config<D, 3, 2, BIAS>(mkv, p, b3, max_ctas, stream);
-    if (2 * (b2 + 1024) <= SM_BYTES) return launch_config<D, 2, 2, BIAS>(mkv, p, b2, max_ctas, stream);
-    return launch_config<D, 4, 1, BIAS>(mkv, p, b4, max_ctas, stream);
+    if (2 * (b3 + 1024) <= SM_BYTES) return launch_config<D, 3, 2, KIND>(mkv, p, b3, max_ctas, stream);
+    if (2 * (b2 + 1024) <= SM_BYTES) return launch_config<D, 2, 2, KIND>(mkv, p, b2, max_ctas, stream);
+    return launch_config<D, 4, 1, KIND>(mkv, p, b4, max_ctas, stream);
 }
 
 }  // namespace
 
 // num_pages: pages of the pool that k_base / v_base belong to (the copy engine needs the extent it may address).
+// cap (0: none): the scaled score s becomes cap * tanh(s / cap); not beside slopes.
 // sink, slopes: [HQ] float32 or null.  gate: rows of HQ * D bfloat16 logits, gate_stride elements apart, or null.
-PH_EXPORT int ph_attention_decode_bulk_biased(const void* q, const void* k_base, const void* v_base, long long page_stride,
+PH_EXPORT int ph_attention_decode_bulk_capped(const void* q, const void* k_base, const void* v_base, long long page_stride,
                                               int page_size, int num_pages, const int32_t* block_table, int table_stride,
                                               const int32_t* row_list, int n_rows, const int32_t* row_seg,
                                               const int32_t* positions, float* part_o, float* part_ml, void* out, int HQ,
                                               int HKV, int D, int splits, int window, int chunk, float scale, int max_ctas,
                                               int* error_flag, const float* sink, const float* slopes, const void* gate,
-                                              long long gate_stride, cudaStream_t stream) {
+                                              long long gate_stride, float cap, cudaStream_t stream) {
     if (!q || !k_base || !v_base || !block_table || !row_seg || !positions || !out || !error_flag || n_rows < 0 ||
         HQ < 1 || HKV < 1 || HQ % HKV || page_size < 1 || num_pages < 1 || window < 0 || chunk < 0 || splits < 1 ||
         (splits > 1 && (!part_o || !part_ml)))
         return fail(PH_ERR_ARG, "attention_decode_bulk: bad arguments (rows %d, HQ %d, HKV %d, splits %d)", n_rows, HQ, HKV, splits);
+    if (cap < 0.0f || (cap > 0.0f && slopes)) return fail(PH_ERR_UNSUPPORTED, "attention_decode_bulk: a cap beside a distance bias");
     if (D != 64 && D != 128) return fail(PH_ERR_UNSUPPORTED, "attention_decode_bulk: head_dim %d is not 64 or 128", D);
     if (HQ / HKV > 16) return fail(PH_ERR_UNSUPPORTED, "attention_decode_bulk: %d query heads per kv head exceed 16", HQ / HKV);
     if (page_size % 8 || BLOCK_KEYS % page_size)
@@ -575,8 +588,22 @@ PH_EXPORT int ph_attention_decode_bulk_biased(const void* q, const void* k_base,
     p.out = (__nv_bfloat16*)out; p.n_rows = n_rows; p.HQ = HQ; p.HKV = HKV; p.splits = splits; p.window = window; p.chunk = chunk;
     p.scale_log2 = scale * LOG2E; p.error_flag = error_flag; p.sink = sink;
     p.slopes = slopes; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride;
-    if (slopes) return D == 64 ? launch_bulk<64, true>(mkv, p, max_ctas, stream) : launch_bulk<128, true>(mkv, p, max_ctas, stream);
-    return D == 64 ? launch_bulk<64, false>(mkv, p, max_ctas, stream) : launch_bulk<128, false>(mkv, p, max_ctas, stream);
+    p.to_cap = cap > 0.0f ? scale / cap : 0.0f; p.cap_log2 = cap * LOG2E;
+    if (cap > 0.0f) return D == 64 ? launch_bulk<64, 2>(mkv, p, max_ctas, stream) : launch_bulk<128, 2>(mkv, p, max_ctas, stream);
+    if (slopes) return D == 64 ? launch_bulk<64, 1>(mkv, p, max_ctas, stream) : launch_bulk<128, 1>(mkv, p, max_ctas, stream);
+    return D == 64 ? launch_bulk<64, 0>(mkv, p, max_ctas, stream) : launch_bulk<128, 0>(mkv, p, max_ctas, stream);
+}
+
+PH_EXPORT int ph_attention_decode_bulk_biased(const void* q, const void* k_base, const void* v_base, long long page_stride,
+                                              int page_size, int num_pages, const int32_t* block_table, int table_stride,
+                                              const int32_t* row_list, int n_rows, const int32_t* row_seg,
+                                              const int32_t* positions, float* part_o, float* part_ml, void* out, int HQ,
+                                              int HKV, int D, int splits, int window, int chunk, float scale, int max_ctas,
+                                              int* error_flag, const float* sink, const float* slopes, const void* gate,
+                                              long long gate_stride, cudaStream_t stream) {
+    return ph_attention_decode_bulk_capped(q, k_base, v_base, page_stride, page_size, num_pages, block_table, table_stride, row_list, n_rows,
+                                           row_seg, positions, part_o, part_ml, out, HQ, HKV, D, splits, window, chunk, scale, max_ctas,
+                                           error_flag, sink, slopes, gate, gate_stride, 0.0f, stream);
 }
 
 PH_EXPORT int ph_attention_decode_bulk_sink(const void* q, const void* k_base, const void* v_base, long long page_stride,

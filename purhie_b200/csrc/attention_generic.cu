@@ -14,6 +14,7 @@
 // cut into steps or on what else is in the batch.
 // A sink (one float32 number per query head, or none) is one more term exp(sink) in the softmax's denominator: it has no
 // key and no value, is not scaled, and counts once whatever the window holds.
+// A cap (0: none) bends the scaled score s to cap * tanh(s / cap).
 // A distance bias (one slope per query head, or none) takes slope_h * (z - p) off the scaled score of the key at p.  A gate
 // (rows of HQ * DV logits, or none) multiplies the output by sigmoid(gate), element by element.
 // Formulas (reference): src/qwen_ops.cpp:26-51 (scores * scale, max-subtracted softmax, weighted sum of
@@ -36,7 +37,7 @@ __global__ void attention_generic_kernel(const TQ* __restrict__ q, const TKV* __
                                          const int32_t* __restrict__ row_seg, const int32_t* __restrict__ positions,
                                          TO* __restrict__ out, int T, int HQ, int HKV, int D, int window, float scale, int DV, int chunk, int VS,
                                          const float* __restrict__ sink, const float* __restrict__ slopes, const TQ* __restrict__ gate,
-                                         long long gate_stride) {
+                                         long long gate_stride, float cap) {
     __shared__ float qs[WARPS][MAX_D];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -69,6 +70,7 @@ __global__ void attention_generic_kernel(const TQ* __restrict__ q, const TKV* __
             float dot = 0.0f;
             for (int d = 0; d < D; ++d) dot += qs[warp][d] * to_float<TKV>(krow[d]);
             s = dot * scale;
+            if (cap > 0.0f) s = cap * tanhf(s / cap);
             if (slopes) s -= slope * (float)(z - p);
         }
         const float m_new = fmaxf(m, warp_max(s));
@@ -112,14 +114,14 @@ __global__ void attention_generic_kernel(const TQ* __restrict__ q, const TKV* __
 }  // namespace
 
 // sink, slopes: [HQ] float32 or null.  gate: rows of HQ * DV logits in q's dtype, gate_stride elements apart, or null.
-PH_EXPORT int ph_attention_generic_biased(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype,
+PH_EXPORT int ph_attention_generic_capped(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype,
                                           long long page_stride, int page_size, const int32_t* block_table,
                                           int table_stride, const int32_t* row_seg, const int32_t* positions, void* out,
                                           int out_dtype, int T, int HQ, int HKV, int D, int window, float scale, int DV,
                                           int chunk, int v_stride, const float* sink, const float* slopes, const void* gate,
-                                          long long gate_stride, cudaStream_t stream) {
+                                          long long gate_stride, float cap, cudaStream_t stream) {
     if (!q || !k_base || !v_base || !block_table || !row_seg || !positions || !out || T < 0 || HQ < 1 || HKV < 1 ||
-        D < 1 || page_size < 1 || window < 0 || chunk < 0 || !valid_dtype(q_dtype) || !valid_dtype(kv_dtype) ||
+        D < 1 || page_size < 1 || window < 0 || chunk < 0 || cap < 0.0f || !valid_dtype(q_dtype) || !valid_dtype(kv_dtype) ||
         !valid_dtype(out_dtype))
         return fail(PH_ERR_ARG, "attention_generic: bad arguments (T %d, HQ %d, HKV %d, D %d)", T, HQ, HKV, D);
     if (HQ % HKV) return fail(PH_ERR_ARG, "attention_generic: %d query heads are not a multiple of %d kv heads", HQ, HKV);
@@ -132,10 +134,21 @@ PH_EXPORT int ph_attention_generic_biased(const void* q, int q_dtype, const void
 #define LAUNCH(TQ, TKV, TO)                                                                                    \
     attention_generic_kernel<TQ, TKV, TO><<<blocks, WARPS * 32, 0, stream>>>(                                  \
         (const TQ*)q, (const TKV*)k_base, (const TKV*)v_base, page_stride, page_size, block_table, table_stride, \
-        row_seg, positions, (TO*)out, T, HQ, HKV, D, window, scale, DV, chunk, v_stride, sink, slopes, (const TQ*)gate, gate_stride)
+        row_seg, positions, (TO*)out, T, HQ, HKV, D, window, scale, DV, chunk, v_stride, sink, slopes, (const TQ*)gate, gate_stride, cap)
     PH_DISPATCH(q_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, PH_DISPATCH(out_dtype, TO, LAUNCH(TQ, TKV, TO))));
 #undef LAUNCH
     return check_launch("attention_generic");
+}
+
+PH_EXPORT int ph_attention_generic_biased(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype,
+                                          long long page_stride, int page_size, const int32_t* block_table,
+                                          int table_stride, const int32_t* row_seg, const int32_t* positions, void* out,
+                                          int out_dtype, int T, int HQ, int HKV, int D, int window, float scale, int DV,
+                                          int chunk, int v_stride, const float* sink, const float* slopes, const void* gate,
+                                          long long gate_stride, cudaStream_t stream) {
+    return ph_attention_generic_capped(q, q_dtype, k_base, v_base, kv_dtype, page_stride, page_size, block_table, table_stride, row_seg,
+                                       positions, out, out_dtype, T, HQ, HKV, D, window, scale, DV, chunk, v_stride, sink, slopes, gate,
+                                       gate_stride, 0.0f, stream);
 }
 
 PH_EXPORT int ph_attention_generic_sink(const void* q, int q_dtype, const void* k_base, const void* v_base, int kv_dtype,

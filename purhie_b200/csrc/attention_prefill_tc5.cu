@@ -80,6 +80,7 @@ struct Tc5Params {
     float* part_ml;                // [T][HQ][splits][2] the exponent's reference and the sum of each partial
     const float* sink;             // [HQ] float32 or null: exp(sink) joins each head's denominator, once per row
     const float* slopes;           // [HQ] float32 or null: taken off the scores per position of distance
+    float to_cap, cap_log2;        // KIND 2: scale / cap and cap * log2(e)
     const __nv_bfloat16* gate; long long gate_stride;      // rows of HQ * D logits, or null
     const int32_t* dense_base;     // [S] or null: keys and values are dense rows, the request's first one
 };
@@ -203,7 +204,51 @@ __device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, u
         ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
 }
 
-template <bool BIAS>
+// Two float32 products in one instruction.
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("{\n.reg .b64 ra, rb, rd;\n"
+        "mov.b64 ra, {%2, %3};\nmov.b64 rb, {%4, %5};\n"
+        "mul.rn.f32x2 rd, ra, rb;\n"
+        "mov.b64 {%0, %1}, rd;\n}"
+        : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+    return d;
+}
+
+// A row's scores bent by a cap: s <- cap_log2 * tanh(s * to_cap).  Where all of them are small against the cap (the rule: a
+// cap is there for the outliers) tanh is its Taylor polynomial through x^11, whose error below |x| = 0.4 is under 3e-8;
+// else (1 - e) / (1 + e) with e = exp(-2 |x|).
+__device__ __forceinline__ void cap_scores(float2 (&s)[BN / 2], float to_cap, float cap_log2) {
+    float far0 = 0.0f, far1 = 0.0f;
+#pragma unroll
+    for (int j = 0; j < BN / 2; ++j) { far0 = fmaxf(far0, fabsf(s[j].x)); far1 = fmaxf(far1, fabsf(s[j].y)); }
+    const float2 to2 = make_float2(to_cap, to_cap), cap2 = make_float2(cap_log2, cap_log2);
+    if (fmaxf(far0, far1) * to_cap < 0.4f) {
+        const float2 one = make_float2(1.0f, 1.0f), c3 = make_float2(-1.0f / 3.0f, -1.0f / 3.0f), c5 = make_float2(2.0f / 15.0f, 2.0f / 15.0f),
+                     c7 = make_float2(-17.0f / 315.0f, -17.0f / 315.0f), c9 = make_float2(62.0f / 2835.0f, 62.0f / 2835.0f),
+                     c11 = make_float2(-1382.0f / 155925.0f, -1382.0f / 155925.0f);
+#pragma unroll
+        for (int j = 0; j < BN / 2; ++j) {
+            const float2 x = mul2(s[j], to2), xx = mul2(x, x);
+            float2 t = fma2(xx, c11, c9);
+            t = fma2(xx, t, c7);
+            t = fma2(xx, t, c5);
+            t = fma2(xx, t, c3);
+            t = fma2(xx, t, one);
+            s[j] = mul2(mul2(x, cap2), t);
+        }
+    } else {
+        auto bent = [&](float v) {
+            const float e = __expf(-2.0f * fabsf(v * to_cap));
+            return copysignf(__fdividef(1.0f - e, 1.0f + e), v) * cap_log2;
+        };
+#pragma unroll
+        for (int j = 0; j < BN / 2; ++j) s[j] = make_float2(bent(s[j].x), bent(s[j].y));
+    }
+}
+
+// KIND: what happens to a scaled score in front of the softmax: 0 nothing, 1 a distance bias, 2 a cap.
+template <int KIND>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, const Tc5Params p) {
@@ -372,7 +417,8 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
         const int z = z_first + min(r, n_rows - 1);      // rows past the portion repeat the last one; never stored
         const int lo = first_seen(z, p.window, p.chunk);
         const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
-        const float slope = BIAS ? p.slopes[h] * LOG2E : 0.0f;
+        constexpr bool LOG2_SCORES = KIND != 0;          // the block's scores are brought to log2 units first
+        const float slope = KIND == 1 ? p.slopes[h] * LOG2E : 0.0f;
         float m_ref = -INFINITY;                         // the maximum the exponents refer to
         float l = 0.0f;
         bool ok = true;
@@ -391,6 +437,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
 #pragma unroll
                 for (int j = 0; j < BN / 2; ++j) s[j] = make_float2(__uint_as_float(raw[2 * j]), __uint_as_float(raw[2 * j + 1]));
             }
+            if constexpr (KIND == 2) cap_scores(s, p.to_cap, p.cap_log2);
             if (key0 + BN - 1 > z || key0 < lo) {            // only the blocks at the diagonal and at the window's edge
 #pragma unroll
                 for (int j = 0; j < BN / 2; ++j) {
@@ -398,7 +445,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
                     if (key0 + 2 * j + 1 > z || key0 + 2 * j + 1 < lo) s[j].y = -INFINITY;
                 }
             }
-            if constexpr (BIAS) {                            // the scores in log2 units, the distance's share taken off
+            if constexpr (KIND == 1) {                       // the scores in log2 units, the distance's share taken off
                 const float base = slope * (float)(key0 - z);
                 const float2 scale2 = make_float2(p.scale_log2, p.scale_log2), slope2 = make_float2(slope, slope), base2 = make_float2(base, base);
 #pragma unroll
@@ -411,7 +458,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 mx0 = fmaxf(mx0, fmaxf(s[j].x, s[j].y));
                 mx1 = fmaxf(mx1, fmaxf(s[j + 1].x, s[j + 1].y));
             }
-            const float mx = BIAS ? fmaxf(mx0, mx1) : fmaxf(mx0, mx1) * p.scale_log2;       // the scale is positive: the maximum commutes with it
+            const float mx = LOG2_SCORES ? fmaxf(mx0, mx1) : fmaxf(mx0, mx1) * p.scale_log2;       // the scale is positive: the maximum commutes with it
             // move the reference only when the maximum has outgrown it by more than RESCALE_STEP
             float corr = 1.0f;
             if (mx > m_ref + RESCALE_STEP || (m_ref == -INFINITY && mx > -INFINITY)) {
@@ -425,7 +472,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
             uint32_t packed[BN / 2];
 #pragma unroll
             for (int j = 0; j < BN / 2; j += 2) {
-                const float2 a0 = BIAS ? add2(s[j], neg2) : fma2(s[j], scale2, neg2), a1 = BIAS ? add2(s[j + 1], neg2) : fma2(s[j + 1], scale2, neg2);
+                const float2 a0 = LOG2_SCORES ? add2(s[j], neg2) : fma2(s[j], scale2, neg2), a1 = LOG2_SCORES ? add2(s[j + 1], neg2) : fma2(s[j + 1], scale2, neg2);
                 const float2 e0 = make_float2(ex2(a0.x), ex2(a0.y)), e1 = make_float2(ex2(a1.x), ex2(a1.y));
                 sum_a = add2(sum_a, e0);
                 sum_b = add2(sum_b, e1);
@@ -623,12 +670,13 @@ struct KvPlace {
 int launch_tc5(const void* q, long long q_stride, int T, const KvPlace& kv, const int32_t* seg_start, const int32_t* seg_ctx_len,
                const int32_t* tile_seg, const int32_t* tile_first, int n_tiles, void* out, int HQ, int HKV, int head_dim, int window, int chunk,
                float scale, int splits, float* part_o, float* part_ml, int* error_flag, const float* sink, const float* slopes,
-               const void* gate, long long gate_stride, cudaStream_t stream) {
+               const void* gate, long long gate_stride, float cap, cudaStream_t stream) {
     const bool dense = kv.dense_base != nullptr;
     if (!q || !kv.k || !kv.v || !seg_start || !seg_ctx_len || !tile_seg || !tile_first || !out || !error_flag || T < 1 || n_tiles < 0 || HQ < 1 ||
-        HKV < 1 || HQ % HKV || window < 0 || chunk < 0 || !(scale > 0.0f) || q_stride < (long long)HQ * D ||
+        HKV < 1 || HQ % HKV || window < 0 || chunk < 0 || !(scale > 0.0f) || cap < 0.0f || q_stride < (long long)HQ * D ||
         (dense ? kv.rows < 1 || kv.row_width < (long long)HKV * D : !kv.block_table || kv.num_pages < 1))
         return fail(PH_ERR_ARG, "attention_prefill_tc5: bad arguments (tiles %d, HQ %d, HKV %d)", n_tiles, HQ, HKV);
+    if (cap > 0.0f && slopes) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: a cap beside a distance bias");
     if (head_dim != D) return fail(PH_ERR_UNSUPPORTED, "attention_prefill_tc5: head_dim %d is not %d", head_dim, D);
     const int page_size = dense ? BN : kv.page_size;
     if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64)
@@ -662,14 +710,17 @@ int launch_tc5(const void* q, long long q_stride, int T, const KvPlace& kv, cons
     p.HQ = HQ; p.HKV = HKV; p.window = window; p.chunk = chunk; p.scale_log2 = scale * LOG2E; p.error_flag = error_flag;
     p.splits = splits; p.part_o = part_o; p.part_ml = part_ml; p.sink = sink;
     p.slopes = slopes; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride; p.dense_base = kv.dense_base;
+    p.to_cap = cap > 0.0f ? scale / cap : 0.0f; p.cap_log2 = cap * LOG2E;
+    auto kernel = cap > 0.0f ? attention_prefill_tc5_kernel<2> : slopes ? attention_prefill_tc5_kernel<1> : attention_prefill_tc5_kernel<0>;
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(attention_prefill_tc5_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess ||
-            cudaFuncSetAttribute(attention_prefill_tc5_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess)
+        if (cudaFuncSetAttribute(attention_prefill_tc5_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(attention_prefill_tc5_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(attention_prefill_tc5_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess)
             return fail(PH_ERR_LAUNCH, "attention_prefill_tc5: cannot reserve %d bytes of shared memory", SMEM_BYTES);
         configured = true;
     }
-    launch_overlapped(slopes ? attention_prefill_tc5_kernel<true> : attention_prefill_tc5_kernel<false>, dim3(HQ, n_tiles, splits), dim3(THREADS), (size_t)SMEM_BYTES, stream, mq, mk, mv, p);
+    launch_overlapped(kernel, dim3(HQ, n_tiles, splits), dim3(THREADS), (size_t)SMEM_BYTES, stream, mq, mk, mv, p);
     if (splits > 1)
         launch_overlapped(attention_prefill_tc5_combine_kernel, dim3(n_tiles, HQ, BM / 4), dim3(128), 0, stream,
                           (const float*)part_o, (const float*)part_ml, seg_start, tile_seg, tile_first, (__nv_bfloat16*)out, HQ, splits, sink, p.gate, gate_stride);
@@ -682,7 +733,22 @@ int launch_tc5(const void* q, long long q_stride, int T, const KvPlace& kv, cons
 // for few tiles that look far back.  tile_seg / tile_first: the step's prompt portions cut into tiles
 // of 128 rows (segment, first row of the tile within the portion).  num_pages: pages of the pool that k_base /
 // v_base belong to.
+// cap (0: none): the scaled score s becomes cap * tanh(s / cap); not beside slopes.
 // sink, slopes: [HQ] float32 or null.  gate: rows of HQ * 128 bfloat16 logits, gate_stride elements apart, or null.
+PH_EXPORT int ph_attention_prefill_tc5_capped(const void* q, int T, const void* k_base, const void* v_base, long long page_stride,
+                                              int page_size, int num_pages, const int32_t* block_table, int table_stride,
+                                              const int32_t* seg_start, const int32_t* seg_ctx_len, const int32_t* tile_seg,
+                                              const int32_t* tile_first, int n_tiles, void* out, int HQ, int HKV, int head_dim,
+                                              int window, int chunk, float scale, int splits, float* part_o, float* part_ml,
+                                              int* error_flag, const float* sink, const float* slopes, const void* gate,
+                                              long long gate_stride, float cap, cudaStream_t stream) {
+    KvPlace kv = {};
+    kv.k = k_base; kv.v = v_base; kv.page_stride = page_stride; kv.page_size = page_size; kv.num_pages = num_pages;
+    kv.block_table = block_table; kv.table_stride = table_stride;
+    return launch_tc5(q, (long long)HQ * D, T, kv, seg_start, seg_ctx_len, tile_seg, tile_first, n_tiles, out, HQ, HKV, head_dim, window, chunk,
+                      scale, splits, part_o, part_ml, error_flag, sink, slopes, gate, gate_stride, cap, stream);
+}
+
 PH_EXPORT int ph_attention_prefill_tc5_biased(const void* q, int T, const void* k_base, const void* v_base, long long page_stride,
                                               int page_size, int num_pages, const int32_t* block_table, int table_stride,
                                               const int32_t* seg_start, const int32_t* seg_ctx_len, const int32_t* tile_seg,
@@ -690,11 +756,9 @@ PH_EXPORT int ph_attention_prefill_tc5_biased(const void* q, int T, const void* 
                                               int window, int chunk, float scale, int splits, float* part_o, float* part_ml,
                                               int* error_flag, const float* sink, const float* slopes, const void* gate,
                                               long long gate_stride, cudaStream_t stream) {
-    KvPlace kv = {};
-    kv.k = k_base; kv.v = v_base; kv.page_stride = page_stride; kv.page_size = page_size; kv.num_pages = num_pages;
-    kv.block_table = block_table; kv.table_stride = table_stride;
-    return launch_tc5(q, (long long)HQ * D, T, kv, seg_start, seg_ctx_len, tile_seg, tile_first, n_tiles, out, HQ, HKV, head_dim, window, chunk,
-                      scale, splits, part_o, part_ml, error_flag, sink, slopes, gate, gate_stride, stream);
+    return ph_attention_prefill_tc5_capped(q, T, k_base, v_base, page_stride, page_size, num_pages, block_table, table_stride, seg_start,
+                                           seg_ctx_len, tile_seg, tile_first, n_tiles, out, HQ, HKV, head_dim, window, chunk, scale, splits,
+                                           part_o, part_ml, error_flag, sink, slopes, gate, gate_stride, 0.0f, stream);
 }
 
 // The same over keys and values that lie densely: k and v [rows, H * 128] bfloat16, row_width elements from a token's row to
@@ -709,7 +773,7 @@ PH_EXPORT int ph_attention_prefill_tc5_dense(const void* q, long long q_stride, 
     kv.k = k; kv.v = v; kv.dense_base = dense_base; kv.row_width = row_width; kv.rows = rows;
     if (!dense_base) return fail(PH_ERR_ARG, "attention_prefill_tc5_dense: no first rows");
     return launch_tc5(q, q_stride, T, kv, seg_start, seg_ctx_len, tile_seg, tile_first, n_tiles, out, H, H, head_dim, 0, 0, scale, splits, part_o,
-                      part_ml, error_flag, nullptr, nullptr, gate, gate_stride, stream);
+                      part_ml, error_flag, nullptr, nullptr, gate, gate_stride, 0.0f, stream);
 }
 
 PH_EXPORT int ph_attention_prefill_tc5_sink(const void* q, int T, const void* k_base, const void* v_base, long long page_stride,

@@ -153,22 +153,76 @@ __global__ void attention_talking_kernel(const TQ* __restrict__ q, const TKV* __
     }
 }
 
-// One block per token.  The row holds [q (QW) | k (KW) | v (VW, or nothing when the keys are the values) | ...].
+// What may happen to a row beside the norms: a factor per token that the norm in front left out (sumsq, see RowScale), a bias
+// [QW + KW + VW] added behind it, a rotation of the first n_rot dimensions of every q and k head (table [max_pos, n_rot]:
+// cosines, then sines, one per pair; halves or neighbours), and the gate's logits behind v, gate_width of them, added up and
+// stored in q's dtype (gate_out).  All optional.
+struct RowExtras {
+    const float* bias = nullptr;
+    const float* table = nullptr; int n_rot = 0, max_pos = 0, interleaved = 0;
+    const int32_t* positions = nullptr;
+    const float* sumsq = nullptr; int chunks = 0, width = 0; float eps = 0.0f;
+    void* gate_out = nullptr; int gate_width = 0;
+};
+__device__ __forceinline__ float row_factor(const RowExtras& x, int t) {
+    if (!x.sumsq) return 1.0f;
+    float s = 0.0f;
+    for (int k = 0; k < x.chunks; ++k) s += x.sumsq[(size_t)t * x.chunks + k];
+    return rsqrtf(s / (float)x.width + x.eps);
+}
+// Element d of a head at `head` (raw values, with factor inv and the weights at w, or none), rotated.
+__device__ __forceinline__ float rotated(const RowExtras& x, const float* turn, const float* head, const float* w, float inv, int d) {
+    auto at = [&](int e) { return w ? head[e] * inv * w[e] : head[e]; };
+    const float own = at(d);
+    if (!turn || d >= x.n_rot) return own;
+    const int half = x.n_rot / 2;
+    int pair; bool second; float other;
+    if (x.interleaved) { pair = d >> 1; second = d & 1; other = at(d ^ 1); }
+    else { second = d >= half; pair = second ? d - half : d; other = at(second ? d - half : d + half); }
+    const float c = turn[pair], s = turn[half + pair];
+    return second ? __fmaf_rn(other, s, __fmul_rn(own, c)) : __fmaf_rn(own, c, -__fmul_rn(other, s));
+}
+__device__ __forceinline__ const float* turn_of(const RowExtras& x, int t) {
+    if (!x.table) return nullptr;
+    int pos = x.positions[t];
+    pos = pos < 0 ? 0 : pos < x.max_pos ? pos : x.max_pos - 1;
+    return x.table + (size_t)pos * x.n_rot;
+}
+
+// The gate's logits, at `first` in the row: added up, scaled and stored.
+template <typename TI, typename TQ>
+__device__ __forceinline__ void finish_gate(const RowExtras& x, const TI* src, int splits, long long split_stride, int first, float factor, int t) {
+    if (!x.gate_out) return;
+    TQ* to = static_cast<TQ*>(x.gate_out) + (size_t)t * x.gate_width;
+    for (int i = threadIdx.x; i < x.gate_width; i += blockDim.x) {
+        float v = 0.0f;
+        for (int s = 0; s < splits; ++s) v += to_float<TI>(src[(size_t)s * split_stride + first + i]);
+        to[i] = from_float<TQ>(v * factor);
+    }
+}
+
+// One block per token.  The row holds [q (QW) | k (KW) | v (VW, or nothing when the keys are the values) | gate | ...].
 template <typename TI, typename TQ, typename TKV>
 __global__ void joint_norm_kv_write_kernel(const TI* __restrict__ rows, int splits, long long split_stride, long long row_width,
                                            const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                                            const int32_t* __restrict__ slot_mapping, TQ* __restrict__ q_out, TKV* __restrict__ k_base,
                                            TKV* __restrict__ v_base, long long page_stride, int page_size, int HQ, int HKV, int D, int DV,
-                                           int v_from_row) {
+                                           int v_from_row, const RowExtras x) {
     extern __shared__ float buf[];             // [QW + KW]
     __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
     const int t = blockIdx.x;
     const int QW = HQ * D, KW = HKV * D;
     const TI* src = rows + (size_t)t * row_width;
+    const float factor = row_factor(x, t);
+    const float* turn = turn_of(x, t);
     float sq = 0.0f, sk = 0.0f;
     for (int i = threadIdx.x; i < QW + KW; i += blockDim.x) {
         float v = 0.0f;
         for (int s = 0; s < splits; ++s) v += to_float<TI>(src[(size_t)s * split_stride + i]);
+        v *= factor;
+        if (x.bias) v += x.bias[i];
         buf[i] = v;
         if (i < QW) sq += v * v; else sk += v * v;
     }
@@ -176,7 +230,11 @@ __global__ void joint_norm_kv_write_kernel(const TI* __restrict__ rows, int spli
     const float ik = k_w ? rsqrtf(block_sum_any(sk, scratch) / (float)KW + eps) : 1.0f;
     __syncthreads();
     TQ* qo = q_out + (size_t)t * QW;
-    for (int i = threadIdx.x; i < QW; i += blockDim.x) qo[i] = from_float<TQ>(q_w ? buf[i] * iq * q_w[i] : buf[i]);
+    for (int i = threadIdx.x; i < QW; i += blockDim.x) {
+        const int h0 = i / D * D;
+        qo[i] = from_float<TQ>(rotated(x, turn, buf + h0, q_w ? q_w + h0 : nullptr, iq, i - h0));
+    }
+    finish_gate<TI, TQ>(x, src, splits, split_stride, QW + KW + (v_from_row ? HKV * DV : 0), factor, t);
     if (!slot_mapping) return;
     const int slot = slot_mapping[t];
     if (slot < 0) return;
@@ -185,7 +243,8 @@ __global__ void joint_norm_kv_write_kernel(const TI* __restrict__ rows, int spli
     for (int i = threadIdx.x; i < KW; i += blockDim.x) {
         const int h = i / D, d = i % D;
         const float raw = buf[QW + i];
-        k_base[page_at + ((size_t)h * page_size + off) * D + d] = from_float<TKV>(k_w ? raw * ik * k_w[i] : raw);
+        k_base[page_at + ((size_t)h * page_size + off) * D + d] =
+            from_float<TKV>(rotated(x, turn, buf + QW + h * D, k_w ? k_w + h * D : nullptr, ik, d));
         if (!v_from_row) v_base[page_at + ((size_t)h * page_size + off) * DV + d] = from_float<TKV>(raw);
     }
     if (v_from_row) {
@@ -193,6 +252,8 @@ __global__ void joint_norm_kv_write_kernel(const TI* __restrict__ rows, int spli
             const int h = i / DV, d = i % DV;
             float v = 0.0f;
             for (int s = 0; s < splits; ++s) v += to_float<TI>(src[(size_t)s * split_stride + QW + KW + i]);
+            v *= factor;
+            if (x.bias) v += x.bias[QW + KW + i];
             v_base[page_at + ((size_t)h * page_size + off) * DV + d] = from_float<TKV>(v);
         }
     }
@@ -206,12 +267,16 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
                                                const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                                                const int32_t* __restrict__ slot_mapping, TQ* __restrict__ q_out, TKV* __restrict__ k_base,
                                                TKV* __restrict__ v_base, long long page_stride, int page_size, int HQ, int HKV, int D, int DV,
-                                               int v_from_row) {
+                                               int v_from_row, const RowExtras x) {
     extern __shared__ float buf[];             // [QW + KW]
     __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
     const int t = blockIdx.x;
     const int QW = HQ * D, KW = HKV * D;
     const TI* src = rows + (size_t)t * row_width;
+    const float factor = row_factor(x, t);
+    const float* turn = turn_of(x, t);
     float sq = 0.0f, sk = 0.0f;
     for (int i = threadIdx.x * 8; i < QW + KW; i += blockDim.x * 8) {
         float v[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
@@ -221,6 +286,8 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
 #pragma unroll
             for (int j = 0; j < 8; ++j) v[j] += u[j];
         }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { v[j] *= factor; if (x.bias) v[j] += x.bias[i + j]; }
         float ss = 0.0f;
 #pragma unroll
         for (int j = 0; j < 8; ++j) { buf[i + j] = v[j]; ss += v[j] * v[j]; }
@@ -233,9 +300,10 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
     for (int i = threadIdx.x * 8; i < QW; i += blockDim.x * 8) {
         float v[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) v[j] = q_w ? buf[i + j] * iq * q_w[i + j] : buf[i + j];
+        for (int j = 0; j < 8; ++j) v[j] = rotated(x, turn, buf + i / D * D, q_w ? q_w + i / D * D : nullptr, iq, i % D + j);
         store8(qo + i, v);
     }
+    finish_gate<TI, TQ>(x, src, splits, split_stride, QW + KW + (v_from_row ? HKV * DV : 0), factor, t);
     if (!slot_mapping) return;
     const int slot = slot_mapping[t];
     if (slot < 0) return;
@@ -245,7 +313,7 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
         const int h = i / D, d = i % D;
         float raw[8], v[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) { raw[j] = buf[QW + i + j]; v[j] = k_w ? raw[j] * ik * k_w[i + j] : raw[j]; }
+        for (int j = 0; j < 8; ++j) { raw[j] = buf[QW + i + j]; v[j] = rotated(x, turn, buf + QW + h * D, k_w ? k_w + h * D : nullptr, ik, d + j); }
         store8(k_base + page_at + ((size_t)h * page_size + off) * D + d, v);
         if (!v_from_row) store8(v_base + page_at + ((size_t)h * page_size + off) * DV + d, raw);
     }
@@ -259,6 +327,8 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
 #pragma unroll
                 for (int j = 0; j < 8; ++j) v[j] += u[j];
             }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) { v[j] *= factor; if (x.bias) v[j] += x.bias[QW + KW + i + j]; }
             store8(v_base + page_at + ((size_t)h * page_size + off) * DV + d, v);
         }
     }
@@ -306,15 +376,15 @@ PH_EXPORT int ph_attention_talking(const void* q, int q_dtype, const void* k_bas
 
 // rows: [splits][T][row_width] in rows_dtype.  q_w [HQ * D] and k_w [HKV * D] float32 or null.  slot_mapping null: no
 // cache write (q only).  v_from_row 0: the values are the keys as projected; 1: the row's third part [HKV * DV].
-PH_EXPORT int ph_joint_norm_kv_write(const void* rows, int rows_dtype, int splits, long long split_stride, long long row_width,
+static int joint_norm(const void* rows, int rows_dtype, int splits, long long split_stride, long long row_width,
                                      const float* q_w, const float* k_w, float eps, const int32_t* slot_mapping, void* q_out, int q_dtype,
                                      void* k_base, void* v_base, int kv_dtype, long long page_stride, int page_size, int T, int HQ,
-                                     int HKV, int D, int DV, int v_from_row, cudaStream_t stream) {
+                                     int HKV, int D, int DV, int v_from_row, const RowExtras& x, cudaStream_t stream) {
     if (!rows || !q_out || T < 0 || HQ < 1 || HKV < 1 || D < 1 || DV < 1 || splits < 1 || page_size < 1 || !valid_dtype(rows_dtype) ||
         !valid_dtype(q_dtype) || !valid_dtype(kv_dtype) || (slot_mapping && (!k_base || !v_base)))
         return fail(PH_ERR_ARG, "joint_norm_kv_write: bad arguments (T %d, HQ %d, HKV %d, D %d)", T, HQ, HKV, D);
     if (!v_from_row && DV != D) return fail(PH_ERR_ARG, "joint_norm_kv_write: values that are the keys are as wide as the keys (%d, not %d)", D, DV);
-    const long long need = (long long)(HQ + HKV) * D + (v_from_row ? (long long)HKV * DV : 0);
+    const long long need = (long long)(HQ + HKV) * D + (v_from_row ? (long long)HKV * DV : 0) + (x.gate_out ? x.gate_width : 0);
     if (row_width < need) return fail(PH_ERR_ARG, "joint_norm_kv_write: rows of %lld elements hold no %lld", row_width, need);
     const size_t smem = (size_t)(HQ + HKV) * D * sizeof(float);
     if (smem > 200 * 1024) return fail(PH_ERR_UNSUPPORTED, "joint_norm_kv_write: rows of %d elements do not fit shared memory", (HQ + HKV) * D);
@@ -328,8 +398,8 @@ PH_EXPORT int ph_joint_norm_kv_write(const void* rows, int rows_dtype, int split
     do {                                                                                                                           \
         auto kern = joint_norm_kv_write_vec_kernel<TI, TQ, TKV>;                                                                   \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                  \
-        kern<<<T, vthreads, smem, stream>>>((const TI*)rows, splits, split_stride, row_width, q_w, k_w, eps, slot_mapping, (TQ*)q_out, \
-                                            (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, D, DV, v_from_row);       \
+        launch_overlapped(kern, dim3(T), dim3(vthreads), smem, stream, (const TI*)rows, splits, split_stride, row_width, q_w, k_w, eps, slot_mapping, (TQ*)q_out, \
+                                            (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, D, DV, v_from_row, x);       \
     } while (0)
         PH_DISPATCH(rows_dtype, TI, PH_DISPATCH(q_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, LAUNCH_VEC(TI, TQ, TKV))));
 #undef LAUNCH_VEC
@@ -339,10 +409,37 @@ PH_EXPORT int ph_joint_norm_kv_write(const void* rows, int rows_dtype, int split
     do {                                                                                                                           \
         auto kern = joint_norm_kv_write_kernel<TI, TQ, TKV>;                                                                       \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                  \
-        kern<<<T, threads, smem, stream>>>((const TI*)rows, splits, split_stride, row_width, q_w, k_w, eps, slot_mapping, (TQ*)q_out, \
-                                           (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, D, DV, v_from_row);        \
+        launch_overlapped(kern, dim3(T), dim3(threads), smem, stream, (const TI*)rows, splits, split_stride, row_width, q_w, k_w, eps, slot_mapping, (TQ*)q_out, \
+                                           (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, D, DV, v_from_row, x);        \
     } while (0)
     PH_DISPATCH(rows_dtype, TI, PH_DISPATCH(q_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, LAUNCH(TI, TQ, TKV))));
 #undef LAUNCH
     return check_launch("joint_norm_kv_write");
+}
+
+PH_EXPORT int ph_joint_norm_kv_write(const void* rows, int rows_dtype, int splits, long long split_stride, long long row_width,
+                                     const float* q_w, const float* k_w, float eps, const int32_t* slot_mapping, void* q_out, int q_dtype,
+                                     void* k_base, void* v_base, int kv_dtype, long long page_stride, int page_size, int T, int HQ,
+                                     int HKV, int D, int DV, int v_from_row, cudaStream_t stream) {
+    return joint_norm(rows, rows_dtype, splits, split_stride, row_width, q_w, k_w, eps, slot_mapping, q_out, q_dtype, k_base, v_base, kv_dtype,
+                      page_stride, page_size, T, HQ, HKV, D, DV, v_from_row, RowExtras(), stream);
+}
+
+// The same for rows [q | k | v | (gate)] with a bias, a rotation, a row's missing factor and the gate's logits (RowExtras says
+// what each is; null: without it).
+PH_EXPORT int ph_joint_norm_rope_kv_write(const void* rows, int rows_dtype, int splits, long long split_stride, long long row_width,
+                                          const float* q_w, const float* k_w, float eps, const int32_t* slot_mapping, void* q_out, int q_dtype,
+                                          void* k_base, void* v_base, int kv_dtype, long long page_stride, int page_size, int T, int HQ,
+                                          int HKV, int D, int DV, const float* bias, const float* cos_sin, int n_rot, int max_pos,
+                                          const int32_t* positions, int interleaved, const float* row_sumsq, int row_chunks, int row_dim,
+                                          float row_eps, void* gate_out, int gate_width, cudaStream_t stream) {
+    if (cos_sin && (n_rot < 2 || n_rot % 2 || n_rot > D || max_pos < 1 || !positions))
+        return fail(PH_ERR_ARG, "joint_norm_rope_kv_write: %d of %d dimensions cannot be rotated", n_rot, D);
+    if ((row_sumsq && (row_chunks < 1 || row_dim < 1)) || (gate_out && gate_width < 1))
+        return fail(PH_ERR_ARG, "joint_norm_rope_kv_write: bad arguments");
+    RowExtras x;
+    x.bias = bias; x.table = cos_sin; x.n_rot = n_rot; x.max_pos = max_pos; x.interleaved = interleaved; x.positions = positions;
+    x.sumsq = row_sumsq; x.chunks = row_chunks; x.width = row_dim; x.eps = row_eps; x.gate_out = gate_out; x.gate_width = gate_width;
+    return joint_norm(rows, rows_dtype, splits, split_stride, row_width, q_w, k_w, eps, slot_mapping, q_out, q_dtype, k_base, v_base, kv_dtype,
+                      page_stride, page_size, T, HQ, HKV, D, DV, 1, x, stream);
 }

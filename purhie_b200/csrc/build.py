@@ -31,8 +31,8 @@ LIBRARIES: Dict[str, dict] = {
         "sources": ["elementwise.cu", "qk_norm_rope.cu", "attention_generic.cu", "gemm_simple.cu", "sampling.cu",
                     "random_fill.cu", "layernorm.cu", "gated.cu", "mamba.cu", "moe.cu", "linear_attention.cu", "dyntanh.cu",
                     "latent_attention.cu", "attention_talking.cu", "attention_talking_mma.cu", "min_gru.cu", "lanes.cu",
-                    "ssd.cu", "core_lib.cu"],
-        "deps": ["../weights/random.h", "attention_mma.cuh"],
+                    "ssd.cu", "delta_rule.cu", "core_lib.cu"],
+        "deps": ["../weights/random.h", "attention_mma.cuh", "delta_rule.cuh"],
         "flags": [],
         "link": [],
     },
@@ -60,8 +60,8 @@ LIBRARIES: Dict[str, dict] = {
                     "../parts/registry.cpp", "../parts/linear.cpp", "../parts/norm.cpp", "../parts/rotary.cpp",
                     "../parts/attention.cpp", "../parts/feed_forward.cpp", "../parts/routed.cpp", "../parts/mamba.cpp",
                     "../parts/linear_attention.cpp", "../parts/latent_attention.cpp", "../parts/embedding.cpp", "../parts/block.cpp",
-                    "../parts/min_gru.cpp", "../config/bozosun.cpp", "../config/sizizen.cpp", "../config/zerusun.cpp", "../config/vokepel.cpp",
-                    "../config/noditar.cpp",
+                    "../parts/min_gru.cpp", "../parts/delta_rule.cpp", "../config/bozosun.cpp", "../config/sizizen.cpp", "../config/zerusun.cpp", "../config/vokepel.cpp",
+                    "../config/noditar.cpp", "../config/defapel.cpp",
                     "../parts/model.cpp", "../cache/cache.cpp", "../sampling/sampler.cpp", "../engine/engine.cpp",
                     "../engine/scheduler.cpp", "../api/capi.cpp", "../api/capi_generate.cpp", "../api/test_hooks.cpp",
                     "../api/test_hooks_host.cpp", "../api/test_hooks_parts.cpp"],

@@ -4,6 +4,7 @@
 //   kind 1 (clamped swish):  g' = min(g, limit), u' = clamp(u, -limit, limit), out = g' * sigmoid(alpha * g') * (u' + shift)
 //   kind 2 (gelu, tanh form): out = 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * u
 // and activations of one argument over plain rows (unary_act): kind 0 silu, kind 1 the square of relu.
+// A factor per row (glu_scaled) multiplies gate and up before the activation: row r's is factor[index[r]].
 // The sums over split-K partial results and the activation are float32.
 #include "common.cuh"
 
@@ -21,7 +22,8 @@ __device__ __forceinline__ float gated(float g, float u, int kind, float alpha, 
 
 template <typename TI, typename TO>
 __global__ void glu_kernel(const TI* __restrict__ gu, int splits, long long split_stride, TO* __restrict__ out, int FF,
-                           long long total, int kind, float alpha, float limit, float shift) {
+                           long long total, int kind, float alpha, float limit, float shift, const float* __restrict__ factor,
+                           const int32_t* __restrict__ index) {
     pdl_launch_dependents();
     pdl_wait();
     const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -32,13 +34,15 @@ __global__ void glu_kernel(const TI* __restrict__ gu, int splits, long long spli
         gv += to_float<TI>(g[(size_t)s * split_stride]);
         uv += to_float<TI>(g[(size_t)s * split_stride + 1]);
     }
+    if (factor) { const float f = factor[index[idx / FF]]; gv *= f; uv *= f; }
     out[idx] = from_float<TO>(gated(gv, uv, kind, alpha, limit, shift));
 }
 
 // four outputs per thread: eight inputs in one or two 16-byte loads per split
 template <typename TI, typename TO>
 __global__ void glu_vec_kernel(const TI* __restrict__ gu, int splits, long long split_stride, TO* __restrict__ out, long long total4,
-                               int kind, float alpha, float limit, float shift) {
+                               int FF, int kind, float alpha, float limit, float shift, const float* __restrict__ factor,
+                               const int32_t* __restrict__ index) {
     pdl_launch_dependents();
     pdl_wait();
     const long long q = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -49,6 +53,11 @@ __global__ void glu_vec_kernel(const TI* __restrict__ gu, int splits, long long 
         load8(gu + (size_t)s * split_stride + q * 8, v);
 #pragma unroll
         for (int i = 0; i < 8; ++i) acc[i] += v[i];
+    }
+    if (factor) {                                          // four outputs never straddle a row: FF is a multiple of 4
+        const float f = factor[index[q * 4 / FF]];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) acc[i] *= f;
     }
     float o[4];
 #pragma unroll
@@ -111,9 +120,11 @@ PH_EXPORT int ph_unary_act(const void* in, int in_dtype, int splits, long long s
     return check_launch("unary_act");
 }
 
-PH_EXPORT int ph_glu(const void* gate_up, int in_dtype, int splits, long long split_stride, void* out, int out_dtype, int T,
-                     int FF, int kind, float alpha, float limit, float shift, cudaStream_t stream) {
-    if (!gate_up || !out || T < 0 || FF < 1 || splits < 1 || kind < 0 || kind > 2 || !valid_dtype(in_dtype) || !valid_dtype(out_dtype))
+// factor null: no factor; else row r of the T rows is multiplied by factor[index[r]] in front of the activation.
+PH_EXPORT int ph_glu_scaled(const void* gate_up, int in_dtype, int splits, long long split_stride, void* out, int out_dtype, int T,
+                            int FF, int kind, float alpha, float limit, float shift, const float* factor, const int32_t* index,
+                            cudaStream_t stream) {
+    if (!gate_up || !out || T < 0 || (factor && !index) || FF < 1 || splits < 1 || kind < 0 || kind > 2 || !valid_dtype(in_dtype) || !valid_dtype(out_dtype))
         return fail(PH_ERR_ARG, "glu: bad arguments (T %d, FF %d, kind %d)", T, FF, kind);
     const long long total = (long long)T * FF;
     if (total == 0) return PH_OK;
@@ -121,12 +132,17 @@ PH_EXPORT int ph_glu(const void* gate_up, int in_dtype, int splits, long long sp
         const long long total4 = total / 4;
         PH_DISPATCH(in_dtype, TI, PH_DISPATCH(out_dtype, TO,
             launch_overlapped(glu_vec_kernel<TI, TO>, dim3((unsigned)((total4 + 255) / 256)), dim3(256), 0, stream, (const TI*)gate_up,
-                              splits, split_stride, (TO*)out, total4, kind, alpha, limit, shift)));
+                              splits, split_stride, (TO*)out, total4, FF, kind, alpha, limit, shift, factor, index)));
         return check_launch("glu");
     }
     const unsigned blocks = (unsigned)((total + 255) / 256);
     PH_DISPATCH(in_dtype, TI, PH_DISPATCH(out_dtype, TO,
         launch_overlapped(glu_kernel<TI, TO>, dim3(blocks), dim3(256), 0, stream, (const TI*)gate_up, splits, split_stride,
-                          (TO*)out, FF, total, kind, alpha, limit, shift)));
+                          (TO*)out, FF, total, kind, alpha, limit, shift, factor, index)));
     return check_launch("glu");
+}
+
+PH_EXPORT int ph_glu(const void* gate_up, int in_dtype, int splits, long long split_stride, void* out, int out_dtype, int T,
+                     int FF, int kind, float alpha, float limit, float shift, cudaStream_t stream) {
+    return ph_glu_scaled(gate_up, in_dtype, splits, split_stride, out, out_dtype, T, FF, kind, alpha, limit, shift, nullptr, nullptr, stream);
 }

@@ -18,7 +18,7 @@
 //                  the tile holds.  This is weight streaming: its bound is the bytes of the chosen experts.
 //   route_combine  out[t] = base[t] (optional: float32 partial sums of a part that runs for every token, times base_scale[t]
 //                  where a factor per token is given) + the sum over the
-//                  token's choices, in the order of the choices, of weight * y[position of (t, j)].
+//                  token's choices, in the order of the choices, of weight * y[position of (t, j)] (weight null: of y alone).
 #include "common.cuh"
 
 namespace {
@@ -379,7 +379,7 @@ __global__ void route_combine_kernel(const TY* __restrict__ y, const int32_t* __
         if (base_scale) acc *= base_scale[t];
     }
     for (int j = 0; j < top; ++j)
-        acc += weight[(size_t)t * top + j] * to_float<TY>(y[(size_t)position[(size_t)t * top + j] * E_out + c]);
+        acc += (weight ? weight[(size_t)t * top + j] : 1.0f) * to_float<TY>(y[(size_t)position[(size_t)t * top + j] * E_out + c]);
     out[idx] = acc;
 }
 
@@ -401,7 +401,7 @@ __global__ void route_combine_vec_kernel(const float* __restrict__ y, const int3
         }
     if (base && base_scale) { const float f = base_scale[t]; acc.x *= f; acc.y *= f; acc.z *= f; acc.w *= f; }
     for (int j = 0; j < top; ++j) {
-        const float wj = weight[(size_t)t * top + j];
+        const float wj = weight ? weight[(size_t)t * top + j] : 1.0f;
         const float4 v = *reinterpret_cast<const float4*>(y + (size_t)position[(size_t)t * top + j] * E_out + c);
         acc.x += wj * v.x; acc.y += wj * v.y; acc.z += wj * v.z; acc.w += wj * v.w;
     }
@@ -508,7 +508,7 @@ PH_EXPORT int ph_gemv_grouped(const void* x, int x_dtype, const int32_t* pair_at
 PH_EXPORT int ph_route_combine(const void* y, int y_dtype, const int32_t* position, const float* weight, int T, int top, int E_out,
                                float* out, const float* base, int base_splits, long long base_stride, const float* base_scale,
                                cudaStream_t stream) {
-    if (!y || !position || !weight || !out || T < 0 || top < 1 || E_out < 1 || !valid_dtype(y_dtype) || (base && base_splits < 1))
+    if (!y || !position || !out || T < 0 || top < 1 || E_out < 1 || !valid_dtype(y_dtype) || (base && base_splits < 1))
         return fail(PH_ERR_ARG, "route_combine: bad arguments (T %d, top %d, width %d)", T, top, E_out);
     const long long total = (long long)T * E_out;
     if (total == 0) return PH_OK;

@@ -160,6 +160,7 @@ const CoreKernels& core_kernels() {
     bind(h, "core", "ph_add_layernorm", g_core.add_layernorm);
     bind(h, "core", "ph_embed_gather_scaled", g_core.embed_gather_scaled);
     bind(h, "core", "ph_glu", g_core.glu);
+    bind(h, "core", "ph_glu_scaled", g_core.glu_scaled);
     bind(h, "core", "ph_unary_act", g_core.unary_act);
     bind(h, "core", "ph_decayed_scan", g_core.decayed_scan);
     bind(h, "core", "ph_rms_pair_mean", g_core.rms_pair_mean);
@@ -191,9 +192,14 @@ const CoreKernels& core_kernels() {
     bind(h, "core", "ph_attention_talking_mma_supports", g_core.attention_talking_mma_supports);
     bind(h, "core", "ph_attention_talking_mma_ctas_per_sm", g_core.attention_talking_mma_ctas_per_sm);
     bind(h, "core", "ph_joint_norm_kv_write", g_core.joint_norm_kv_write);
+    bind(h, "core", "ph_joint_norm_rope_kv_write", g_core.joint_norm_rope_kv_write);
+    bind(h, "core", "ph_attention_generic_capped", g_core.attention_generic_capped);
     bind(h, "core", "ph_min_gru_scan", g_core.min_gru_scan);
     bind(h, "core", "ph_pair_sum", g_core.pair_sum);
     bind(h, "core", "ph_add_scaled_rmsnorm", g_core.add_scaled_rmsnorm);
+    bind(h, "core", "ph_delta_prepare", g_core.delta_prepare);
+    bind(h, "core", "ph_delta_scan", g_core.delta_scan);
+    bind(h, "core", "ph_head_norm_gate", g_core.head_norm_gate);
     bind(h, "core", "ph_scale_softcap", g_core.scale_softcap);
     bind(h, "core", "ph_core_last_error", g_core.last_error);
     g_core_ok = true;
@@ -209,8 +215,8 @@ const FlashKernels& flash_kernels() {
     bind(h, "flash", "ph_attention_decode", g_flash.decode);
     bind(h, "flash", "ph_attention_decode_bulk", g_flash.decode_bulk);
     bind(h, "flash", "ph_attention_prefill_tc5", g_flash.prefill_tc5);
-    bind(h, "flash", "ph_attention_decode_bulk_biased", g_flash.decode_bulk_biased);
-    bind(h, "flash", "ph_attention_prefill_tc5_biased", g_flash.prefill_tc5_biased);
+    bind(h, "flash", "ph_attention_decode_bulk_capped", g_flash.decode_bulk_capped);
+    bind(h, "flash", "ph_attention_prefill_tc5_capped", g_flash.prefill_tc5_capped);
     bind(h, "flash", "ph_attention_prefill_tc5_dense", g_flash.prefill_tc5_dense);
     bind(h, "flash", "ph_flash_last_error", g_flash.last_error);
     g_flash_ok = true;

@@ -118,6 +118,8 @@ struct CoreKernels {
     int (*embed_gather_scaled)(const void*, int, const int32_t*, float*, int, int, int, float, cudaStream_t);
     // gated activations by kind (0 silu, 1 clamped swish with alpha, limit, shift)
     int (*glu)(const void*, int, int, long long, void*, int, int, int, int, float, float, float, cudaStream_t);
+    int (*glu_scaled)(const void*, int, int, long long, void*, int, int, int, int, float, float, float, const float*, const int32_t*,
+                      cudaStream_t);     // with a factor per row in front of the activation
     // activations of one argument over plain rows (0 silu, 1 the square of relu)
     int (*unary_act)(const void*, int, int, long long, void*, int, long long, int, cudaStream_t);
     // gated linear attention: the decayed matrix state token by token with the head norm and gate behind it; two mixers'
@@ -168,6 +170,10 @@ struct CoreKernels {
     int (*attention_generic_biased)(const void*, int, const void*, const void*, int, long long, int, const int32_t*, int,
                                     const int32_t*, const int32_t*, void*, int, int, int, int, int, int, float, int, int, int, const float*,
                                     const float*, const void*, long long, cudaStream_t);
+    // (the same with a cap on the scores)
+    int (*attention_generic_capped)(const void*, int, const void*, const void*, int, long long, int, const int32_t*, int,
+                                    const int32_t*, const int32_t*, void*, int, int, int, int, int, int, float, int, int, int, const float*,
+                                    const float*, const void*, long long, float, cudaStream_t);
     int (*attention_talking)(const void*, int, const void*, const void*, int, long long, int, const int32_t*, int, const int32_t*,
                              const int32_t*, void*, int, int, int, int, int, int, int, int, float, float, const float*, const float*,
                              const float*, const float*, const void*, int, long long, cudaStream_t);
@@ -179,6 +185,10 @@ struct CoreKernels {
     int (*attention_talking_mma_ctas_per_sm)(int, int, int, int);
     int (*joint_norm_kv_write)(const void*, int, int, long long, long long, const float*, const float*, float, const int32_t*, void*, int,
                                void*, void*, int, long long, int, int, int, int, int, int, int, cudaStream_t);
+    // the same with a bias, a rotation, a row's missing factor and the gate's logits
+    int (*joint_norm_rope_kv_write)(const void*, int, int, long long, long long, const float*, const float*, float, const int32_t*, void*, int,
+                                    void*, void*, int, long long, int, int, int, int, int, int, const float*, const float*, int, int,
+                                    const int32_t*, int, const float*, int, int, float, void*, int, cudaStream_t);
     // a minimal gated recurrent unit over the rows of each request; the weighted sum of two mixers' outputs
     int (*min_gru_scan)(const void*, int, int, long long, long long, const float*, const float*, float*, const int32_t*, const int32_t*,
                         int, int, int, const int32_t*, int, const int32_t*, float*, void*, int, cudaStream_t);
@@ -196,6 +206,15 @@ struct CoreKernels {
                      const int32_t*, const int32_t*, int, int, int, int, int, int, int, int, float*, cudaStream_t);
     int (*ssd_chunk_supports)(int, int, int);
     int (*gate_rms)(const float*, const void*, int, long long, const float*, float, void*, int, int, int, int, cudaStream_t);
+    // the gated delta rule: convolutions, unit norms and step sizes in front of it; the recurrence token by token; the head norm
+    // with its gate behind it
+    int (*delta_prepare)(const void*, int, int, long long, long long, const float*, int, const float*, long long, long long, const int32_t*,
+                         const int32_t*, const int32_t*, int, int, int, int, int, float, float*, int, float*, int, const float*, const float*,
+                         float*, int, int, void*, int, int, void*, int, cudaStream_t);
+    int (*delta_scan)(const float*, const float*, const float*, const float*, long long, const float*, const float*, const void*, int, int,
+                      long long, long long, float*, long long, long long, const int32_t*, const int32_t*, int, int, int, int, int, int, int, int,
+                      float*, cudaStream_t);
+    int (*head_norm_gate)(const float*, const float*, float, const void*, int, long long, int, void*, int, int, int, int, cudaStream_t);
     // logits scaled and softly capped in place
     int (*scale_softcap)(float*, long long, float, float, cudaStream_t);
     const char* (*last_error)(void);
@@ -211,13 +230,14 @@ struct FlashKernels {
     int (*prefill_tc5)(const void*, int, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*,
                        const int32_t*, const int32_t*, const int32_t*, int, void*, int, int, int, int, int, float, int, float*,
                        float*, int*, cudaStream_t);
-    // the two kernels above with a sink in the softmax's denominator, a distance bias and an output gate, each optional
-    int (*decode_bulk_biased)(const void*, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*, int,
+    // the two kernels above with a sink in the softmax's denominator, a distance bias, an output gate and a cap on the scores,
+    // each optional (a bias and a cap exclude each other)
+    int (*decode_bulk_capped)(const void*, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*, int,
                               const int32_t*, const int32_t*, float*, float*, void*, int, int, int, int, int, int, float, int, int*,
-                              const float*, const float*, const void*, long long, cudaStream_t);
-    int (*prefill_tc5_biased)(const void*, int, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*,
+                              const float*, const float*, const void*, long long, float, cudaStream_t);
+    int (*prefill_tc5_capped)(const void*, int, const void*, const void*, long long, int, int, const int32_t*, int, const int32_t*,
                               const int32_t*, const int32_t*, const int32_t*, int, void*, int, int, int, int, int, float, int, float*,
-                              float*, int*, const float*, const float*, const void*, long long, cudaStream_t);
+                              float*, int*, const float*, const float*, const void*, long long, float, cudaStream_t);
     // the prompt kernel over dense keys and values, a row per token with the heads side by side
     int (*prefill_tc5_dense)(const void*, long long, int, const void*, const void*, long long, int, const int32_t*, const int32_t*,
                              const int32_t*, const int32_t*, const int32_t*, int, void*, int, int, float, int, float*, float*, int*, const void*,

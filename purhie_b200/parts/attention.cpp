@@ -16,7 +16,9 @@
 // the softmax's denominator as exp(sink), without a key or a value; "sink_value": the same with one constant for all
 // heads); norms of q and k without a weight ("qk_norm_weight": false); a distance bias ("distance_slopes": one number per
 // query head, taken off the scaled score times the distance); an output gate (names.gate_proj: the heads side by side
-// times sigmoid(Wg x), element by element, before Wo).
+// times sigmoid(Wg x), element by element, before Wo); a cap on the scores ("softcap": the scaled score s becomes
+// softcap * tanh(s / softcap), in front of the softmax); one RMS norm over all heads of q, and one over all heads of k, in
+// place of a norm per head ("qk_norm_over": "heads", the default, or "row": q_norm and k_norm then have a weight per element).
 //
 // K and V are written to pages before attention runs, and attention reads everything, the current step's keys
 // included, from pages: a whole prompt, a portion and a decoded token are one algorithm per kernel.
@@ -128,7 +130,7 @@ void add_tiles(StepPlan& plan, int rows, const std::string& name, bool single_ro
 // params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim (null: head_dim), qk_norm_eps (null: no q/k norm),
 // bias, position (a PartSpec as {kind, params}, or null), window (null: all positions), chunk (null: no block mask),
 // scale (null: 1/sqrt(head_dim)), value_mix (null | "first" | "blend"),
-// qk_norm_weight (default true), distance_slopes (null, or a list of num_heads numbers), sink_value (null: none),
+// qk_norm_weight (default true), qk_norm_over ("heads" | "row"), softcap (null: none), distance_slopes (null, or a list of num_heads numbers), sink_value (null: none),
 // names{q_proj, k_proj, v_proj, o_proj, q_norm, k_norm, q_bias, k_bias, v_bias, value_mix_factor, sink, gate_proj}.
 class Attention : public Mixer {
 public:
@@ -149,6 +151,15 @@ public:
         eps_ = has_norm_ ? eps->as_double() : 0.0;
         has_bias_ = p.get_bool("bias", false);
         norm_weight_ = p.get_bool("qk_norm_weight", true);
+        const std::string over = p.get_string("qk_norm_over", "heads");
+        if (over != "heads" && over != "row") throw ConfigError("attention: qk_norm_over is 'heads' or 'row', got '" + over + "'");
+        row_norm_ = has_norm_ && over == "row";
+        if (row_norm_ && (!norm_weight_ || value_mix_)) throw ConfigError("attention: a norm over the row has weights and mixes no values");
+        if (const Json* cap = p.find("softcap"))
+            if (!cap->is_null()) {
+                softcap_ = cap->as_double();
+                if (!(softcap_ > 0.0)) throw ConfigError("attention: softcap must be positive");
+            }
         has_sink_ = names_.count("sink") != 0;
         if (const Json* sv = p.find("sink_value"))
             if (!sv->is_null()) {
@@ -161,6 +172,7 @@ public:
                 if (!ds->is_array() || (int)ds->size() != heads_) throw ConfigError("attention: distance_slopes must list one number per query head");
                 for (const Json& v : ds->items()) slopes_host_.push_back((float)v.as_double());
             }
+        if (softcap_ > 0.0 && !slopes_host_.empty()) throw ConfigError("attention: a cap beside a distance bias is not supported");
         has_gate_ = names_.count("gate_proj") != 0;
         window_ = (int)p.get_int("window", 0);
         chunk_ = (int)p.get_int("chunk", 0);
@@ -184,7 +196,7 @@ public:
         v_width_ = (int64_t)kv_heads_ * value_dim_;
         o_width_ = (int64_t)heads_ * value_dim_;
         g_width_ = has_gate_ ? o_width_ : 0;
-        if (has_gate_ && has_bias_) throw ConfigError("attention: biases beside an output gate are not supported");
+        if (has_gate_ && has_bias_ && !row_norm_) throw ConfigError("attention: biases beside an output gate need a norm over the row");
     }
 
     // ---- weights ----------------------------------------------------------------------------------------------
@@ -197,8 +209,8 @@ public:
         if (has_sink_ && !constant_sink_) s.push_back({name_of("sink"), {heads_}, Role::Vector, Init::Normal});
         if (has_gate_) s.push_back({name_of("gate_proj"), {g_width_, hidden_}, Role::Matrix, Init::Normal});
         if (has_norm_ && norm_weight_) {
-            s.push_back({name_of("q_norm"), {head_dim_}, Role::Vector, Init::Scale});
-            s.push_back({name_of("k_norm"), {head_dim_}, Role::Vector, Init::Scale});
+            s.push_back({name_of("q_norm"), {row_norm_ ? q_width_ : head_dim_}, Role::Vector, Init::Scale});
+            s.push_back({name_of("k_norm"), {row_norm_ ? kv_width_ : head_dim_}, Role::Vector, Init::Scale});
         }
         if (has_bias_) {
             s.push_back({name_of("q_bias"), {q_width_}, Role::Vector, Init::Normal});
@@ -292,8 +304,8 @@ public:
     // ---- cache and step metadata ------------------------------------------------------------------------------
     CacheNeed cache_need() const override { return CacheNeed::pages(kv_heads_, head_dim_, window_, value_dim_, chunk_); }
 
-    // a sink, a distance bias or a gate inside the attention kernel
-    bool extended() const { return has_sink_ || has_gate_ || !slopes_host_.empty(); }
+    // a sink, a distance bias, a cap or a gate inside the attention kernel
+    bool extended() const { return has_sink_ || has_gate_ || softcap_ > 0.0 || !slopes_host_.empty(); }
 
     // which in bfloat16 runs on the tensor-core kernel that knows them (a tile of 16 rows, all heads)
     bool use_tile_kernel() const {
@@ -333,7 +345,7 @@ public:
         const Linear& proj = cache.writable ? qkv_proj_ : q_only_proj_;
         // rows without their factor (RowScale): the product's epilogue applies it where it can, else the kernel behind it
         const bool scale_in_product = ctx.row_scale.defined() && proj.applies_row_scale(T, dt, false, true);
-        if (!cache.writable && (value_mix_ || has_gate_)) throw Error(kInvalidState, "a layer that mixes values or gates its heads writes a cache of its own");
+        if (!cache.writable && (value_mix_ || has_gate_ || row_norm_)) throw Error(kInvalidState, "a layer that mixes values, norms whole rows or gates its heads writes a cache of its own");
         Addend qkv = proj(x, ctx, "qkv", dt, T, true, false, nullptr, scale_in_product ? &ctx.row_scale : nullptr);
         // the values of the first mixing layer, per token of the step: written by that layer, read by the later ones
         float* v_first = value_mix_ ? ws.get("attention.v_first", {T, v_width_}, DType::F32).as<float>() : nullptr;
@@ -362,7 +374,15 @@ public:
             const double row = (double)(q_width_ + (int64_t)kv_heads_written * (head_dim_ + value_dim_) + (gate_rows.defined() ? g_width_ : 0));
             LaunchProfile::get().note_cost((double)T * row * (qkv.splits * dtype_size(qkv.tensor.dtype) + dtype_size(dt)), 0.0);
         }
-        if (has_gate_)
+        if (row_norm_)
+            QE_LAUNCH(core, core.joint_norm_rope_kv_write(
+                qkv.tensor.data, qkv.tensor.code(), qkv.splits, (long long)T * product_width, product_width, q_norm_.as<float>(), k_norm_.as<float>(),
+                (float)eps_, g.slot_mapping, q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype, cache.page_stride, cache.page_size, T,
+                heads_, kv_heads_, head_dim_, value_dim_, bias_.defined() ? bias_.as<float>() : nullptr,
+                table_.defined() ? table_.as<float>() : nullptr, position_ ? position_->n_rot() : 0, table_.defined() ? (int)table_.shape[0] : 0,
+                positions, position_ && position_->interleaved() ? 1 : 0, later.sumsq, later.chunks, later.width, later.eps, gate_rows.data,
+                (int)g_width_, ctx.stream));
+        else if (has_gate_)
             QE_LAUNCH(core, core.qk_norm_rope_gate_kv_write(
                 qkv.tensor.data, qkv.tensor.code(), qkv.splits, (long long)T * product_width, nullptr, has_norm_ ? q_norm_.as<float>() : nullptr,
                 has_norm_ ? k_norm_.as<float>() : nullptr, (float)eps_, table_.defined() ? table_.as<float>() : nullptr,
@@ -398,7 +418,7 @@ public:
                                            2.0 * seen * heads_ * (head_dim_ + value_dim_));
         }
         const StepArray t16 = ctx.array("attention.tiles16.seg"), t16f = ctx.array("attention.tiles16.first");
-        // a sink, a bias and a gate ride in the tcgen05 prompt kernel and the TMA decode kernel only: pages they take, and no
+        // a sink, a bias, a cap and a gate ride in the tcgen05 prompt kernel and the TMA decode kernel only: pages they take, and no
         // other choice by option
         const bool pages_ok = (cache.page_size == 8 || cache.page_size == 16 || cache.page_size == 32 || cache.page_size == 64) && cache.num_pages > 0;
         const bool extras_ok = !extended() || (pages_ok && ctx.option("prefill_kernel") != "mma_sync" && ctx.option("decode_kernel") != "cp_async" &&
@@ -419,13 +439,13 @@ public:
             }
             QE_LAUNCH(core, core.attention_talking_mma(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, g.block_table,
                                                        g.table_width, ctx.seg_start, ctx.seg_ctx_len, t16.data, t16f.data, t16.count, out.data,
-                                                       heads_, kv_heads_, head_dim_, value_dim_, window_, 0, (float)scale_, 0.0f, slopes(),
+                                                       heads_, kv_heads_, head_dim_, value_dim_, window_, 0, (float)scale_, (float)softcap_, slopes(),
                                                        nullptr, nullptr, sink(), gate, gate_stride, splits, T, part_o, part_ml, ctx.stream));
         } else if (extended()) {
-            QE_LAUNCH(core, core.attention_generic_biased(q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype, cache.page_stride,
+            QE_LAUNCH(core, core.attention_generic_capped(q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype, cache.page_stride,
                                                           cache.page_size, g.block_table, g.table_width, ctx.row_seg, abs_positions, out.data,
                                                           out.code(), T, heads_, kv_heads_, head_dim_, window_, (float)scale_, value_dim_, chunk_, 0,
-                                                          sink(), slopes(), gate, gate_stride, ctx.stream));
+                                                          sink(), slopes(), gate, gate_stride, (float)softcap_, ctx.stream));
         } else {
             QE_LAUNCH(core, core.attention_generic(q.data, q.code(), cache.k_base, cache.v_base, (int)cache.kv_dtype, cache.page_stride,
                                                    cache.page_size, g.block_table, g.table_width, ctx.row_seg, abs_positions, out.data,
@@ -454,17 +474,17 @@ private:
                 part_ml = ws.get("attn_tile_part_ml", {ctx.T, heads_, splits, 2}, DType::F32).as<float>();
             }
             if (extended())
-                QE_LAUNCH(f, f.prefill_tc5_biased(q.data, ctx.T, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages,
+                QE_LAUNCH(f, f.prefill_tc5_capped(q.data, ctx.T, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages,
                                                 g.block_table, g.table_width, ctx.seg_start, ctx.seg_ctx_len, t128.data, t128f.data, t128.count,
                                                 out.data, heads_, kv_heads_, head_dim_, window_, chunk_, (float)scale_, splits, part_o, part_ml,
-                                                ctx.attention_error, sink(), slopes(), gate, gate_stride, ctx.stream));
+                                                ctx.attention_error, sink(), slopes(), gate, gate_stride, (float)softcap_, ctx.stream));
             else
                 QE_LAUNCH(f, f.prefill_tc5(q.data, ctx.T, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages,
                                            g.block_table, g.table_width, ctx.seg_start, ctx.seg_ctx_len, t128.data, t128f.data, t128.count,
                                            out.data, heads_, kv_heads_, head_dim_, window_, chunk_, (float)scale_, splits, part_o, part_ml,
                                            ctx.attention_error, ctx.stream));
         } else if (t64.count) {
-            if (extended()) throw Error(kInvalidState, "attention: the tiled prompt kernel knows no sink, bias or gate");
+            if (extended()) throw Error(kInvalidState, "attention: the tiled prompt kernel knows no sink, bias, cap or gate");
             QE_LAUNCH(f, f.prefill(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, g.block_table, g.table_width,
                                    ctx.seg_start, ctx.seg_ctx_len, t64.data, t64f.data, t64.count, out.data, heads_, kv_heads_,
                                    head_dim_, window_, chunk_, (float)scale_, ctx.stream));
@@ -483,16 +503,16 @@ private:
             part_ml = ws.get("attn_part_ml", {n, heads_, splits, 2}, DType::F32).as<float>();
         }
         if (bulk && extended())
-            QE_LAUNCH(f, f.decode_bulk_biased(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages, g.block_table,
+            QE_LAUNCH(f, f.decode_bulk_capped(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages, g.block_table,
                                             g.table_width, ctx.decode_rows, n, ctx.row_seg, positions, part_o, part_ml, out.data, heads_,
                                             kv_heads_, head_dim_, splits, window_, chunk_, (float)scale_, 0, ctx.attention_error,
-                                            sink(), slopes(), gate, gate_stride, ctx.stream));
+                                            sink(), slopes(), gate, gate_stride, (float)softcap_, ctx.stream));
         else if (bulk)
             QE_LAUNCH(f, f.decode_bulk(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, cache.num_pages, g.block_table,
                                        g.table_width, ctx.decode_rows, n, ctx.row_seg, positions, part_o, part_ml, out.data, heads_,
                                        kv_heads_, head_dim_, splits, window_, chunk_, (float)scale_, 0, ctx.attention_error, ctx.stream));
         else if (extended())
-            throw Error(kInvalidState, "attention: the cp.async decode kernel knows no sink, bias or gate");
+            throw Error(kInvalidState, "attention: the cp.async decode kernel knows no sink, bias, cap or gate");
         else
             QE_LAUNCH(f, f.decode(q.data, cache.k_base, cache.v_base, cache.page_stride, cache.page_size, g.block_table, g.table_width,
                                   ctx.decode_rows, n, ctx.row_seg, positions, part_o, part_ml, out.data, heads_, kv_heads_, head_dim_,
@@ -504,8 +524,8 @@ private:
 
     int64_t hidden_, q_width_, kv_width_, v_width_, o_width_, g_width_;
     int heads_, kv_heads_, head_dim_, value_dim_, window_, chunk_ = 0, value_mix_ = 0;
-    bool has_norm_, norm_weight_ = true, has_bias_, has_sink_ = false, constant_sink_ = false, has_gate_ = false;
-    double eps_, scale_, sink_value_ = 0.0;
+    bool has_norm_, norm_weight_ = true, has_bias_, has_sink_ = false, constant_sink_ = false, has_gate_ = false, row_norm_ = false;
+    double eps_, scale_, softcap_ = 0.0, sink_value_ = 0.0;
     std::vector<float> slopes_host_;
     std::string gemm_, attention_;
     std::shared_ptr<PositionEncoding> position_;

@@ -318,6 +318,7 @@ void register_routed_parts();
 void register_state_space_parts();
 void register_linear_attention_parts();
 void register_recurrent_parts();
+void register_delta_parts();
 void register_latent_attention_parts();
 void register_position_parts();
 void register_mixer_parts();
@@ -337,6 +338,7 @@ void register_builtin_parts() {
     register_state_space_parts();
     register_linear_attention_parts();
     register_recurrent_parts();
+    register_delta_parts();
     register_latent_attention_parts();
     register_arrangement("sandwich_norm", [](const LayerSpec& layer, BuildContext& build) {
         return std::unique_ptr<Arrangement>(new SandwichNormBlock(layer, build));

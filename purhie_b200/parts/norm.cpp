@@ -2,7 +2,7 @@
 // itself, each with the residual add folded in.
 //
 // y = v * rsqrt(mean(v^2) + eps) * w, v = x + pending addend; the weight multiplies after normalising (plain w,
-// not 1 + w).  Reference: src/gpu_ops.hip:24-56 (add + norm in one kernel), src/qwen_ops.cpp:8-13.
+// not 1 + w, unless the part is told that the weight is stored around zero).  Reference: src/gpu_ops.hip:24-56 (add + norm in one kernel), src/qwen_ops.cpp:8-13.
 #include "parts.h"
 
 namespace qe {
@@ -94,14 +94,30 @@ Tensor Norm::forward_lanes(ResidualStream& stream, StepContext& ctx, const float
     return forward(read, ctx, rows, n_rows);
 }
 
-// params: size, eps, names{weight}.
+// params: size, eps, weight_offset (default 0: added to the stored weight; 1 for weights stored around zero), names{weight}.
 class RMSNorm : public Norm {
 public:
-    RMSNorm(const Json& p, BuildContext& b) : Norm(p, b), size_(p.at("size").as_int()), eps_(p.at("eps").as_double()) {
+    RMSNorm(const Json& p, BuildContext& b)
+        : Norm(p, b), size_(p.at("size").as_int()), eps_(p.at("eps").as_double()), offset_(p.get_double("weight_offset", 0.0)) {
         if (size_ < 1 || !(eps_ > 0)) throw ConfigError("rmsnorm: size must be positive and eps > 0");
     }
-    std::vector<TensorSpec> tensor_specs() const override { return {{name_of("weight"), {size_}, Role::Vector, Init::Scale}}; }
-    void bind(WeightSource& src) override { weight_ = src.fetch(name_of("weight")); }
+    std::vector<TensorSpec> tensor_specs() const override {
+        return {{name_of("weight"), {size_}, Role::Vector, offset_ == 0.0 ? Init::Scale : Init::Normal}};
+    }
+    void bind(WeightSource& src) override {
+        weight_ = src.fetch(name_of("weight"));
+        if (offset_ == 0.0) return;
+        // the factor itself, once, in float32: every kernel of this norm multiplies by what it is given
+        std::vector<float> host((size_t)size_);
+        QE_CUDA(cudaMemcpyAsync(host.data(), weight_.data, host.size() * sizeof(float), cudaMemcpyDeviceToHost, src.stream()));
+        QE_CUDA(cudaStreamSynchronize(src.stream()));
+        for (float& v : host) v += (float)offset_;
+        Tensor shifted = src.arena().alloc(DType::F32, {size_});
+        QE_CUDA(cudaMemcpyAsync(shifted.data, host.data(), host.size() * sizeof(float), cudaMemcpyHostToDevice, src.stream()));
+        QE_CUDA(cudaStreamSynchronize(src.stream()));
+        src.release(weight_);
+        weight_ = shifted;
+    }
 
     Tensor forward(ResidualStream& stream, StepContext& ctx, const int32_t* rows, int n_rows) override {
         const int n = rows ? n_rows : ctx.T;
@@ -169,7 +185,7 @@ public:
 
 private:
     int64_t size_;
-    double eps_;
+    double eps_, offset_ = 0.0;
     Tensor weight_;
 };
 

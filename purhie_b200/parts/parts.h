@@ -464,7 +464,7 @@ template <typename T> std::shared_ptr<T> make_part_as(const std::string& family,
 }
 
 // Registers the parts this library brings (rmsnorm, layernorm, none, dyntanh, rope_neox, attention, talking_attention,
-// latent_attention, mamba1, mamba2, gated_linear_attention, lightning_attention, min_gru, side_by_side, swiglu, mlp, routed_glu, embedding, lm_head,
+// latent_attention, mamba1, mamba2, gated_linear_attention, lightning_attention, delta_rule, min_gru, side_by_side, swiglu, mlp, routed_glu, embedding, lm_head,
 // pre_norm, sandwich_norm, parallel, reinject, hyper_connection).
 QE_API void register_builtin_parts();
 

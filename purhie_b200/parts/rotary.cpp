@@ -11,6 +11,9 @@
 // theta); with lo = max(floor(pair(fast)), 0), hi = min(ceil(pair(slow)), n_rot - 1) and ramp_i = clamp((i - lo) /
 // max(hi - lo, 0.001), 0, 1), pair i turns with f_i / factor * ramp_i + f_i * (1 - ramp_i) (fast pairs keep their
 // frequency, slow ones are stretched by the factor), and every cosine and sine is multiplied by 0.1 ln(factor) + 1.
+// Scaling by wavelength ("scaling": {"kind": "wavelength", factor, low, high, original}): a pair of frequency f makes
+// t = original f / (2 pi) turns over `original` positions; it keeps f when t > high, turns with f / factor when t < low, and
+// in between with ((1 - s) / factor + s) f, s = (t - low) / (high - low).  Cosines and sines are not stretched.
 #include <algorithm>
 #include <cmath>
 
@@ -19,7 +22,8 @@
 namespace qe {
 
 // params: theta, n_rot, max_position; optional pairing ("half" | "interleaved"), freq_factors [n_rot/2] (each
-// pair's frequency is divided by its factor), scaling (null or {"kind": "yarn", ...} as above), position_column.
+// pair's frequency is divided by its factor), scaling (null, or {"kind": "yarn" | "wavelength", ...} as above),
+// position_column.
 class RotaryTable : public PositionEncoding {
 public:
     RotaryTable(const Json& p, BuildContext& b) : PositionEncoding(p, b) {
@@ -39,10 +43,19 @@ public:
         if (const Json* sc = p.find("scaling")) {
             if (!sc->is_null()) {
                 const std::string kind = sc->get_string("kind", "");
-                if (kind != "yarn") throw ConfigError("rotary: scaling of kind '" + kind + "' is not known (yarn is)");
-                yarn_ = true;
+                if (kind != "yarn" && kind != "wavelength")
+                    throw ConfigError("rotary: scaling of kind '" + kind + "' is not known (yarn, wavelength)");
                 factor_ = sc->at("factor").as_double();
                 original_ = sc->at("original").as_double();
+                if (kind == "wavelength") {
+                    wavelength_ = true;
+                    low_ = sc->at("low").as_double();
+                    high_ = sc->at("high").as_double();
+                    if (!(factor_ > 0) || !(original_ > 0) || !(low_ > 0) || !(high_ >= low_))
+                        throw ConfigError("rotary: wavelength scaling needs positive factor, original and low, and high not below low");
+                    return;
+                }
+                yarn_ = true;
                 fast_ = sc->at("fast").as_double();
                 slow_ = sc->at("slow").as_double();
                 if (!(factor_ > 0) || !(original_ > 0) || !(fast_ > 0) || !(slow_ > 0) || !(theta_ != 1.0))
@@ -64,8 +77,16 @@ public:
             if (!factors_.empty()) inv[i] /= factors_[i];
         }
         double stretch = 1.0;
+        const double kPi = 3.14159265358979323846;
+        if (wavelength_)
+            for (int i = 0; i < half; i++) {
+                const double wave = 2.0 * kPi / inv[i];
+                if (wave < original_ / high_) continue;
+                if (wave > original_ / low_) { inv[i] /= factor_; continue; }
+                const double s = high_ > low_ ? (original_ / wave - low_) / (high_ - low_) : 1.0;
+                inv[i] = (1.0 - s) * inv[i] / factor_ + s * inv[i];
+            }
         if (yarn_) {
-            const double kPi = 3.14159265358979323846;
             auto pair_of = [&](double turns) { return n_rot_ * std::log(original_ / (2.0 * kPi * turns)) / (2.0 * std::log(theta_)); };
             const double lo = std::max(std::floor(pair_of(fast_)), 0.0), hi = std::min(std::ceil(pair_of(slow_)), (double)n_rot_ - 1.0);
             for (int i = 0; i < half; i++) {
@@ -90,8 +111,8 @@ private:
     int n_rot_, column_;
     int64_t max_position_;
     bool interleaved_;
-    bool yarn_ = false;
-    double factor_ = 1.0, original_ = 0.0, fast_ = 0.0, slow_ = 0.0;
+    bool yarn_ = false, wavelength_ = false;
+    double factor_ = 1.0, original_ = 0.0, fast_ = 0.0, slow_ = 0.0, low_ = 0.0, high_ = 0.0;
     std::vector<double> factors_;
     Tensor table_;
 };

@@ -12,6 +12,8 @@
 // s within the `keep` runs whose largest s is highest; the weights are the chosen s over their sum (+ 1e-20), times `scale`.
 // names.shared_gate (a vector [hidden]): the shared part's sum is multiplied by sigmoid(gate . x), one number per token.
 // "gated": false: an expert is Wd act(Wu x) with an activation of one argument ("relu2").
+// "weight_on": "input": the weight multiplies what an expert reads, not what it gives: y = sum of expert(w x).  The experts
+// have no biases, so their first two products are linear in x and the factor enters behind them, in front of the activation.
 // "shared": {kind, params}: a feed-forward that runs for every token and is added to the chosen experts' sum.
 //
 // The (token, choice) pairs are sorted by expert on the device.  Which kernels then multiply:
@@ -33,7 +35,8 @@
 namespace qe {
 
 // params: hidden_size, intermediate_size, experts, top, gated (default true), activation (as the gated feed-forward's;
-// without a gate a name as the plain feed-forward's), scoring (null or as above), shared (null or {kind, params}),
+// without a gate a name as the plain feed-forward's), scoring (null or as above), weight_on ("output", the default,
+// or "input": gated experts only), shared (null or {kind, params}),
 // names{router, router_bias (optional), correction (optional), shared_gate (optional)}, expert_names [{gate_proj, up_proj, down_proj} per
 // expert; without a gate {up_proj, down_proj}].
 class RoutedGLU : public FeedForward {
@@ -68,6 +71,10 @@ public:
                                       std::to_string(experts_) + " experts cannot give " + std::to_string(top_) + " choices");
             }
         }
+        const std::string weight_on = p.get_string("weight_on", "output");
+        if (weight_on != "output" && weight_on != "input") throw ConfigError("routed feed-forward: weight_on is 'output' or 'input', got '" + weight_on + "'");
+        weight_on_input_ = weight_on == "input";
+        if (weight_on_input_ && !gated_) throw ConfigError("routed feed-forward: only gated experts take their weight on the input");
         has_shared_gate_ = names_.count("shared_gate") != 0;
         if (has_correction_ && scoring_ != 1) throw ConfigError("routed feed-forward: a correction of the choice needs sigmoid scoring");
         if (const Json* sh = p.find("shared"))
@@ -211,7 +218,10 @@ public:
             grouped(x, pair_at.as<int32_t>(), top_, gate_up_, gu, up_width_, hidden_);
         }
         if (LaunchProfile::get().on()) LaunchProfile::get().note_cost((double)R * (up_width_ + inter_) * dtype_size(compute_dtype), 0.0);
-        if (gated_)
+        if (weight_on_input_)
+            QE_LAUNCH(k, k.glu_scaled(gu.data, gu.code(), 1, 0, act.data, act.code(), R, (int)inter_, gate_.kind, gate_.alpha, gate_.limit,
+                                      gate_.shift, weight.as<float>(), pair_at.as<int32_t>(), ctx.stream));
+        else if (gated_)
             QE_LAUNCH(k, k.glu(gu.data, gu.code(), 1, 0, act.data, act.code(), R, (int)inter_, gate_.kind, gate_.alpha, gate_.limit,
                                gate_.shift, ctx.stream));
         else
@@ -225,7 +235,7 @@ public:
             grouped(act, nullptr, 1, down_, y, hidden_, inter_);
         }
         Tensor out = ws.get("moe_out", {T, hidden_}, DType::F32);
-        QE_LAUNCH(k, k.route_combine(y.data, y.code(), position.as<int32_t>(), weight.as<float>(), T, top_, (int)hidden_, out.as<float>(),
+        QE_LAUNCH(k, k.route_combine(y.data, y.code(), position.as<int32_t>(), weight_on_input_ ? nullptr : weight.as<float>(), T, top_, (int)hidden_, out.as<float>(),
                                      always.tensor.defined() ? always.tensor.as<float>() : nullptr, always.tensor.defined() ? always.splits : 0,
                                      (long long)T * hidden_, always.tensor.defined() ? shared_scale : nullptr, ctx.stream));
         return Addend(out, 1);
@@ -236,7 +246,7 @@ private:
     int64_t hidden_, inter_;
     int experts_, top_;
     GateSpec gate_;
-    bool gated_ = true, has_bias_ = false, has_correction_ = false;
+    bool gated_ = true, weight_on_input_ = false, has_bias_ = false, has_correction_ = false;
     bool has_shared_gate_ = false;
     int unary_ = 0, scoring_ = 0, groups_ = 1, keep_ = 1;
     float weight_scale_ = 1.0f;
