@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine at the Qwen3-8B shape with random weights, on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--shape 8b|0.6b|32b] [--impl ours|reference]
-    python bench.py --design bozosun|sizizen|zerusun|vokepel|noditar [--size 1k|2k|4k]   (another design beside the Qwen3 layers of equal size; see below)
+    python bench.py --design bozosun|sizizen|zerusun|vokepel|noditar|defapel [--size 1k|2k|4k]   (another design beside the Qwen3 layers of equal size; see below)
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 from 2,048-token prefixes, timed on the
 device (CUDA events on the engine's stream) over exactly K decode steps after W warm-up steps, each step fed its
@@ -188,7 +188,25 @@ def noditar_config(z):
             "max_position": CONTEXT}
 
 
-DESIGN_CONFIGS = {"bozosun": bozosun_config, "sizizen": sizizen_config, "zerusun": zerusun_config, "vokepel": vokepel_config, "noditar": noditar_config}
+def defapel_config(z):
+    """Four layers with routed experts weighted on the input: a delta rule with a decay per channel (half as many heads of 128 x
+    128 state as the attention has, low ranks of 128) in the first and third, attention (heads of 128 rotated over their whole
+    width in interleaved pairs, q and k normed over all heads, capped scores, a window of 1,024 positions, gated heads) side
+    by side with a delta rule with a decay per head (as many value heads, half as many key heads) in the second and fourth."""
+    heads = z["heads"] // 2
+    channel = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128, "gate_rank": 128}
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "mask": {"size": 1024}, "softcap": 30.0,
+            "rot": {"base": 1e6, "dims": z["dim"], "scaling": {"factor": 4.0, "low": 1.0, "high": 8.0, "original": 2048}}, "scale": z["dim"] ** -0.5}
+    right = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
+    both = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 1.1}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    layers = [{"type": "channel_delta", "mixer": channel, "mlp": moe}, {"type": "parallel", "mixer": both, "mlp": moe}] * 2
+    return {"architecture": "Defapel", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "logit_scale": 0.5, "layers": layers,
+            "max_position": CONTEXT}
+
+
+DESIGN_CONFIGS = {"bozosun": bozosun_config, "sizizen": sizizen_config, "zerusun": zerusun_config, "vokepel": vokepel_config, "noditar": noditar_config,
+                  "defapel": defapel_config}
 
 
 def design_bench(args):
@@ -278,7 +296,7 @@ def main():
     ap.add_argument("--page-size", type=int, default=16, help="tokens per cache page (the benchmark's configuration has 16)")
     ap.add_argument("--step-options", default="", metavar="JSON",
                     help="kernel choices of the step, for comparing two forms of it on one box, e.g. '{\"norm_ahead\": \"off\"}'")
-    ap.add_argument("--design", default="", choices=["", "bozosun", "sizizen", "zerusun", "vokepel", "noditar"],
+    ap.add_argument("--design", default="", choices=["", "bozosun", "sizizen", "zerusun", "vokepel", "noditar", "defapel"],
                     help="instead of the headline workload: prefill and decode of this design at real layer sizes beside four "
                          "Qwen3 layers of equal size, with the time and roofline fraction of every kernel class")
     ap.add_argument("--size", default="4k", choices=sorted(DESIGN_SIZES), help="with --design: the layer sizes")

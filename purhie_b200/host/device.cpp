@@ -199,6 +199,10 @@ const CoreKernels& core_kernels() {
     bind(h, "core", "ph_add_scaled_rmsnorm", g_core.add_scaled_rmsnorm);
     bind(h, "core", "ph_delta_prepare", g_core.delta_prepare);
     bind(h, "core", "ph_delta_scan", g_core.delta_scan);
+    bind(h, "core", "ph_delta_chunk", g_core.delta_chunk);
+    bind(h, "core", "ph_delta_chunk_supports", g_core.delta_chunk_supports);
+    bind(h, "core", "ph_delta_chunk_tokens", g_core.delta_chunk_tokens);
+    bind(h, "core", "ph_delta_chunk_scratch_bytes", g_core.delta_chunk_scratch_bytes);
     bind(h, "core", "ph_head_norm_gate", g_core.head_norm_gate);
     bind(h, "core", "ph_scale_softcap", g_core.scale_softcap);
     bind(h, "core", "ph_core_last_error", g_core.last_error);

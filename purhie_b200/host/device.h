@@ -214,6 +214,13 @@ struct CoreKernels {
     int (*delta_scan)(const float*, const float*, const float*, const float*, long long, const float*, const float*, const void*, int, int,
                       long long, long long, float*, long long, long long, const int32_t*, const int32_t*, int, int, int, int, int, int, int, int,
                       float*, cudaStream_t);
+    // (long portions of a bfloat16 model: in chunks on the tensor cores)
+    int (*delta_chunk)(const float*, const float*, const float*, const float*, long long, const float*, const float*, const void*, int, int,
+                       long long, long long, float*, long long, long long, const int32_t*, const int32_t*, int, const int32_t*, int,
+                       const int32_t*, void*, int, int, int, int, int, float*, cudaStream_t);
+    int (*delta_chunk_supports)(int, int);
+    int (*delta_chunk_tokens)(void);
+    long long (*delta_chunk_scratch_bytes)(int, int);
     int (*head_norm_gate)(const float*, const float*, float, const void*, int, long long, int, void*, int, int, int, int, cudaStream_t);
     // logits scaled and softly capped in place
     int (*scale_softcap)(float*, long long, float, float, cudaStream_t);

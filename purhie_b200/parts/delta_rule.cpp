@@ -18,6 +18,9 @@
 // One product gives the rows [q | k | v | (g) | (low) | beta | (z)]: low is decay_down's and gate_down's rows side by side,
 // which one product over a matrix with decay_up and gate_up on its diagonal turns into [z | g].  Columns without a weight
 // (zero rows) bring the widths to multiples of 8.
+//
+// In a bfloat16 model a portion of kChunkRows tokens or more runs in chunks on the tensor cores (csrc/delta_chunk.cu), every
+// other one token by token; the chunk list is the mixer's own step metadata.
 #include <algorithm>
 #include <cmath>
 
@@ -185,6 +188,24 @@ public:
     int preferred_row_multiple() const override { return (in_proj_.fast() || o_proj_.fast()) ? 256 : 0; }
     CacheNeed cache_need() const override { return CacheNeed::state({state_floats()}, DType::F32); }
 
+    // first row and rows of every chunk of the portions that run in chunks, and where each request's chunks start
+    void prepare_step(StepPlan& plan) override {
+        if (compute_dtype != DType::BF16 || plan.has("delta.chunks")) return;
+        const int chunk = core_kernels().delta_chunk_tokens();
+        std::vector<int32_t> items, seg_items = {0};
+        int row = 0;
+        for (int s = 0; s < plan.S; s++) {
+            const int n = plan.q_lens[s];
+            if (n >= kChunkRows)
+                for (int at = 0; at < n; at += chunk) { items.push_back(row + at); items.push_back(std::min(chunk, n - at)); }
+            row += n;
+            seg_items.push_back((int32_t)(items.size() / 2));
+        }
+        if (items.empty()) return;
+        plan.add("delta.chunks", std::move(items));
+        plan.add("delta.seg_chunks", std::move(seg_items));
+    }
+
     Addend forward(const Tensor& x, StepContext& ctx, const CacheView& cache) override {
         if (!cache.state.defined() || cache.state.dtype != DType::F32 || cache.state.shape.size() != 2 || cache.state.shape[1] != state_floats())
             throw Error(kInvalidState, "delta_rule: the cache manager gave no state of this mixer's shape");
@@ -233,11 +254,27 @@ public:
                                                    2.0 * requests * (double)state_floats() * 4.0,
                                                (double)rows * heads_ * dim_ * vdim_ * 7.0);
         };
-        note(ctx.S, T);
-        QE_LAUNCH(k, k.delta_scan(qkv.as<float>(), beta.as<float>(), low_decay_ ? nullptr : log_decay.as<float>(), z, up_width_,
+        // long portions in chunks on the tensor cores, the others token by token (the option "delta": "scan" keeps all of them there)
+        const StepArray chunks = ctx.array("delta.chunks"), seg_chunks = ctx.array("delta.seg_chunks");
+        const int n_chunks = ctx.option("delta") != "scan" && channels_ % 4 == 0 && k.delta_chunk_supports(dim_, vdim_) ? chunks.count / 2 : 0;
+        int n_long = 0, rows_long = 0;
+        if (n_chunks) {
+            for (int n : ctx.q_lens)
+                if (n >= kChunkRows) { n_long++; rows_long += n; }
+            Tensor scratch = ws.get("delta_scratch", {(int64_t)n_chunks * heads_ * k.delta_chunk_scratch_bytes(dim_, vdim_)}, DType::U8);
+            note(n_long, rows_long);
+            QE_LAUNCH(k, k.delta_chunk(qkv.as<float>(), beta.as<float>(), low_decay_ ? nullptr : log_decay.as<float>(), z, up_width_,
+                                       low_decay_ ? dt_bias_.as<float>() : nullptr, rate_.as<float>(), in.tensor.data, in.tensor.code(), in.splits,
+                                       split_stride, width_, state, state_floats(), conv_at(), ctx.seg_start, ctx.seg_slot, ctx.S, chunks.data,
+                                       n_chunks, seg_chunks.data, scratch.data, heads_, kv_heads_, dim_, vdim_, taps_, o.as<float>(), ctx.stream));
+        }
+        if (n_long < ctx.S) {
+            note(ctx.S - n_long, T - rows_long);
+            QE_LAUNCH(k, k.delta_scan(qkv.as<float>(), beta.as<float>(), low_decay_ ? nullptr : log_decay.as<float>(), z, up_width_,
                                   low_decay_ ? dt_bias_.as<float>() : nullptr, rate_.as<float>(), in.tensor.data, in.tensor.code(), in.splits,
                                   split_stride, width_, state, state_floats(), conv_at(), ctx.seg_start, ctx.seg_slot, ctx.S, heads_, kv_heads_,
-                                  dim_, vdim_, taps_, 0, 0, o.as<float>(), ctx.stream));
+                                  dim_, vdim_, taps_, 0, n_long ? kChunkRows - 1 : 0, o.as<float>(), ctx.stream));
+        }
         Tensor y = ws.get("delta_y", {T, v_width_}, dt);
         if (profile.on()) LaunchProfile::get().note_cost((double)T * v_width_ * (4.0 + (gate_code ? 2.0 : 4.0) + es), 0.0);
         QE_LAUNCH(k, k.head_norm_gate(o.as<float>(), norm_.as<float>(), (float)eps_, gate, gate_code, gate_stride, gate_act_, y.data, y.code(), T,
@@ -246,6 +283,7 @@ public:
     }
 
 private:
+    static constexpr int kChunkRows = 32;       // the shortest portion that runs in chunks
     static Tensor upload(WeightSource& src, const std::vector<float>& values) {
         Tensor t = src.arena().alloc(DType::F32, {(int64_t)values.size()});
         QE_CUDA(cudaMemcpyAsync(t.data, values.data(), values.size() * sizeof(float), cudaMemcpyHostToDevice, src.stream()));
