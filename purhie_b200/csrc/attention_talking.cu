@@ -267,7 +267,7 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
                                                const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                                                const int32_t* __restrict__ slot_mapping, TQ* __restrict__ q_out, TKV* __restrict__ k_base,
                                                TKV* __restrict__ v_base, long long page_stride, int page_size, int HQ, int HKV, int D, int DV,
-                                               int v_from_row, const RowExtras x) {
+                                               int v_from_row) {
     extern __shared__ float buf[];             // [QW + KW]
     __shared__ float scratch[32];
     pdl_launch_dependents();
@@ -275,8 +275,6 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
     const int t = blockIdx.x;
     const int QW = HQ * D, KW = HKV * D;
     const TI* src = rows + (size_t)t * row_width;
-    const float factor = row_factor(x, t);
-    const float* turn = turn_of(x, t);
     float sq = 0.0f, sk = 0.0f;
     for (int i = threadIdx.x * 8; i < QW + KW; i += blockDim.x * 8) {
         float v[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
@@ -286,8 +284,6 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
 #pragma unroll
             for (int j = 0; j < 8; ++j) v[j] += u[j];
         }
-#pragma unroll
-        for (int j = 0; j < 8; ++j) { v[j] *= factor; if (x.bias) v[j] += x.bias[i + j]; }
         float ss = 0.0f;
 #pragma unroll
         for (int j = 0; j < 8; ++j) { buf[i + j] = v[j]; ss += v[j] * v[j]; }
@@ -300,10 +296,9 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
     for (int i = threadIdx.x * 8; i < QW; i += blockDim.x * 8) {
         float v[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) v[j] = rotated(x, turn, buf + i / D * D, q_w ? q_w + i / D * D : nullptr, iq, i % D + j);
+        for (int j = 0; j < 8; ++j) v[j] = q_w ? buf[i + j] * iq * q_w[i + j] : buf[i + j];
         store8(qo + i, v);
     }
-    finish_gate<TI, TQ>(x, src, splits, split_stride, QW + KW + (v_from_row ? HKV * DV : 0), factor, t);
     if (!slot_mapping) return;
     const int slot = slot_mapping[t];
     if (slot < 0) return;
@@ -313,7 +308,7 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
         const int h = i / D, d = i % D;
         float raw[8], v[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) { raw[j] = buf[QW + i + j]; v[j] = rotated(x, turn, buf + QW + h * D, k_w ? k_w + h * D : nullptr, ik, d + j); }
+        for (int j = 0; j < 8; ++j) { raw[j] = buf[QW + i + j]; v[j] = k_w ? raw[j] * ik * k_w[i + j] : raw[j]; }
         store8(k_base + page_at + ((size_t)h * page_size + off) * D + d, v);
         if (!v_from_row) store8(v_base + page_at + ((size_t)h * page_size + off) * DV + d, raw);
     }
@@ -327,10 +322,139 @@ __global__ void joint_norm_kv_write_vec_kernel(const TI* __restrict__ rows, int 
 #pragma unroll
                 for (int j = 0; j < 8; ++j) v[j] += u[j];
             }
-#pragma unroll
-            for (int j = 0; j < 8; ++j) { v[j] *= factor; if (x.bias) v[j] += x.bias[QW + KW + i + j]; }
             store8(v_base + page_at + ((size_t)h * page_size + off) * DV + d, v);
         }
+    }
+}
+
+// The form with extras, eight consecutive elements per access in registers.  Two blocks per token: one norms, rotates and
+// stores q and k, the other stores v and the gate.  A thread has IT runs of eight elements; weights are on their way before the
+// kernel in front is done.
+template <typename TI>
+__device__ __forceinline__ void sum8(const TI* src, int splits, long long split_stride, float factor, float* v) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = 0.0f;
+#pragma unroll 4
+    for (int s = 0; s < splits; ++s) {
+        float u[8];
+        load8(src + (size_t)s * split_stride, u);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] += u[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] *= factor;
+}
+template <typename TI, typename TQ, typename TKV, int IT>
+__global__ void joint_norm_rope_vec_kernel(const TI* __restrict__ rows, int splits, long long split_stride, long long row_width,
+                                           const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
+                                           const int32_t* __restrict__ slot_mapping, TQ* __restrict__ q_out, TKV* __restrict__ k_base,
+                                           TKV* __restrict__ v_base, long long page_stride, int page_size, int HQ, int HKV, int D, int DV,
+                                           const RowExtras x) {
+    extern __shared__ float buf[];             // [QW + KW] where pairs are halves of a head apart
+    __shared__ float2 scratch[32];
+    pdl_launch_dependents();
+    const int t = blockIdx.x, QW = HQ * D, KW = HKV * D, VW = HKV * DV, step = blockDim.x * 8;
+    const TI* src = rows + (size_t)t * row_width;
+    if (blockIdx.y == 1) {
+        pdl_wait();
+        const float factor = row_factor(x, t);
+        const int slot = slot_mapping ? slot_mapping[t] : -1;
+        const size_t page_at = slot >= 0 ? (size_t)(slot / page_size) * page_stride : 0;
+        const int off = slot >= 0 ? slot % page_size : 0, all = VW + (x.gate_out ? x.gate_width : 0);
+        for (int i = threadIdx.x * 8; i < all; i += step) {
+            float v[8];
+            sum8(src + QW + KW + i, splits, split_stride, factor, v);
+            if (i >= VW) { store8(static_cast<TQ*>(x.gate_out) + (size_t)t * x.gate_width + (i - VW), v); continue; }
+            if (slot < 0) continue;
+            if (x.bias) {
+                float b[8];
+                load8(x.bias + QW + KW + i, b);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) v[j] += b[j];
+            }
+            const int h = i / DV, d = i - h * DV;
+            store8(v_base + page_at + ((size_t)h * page_size + off) * DV + d, v);
+        }
+        return;
+    }
+    float v[IT][8], w[IT][8];
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+        const int i = threadIdx.x * 8 + it * step;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) w[it][j] = 1.0f;
+        const float* from = i < QW ? (q_w ? q_w + i : nullptr) : i < QW + KW ? (k_w ? k_w + (i - QW) : nullptr) : nullptr;
+        if (from) load8(from, w[it]);
+    }
+    pdl_wait();
+    const float factor = row_factor(x, t);
+    const float* turn = turn_of(x, t);
+    const int slot = slot_mapping ? slot_mapping[t] : -1;
+    float2 ss = make_float2(0.0f, 0.0f);
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+        const int i = threadIdx.x * 8 + it * step;
+        if (i >= QW + KW) continue;
+        sum8(src + i, splits, split_stride, factor, v[it]);
+        if (x.bias) {
+            float b[8];
+            load8(x.bias + i, b);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[it][j] += b[j];
+        }
+        float s8 = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s8 += v[it][j] * v[it][j];
+        if (i < QW) ss.x += s8; else ss.y += s8;
+    }
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    ss.x = warp_sum(ss.x); ss.y = warp_sum(ss.y);
+    if (lane == 0) scratch[warp] = ss;
+    __syncthreads();
+    ss = lane < warps ? scratch[lane] : make_float2(0.0f, 0.0f);
+    const float iq = q_w ? rsqrtf(warp_sum(ss.x) / (float)QW + eps) : 1.0f, ik = k_w ? rsqrtf(warp_sum(ss.y) / (float)KW + eps) : 1.0f;
+    const int half = x.n_rot / 2;
+    const bool apart = turn && !x.interleaved;
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+        const int i = threadIdx.x * 8 + it * step;
+        if (i >= QW + KW) continue;
+        const float inv = i < QW ? iq : ik;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[it][j] = v[it][j] * inv * w[it][j];
+        if (apart) store8(buf + i, v[it]);
+    }
+    if (apart) __syncthreads();
+    const size_t page_at = slot >= 0 ? (size_t)(slot / page_size) * page_stride : 0;
+    const int off = slot >= 0 ? slot % page_size : 0;
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+        const int i = threadIdx.x * 8 + it * step;
+        if (i >= QW + KW) continue;
+        const int head = i / D, d = i - head * D;
+        if (turn && d < x.n_rot) {
+            if (x.interleaved) {
+                const float4 c = load4(turn + d / 2), s = load4(turn + half + d / 2);
+                const float cc[4] = {c.x, c.y, c.z, c.w}, sn[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float a = v[it][2 * e], b = v[it][2 * e + 1];
+                    v[it][2 * e] = __fmaf_rn(a, cc[e], -__fmul_rn(b, sn[e]));
+                    v[it][2 * e + 1] = __fmaf_rn(a, sn[e], __fmul_rn(b, cc[e]));
+                }
+            } else {
+                const bool second = d >= half;
+                float c[8], s[8], other[8];
+                load8(turn + (second ? d - half : d), c);
+                load8(turn + half + (second ? d - half : d), s);
+                load8(buf + (second ? i - half : i + half), other);
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    v[it][j] = second ? __fmaf_rn(other[j], s[j], __fmul_rn(v[it][j], c[j])) : __fmaf_rn(v[it][j], c[j], -__fmul_rn(other[j], s[j]));
+            }
+        }
+        if (i < QW) store8(q_out + (size_t)t * QW + i, v[it]);
+        else if (slot >= 0) store8(k_base + page_at + ((size_t)(head - HQ) * page_size + off) * D + d, v[it]);
     }
 }
 
@@ -392,14 +516,37 @@ static int joint_norm(const void* rows, int rows_dtype, int splits, long long sp
     const int threads = (HQ + HKV) * D >= 2048 ? 512 : 256;
     const bool vec = D % 8 == 0 && DV % 8 == 0 && row_width % 8 == 0 && split_stride % 8 == 0 && page_stride % 8 == 0 &&
                      (((uintptr_t)rows | (uintptr_t)q_out | (uintptr_t)k_base | (uintptr_t)v_base) % 32) == 0;
-    if (vec) {
+    const bool plain = !x.bias && !x.table && !x.sumsq && !x.gate_out;
+    const bool turns_ok = !x.table || (((uintptr_t)x.table & 15) == 0 && (x.interleaved ? x.n_rot % 8 == 0 : x.n_rot % 16 == 0));
+    const int runs = (HQ + HKV) * D / 8;
+    if (vec && !plain && v_from_row && turns_ok && runs <= 4 * 512 && (!x.gate_out || (x.gate_width % 8 == 0 && ((uintptr_t)x.gate_out & 15) == 0)) &&
+        (((uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)x.bias) & 15) == 0) {
+        const int it = runs <= 512 ? 1 : runs <= 1024 ? 2 : 4, threads_x = ((runs + it - 1) / it + 31) / 32 * 32;
+        const size_t bytes = x.table && !x.interleaved ? smem : 0;
+#define LAUNCH_X(TI, TQ, TKV, N)                                                                                                   \
+    do {                                                                                                                           \
+        auto kern = joint_norm_rope_vec_kernel<TI, TQ, TKV, N>;                                                                    \
+        if (bytes > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);                \
+        launch_overlapped(kern, dim3(T, 2), dim3(threads_x), bytes, stream, (const TI*)rows, splits, split_stride, row_width, q_w, k_w, eps, \
+                          slot_mapping, (TQ*)q_out, (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, D, DV, x);         \
+    } while (0)
+#define LAUNCH_X_ALL(TI, TQ, TKV)                                                                                                  \
+    do {                                                                                                                           \
+        if (it == 1) LAUNCH_X(TI, TQ, TKV, 1); else if (it == 2) LAUNCH_X(TI, TQ, TKV, 2); else LAUNCH_X(TI, TQ, TKV, 4);           \
+    } while (0)
+        PH_DISPATCH(rows_dtype, TI, PH_DISPATCH(q_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, LAUNCH_X_ALL(TI, TQ, TKV))));
+#undef LAUNCH_X_ALL
+#undef LAUNCH_X
+        return check_launch("joint_norm_rope_kv_write");
+    }
+    if (vec && plain) {
         const int vthreads = (HQ + HKV) * D / 8 >= 256 ? 256 : 128;
 #define LAUNCH_VEC(TI, TQ, TKV)                                                                                                    \
     do {                                                                                                                           \
         auto kern = joint_norm_kv_write_vec_kernel<TI, TQ, TKV>;                                                                   \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                  \
         launch_overlapped(kern, dim3(T), dim3(vthreads), smem, stream, (const TI*)rows, splits, split_stride, row_width, q_w, k_w, eps, slot_mapping, (TQ*)q_out, \
-                                            (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, D, DV, v_from_row, x);       \
+                                            (TKV*)k_base, (TKV*)v_base, page_stride, page_size, HQ, HKV, D, DV, v_from_row);       \
     } while (0)
         PH_DISPATCH(rows_dtype, TI, PH_DISPATCH(q_dtype, TQ, PH_DISPATCH(kv_dtype, TKV, LAUNCH_VEC(TI, TQ, TKV))));
 #undef LAUNCH_VEC

@@ -468,43 +468,64 @@ PH_EXPORT int ph_delta_chunk_tokens(void) { return C; }
 // bytes of scratch per (chunk, head): the operands, U0, and the chunk's decay
 PH_EXPORT long long ph_delta_chunk_scratch_bytes(int D, int DV) { return (ops_elems(D) * 2 + 4LL * C * DV + 4LL * D + 255) / 256 * 256; }
 
-// The requests whose rows the chunk list holds: chunks [n_chunks][2] (first row of the step, rows, at most 64), seg_chunks [S + 1]
-// (a request without chunks is left alone).  scratch: n_chunks * H * ph_delta_chunk_scratch_bytes, 256-byte aligned.  The rest
-// as ph_delta_scan.
-PH_EXPORT int ph_delta_chunk(const float* qkv, const float* beta, const float* log_decay, const float* z, long long z_stride, const float* z_bias,
-                             const float* rate, const void* rows, int rows_dtype, int splits, long long split_stride, long long width,
-                             float* state, long long state_stride, long long conv_at, const int32_t* seg_start, const int32_t* seg_slot, int S,
-                             const int32_t* chunks, int n_chunks, const int32_t* seg_chunks, void* scratch, int H, int G, int D, int DV, int K,
-                             float* o, cudaStream_t stream) {
-    if (!qkv || !beta || (!log_decay == !z) || (z && (!z_bias || !rate)) || !rows || !state || !seg_start || !seg_slot || !o || !chunks ||
-        !seg_chunks || !scratch || S < 1 || n_chunks < 1 || H < 1 || G < 1 || H % G || K < 1 || splits < 1 || !valid_dtype(rows_dtype))
-        return fail(PH_ERR_ARG, "delta_chunk: bad arguments (S %d, chunks %d, H %d, G %d, D %d, DV %d)", S, n_chunks, H, G, D, DV);
+namespace {
+int fill(ChunkParams& p, const int32_t* chunks, int n_chunks, const int32_t* seg_chunks, void* scratch, int H, int G, int D, int DV) {
+    if (!chunks || !scratch || n_chunks < 1 || H < 1 || G < 1 || H % G)
+        return fail(PH_ERR_ARG, "delta_chunk: bad arguments (chunks %d, H %d, G %d, D %d, DV %d)", n_chunks, H, G, D, DV);
     if (!ph_delta_chunk_supports(D, DV)) return fail(PH_ERR_UNSUPPORTED, "delta_chunk: heads of %d / %d are not taken", D, DV);
-    if ((2LL * G * D + (long long)H * DV) % 4 || ((uintptr_t)qkv & 15) || ((uintptr_t)o & 7) || ((uintptr_t)scratch & 255))
+    if ((2LL * G * D + (long long)H * DV) % 4 || ((uintptr_t)scratch & 255))
         return fail(PH_ERR_UNSUPPORTED, "delta_chunk: rows must be 16-byte aligned");
-    ChunkParams p;
-    p.s.qkv = qkv; p.s.beta = beta; p.s.log_decay = log_decay; p.s.z = z; p.s.z_stride = z_stride; p.s.z_bias = z_bias; p.s.rate = rate;
-    p.s.rows = rows; p.s.splits = splits; p.s.split_stride = split_stride; p.s.width = width; p.s.state = state; p.s.state_stride = state_stride;
-    p.s.conv_at = conv_at; p.s.seg_start = seg_start; p.s.seg_slot = seg_slot; p.s.o = o; p.s.H = H; p.s.G = G; p.s.D = D; p.s.DV = DV; p.s.K = K;
-    p.s.rows_from = 0; p.s.rows_to = 0;
-    p.chunks = chunks; p.seg_chunks = seg_chunks; p.rows_bf16 = rows_dtype == PH_BF16;
     const long long units = (long long)n_chunks * H;
+    p.s.H = H; p.s.G = G; p.s.D = D; p.s.DV = DV;
+    p.chunks = chunks; p.seg_chunks = seg_chunks;
     p.ops = static_cast<__nv_bfloat16*>(scratch);
     p.u0 = reinterpret_cast<float*>(p.ops + units * ops_elems(D));
     p.last = p.u0 + units * C * DV;
-    const size_t make = (size_t)make_floats(D) * sizeof(float), walk = (size_t)walk_smem(D);
-    static size_t make_set = 0, walk_set = 0;
-    if (make > make_set) {
-        if (cudaFuncSetAttribute(delta_chunk_make_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)make) != cudaSuccess)
-            return fail(PH_ERR_LAUNCH, "delta_chunk: cannot reserve %zu bytes of shared memory", make);
-        make_set = make;
+    return PH_OK;
+}
+}  // namespace
+
+// The operands of every chunk and head.  chunks [n_chunks][2]: first row of the step and rows, at most 64; scratch: n_chunks * H *
+// ph_delta_chunk_scratch_bytes, 256-byte aligned.  qkv, beta, log_decay / z as in ph_delta_scan.
+PH_EXPORT int ph_delta_chunk_make(const float* qkv, const float* beta, const float* log_decay, const float* z, long long z_stride,
+                                  const float* z_bias, const float* rate, const int32_t* chunks, int n_chunks, void* scratch, int H, int G, int D,
+                                  int DV, cudaStream_t stream) {
+    if (!qkv || !beta || (!log_decay == !z) || (z && (!z_bias || !rate)) || ((uintptr_t)qkv & 15))
+        return fail(PH_ERR_ARG, "delta_chunk_make: bad arguments");
+    ChunkParams p = {};
+    if (int rc = fill(p, chunks, n_chunks, nullptr, scratch, H, G, D, DV)) return rc;
+    p.s.qkv = qkv; p.s.beta = beta; p.s.log_decay = log_decay; p.s.z = z; p.s.z_stride = z_stride; p.s.z_bias = z_bias; p.s.rate = rate;
+    const size_t smem = (size_t)make_floats(D) * sizeof(float);
+    static size_t set = 0;
+    if (smem > set) {
+        if (cudaFuncSetAttribute(delta_chunk_make_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+            return fail(PH_ERR_LAUNCH, "delta_chunk_make: cannot reserve %zu bytes of shared memory", smem);
+        set = smem;
     }
-    if (walk > walk_set) {
-        if (cudaFuncSetAttribute(delta_chunk_walk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk) != cudaSuccess)
-            return fail(PH_ERR_LAUNCH, "delta_chunk: cannot reserve %zu bytes of shared memory", walk);
-        walk_set = walk;
+    launch_overlapped(delta_chunk_make_kernel, dim3(n_chunks, H), dim3(MAKE_THREADS), smem, stream, p);
+    return check_launch("delta_chunk_make");
+}
+
+// The recurrence over the chunks of each request (seg_chunks [S + 1]; a request without chunks is left alone); what is left of
+// its rows in the state as in ph_delta_scan.
+PH_EXPORT int ph_delta_chunk_walk(const void* rows, int rows_dtype, int splits, long long split_stride, long long width, float* state,
+                                  long long state_stride, long long conv_at, const int32_t* seg_start, const int32_t* seg_slot, int S,
+                                  const int32_t* chunks, int n_chunks, const int32_t* seg_chunks, const void* scratch, int H, int G, int D,
+                                  int DV, int K, float* o, cudaStream_t stream) {
+    if (!rows || !state || !seg_start || !seg_slot || !seg_chunks || !o || S < 1 || K < 1 || splits < 1 || !valid_dtype(rows_dtype) || ((uintptr_t)o & 7))
+        return fail(PH_ERR_ARG, "delta_chunk_walk: bad arguments (S %d)", S);
+    ChunkParams p = {};
+    if (int rc = fill(p, chunks, n_chunks, seg_chunks, const_cast<void*>(scratch), H, G, D, DV)) return rc;
+    p.s.rows = rows; p.s.splits = splits; p.s.split_stride = split_stride; p.s.width = width; p.s.state = state; p.s.state_stride = state_stride;
+    p.s.conv_at = conv_at; p.s.seg_start = seg_start; p.s.seg_slot = seg_slot; p.s.o = o; p.s.K = K;
+    p.rows_bf16 = rows_dtype == PH_BF16;
+    const size_t smem = (size_t)walk_smem(D);
+    static size_t set = 0;
+    if (smem > set) {
+        if (cudaFuncSetAttribute(delta_chunk_walk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+            return fail(PH_ERR_LAUNCH, "delta_chunk_walk: cannot reserve %zu bytes of shared memory", smem);
+        set = smem;
     }
-    launch_overlapped(delta_chunk_make_kernel, dim3(n_chunks, H), dim3(MAKE_THREADS), make, stream, p);
-    launch_overlapped(delta_chunk_walk_kernel, dim3((DV + NC - 1) / NC, H, S), dim3(WALK_THREADS), walk, stream, p);
-    return check_launch("delta_chunk");
+    launch_overlapped(delta_chunk_walk_kernel, dim3((DV + NC - 1) / NC, H, S), dim3(WALK_THREADS), smem, stream, p);
+    return check_launch("delta_chunk_walk");
 }

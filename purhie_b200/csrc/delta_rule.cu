@@ -116,41 +116,110 @@ __device__ __forceinline__ void conv_any(const PrepParams& p, int t, int kind, i
     }
 }
 
+// The same for the tokens t0 .. t0 + count - 1 with the last KT inputs in registers, so that a row is read once: heads of up to
+// 128 channels, four per lane.  The order of each sum is the one above.
+template <typename TI, int KT>
+__device__ __forceinline__ void conv_run(const PrepParams& p, int t0, int count, int kind, int c0, int n) {
+    const int lane = threadIdx.x & 31, d = lane * 4, CH = 2 * p.G * p.D + p.H * p.DV;
+    const bool on = d < n;
+    const TI* rows = static_cast<const TI*>(p.rows);
+    float4 w[KT], x[KT];
+#pragma unroll
+    for (int j = 0; j < KT; ++j) w[j] = on ? load4(p.taps + (size_t)j * CH + c0 + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    auto input = [&](int row) {
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (!on) return v;
+        const TI* at = rows + (size_t)row * p.width + c0 + d;
+        v = load4(at);
+        for (int sp = 1; sp < p.splits; ++sp) {
+            const float4 m = load4(at + (size_t)sp * p.split_stride);
+            v.x += m.x; v.y += m.y; v.z += m.z; v.w += m.w;
+        }
+        return v;
+    };
+    int seg = -1;
+    float4 next = input(t0);
+    for (int r = 0; r < count; ++r) {
+        const int t = t0 + r, s = p.row_seg[t];
+        if (s != seg) {                                    // the run's first row, or another request's
+            seg = s;
+            const int first = p.seg_start[s], i0 = t - first;
+            const float* past = p.state + (size_t)p.seg_slot[s] * p.state_stride + p.conv_at;
+#pragma unroll
+            for (int j = 0; j < KT - 1; ++j) {
+                const int src = i0 - (KT - 1) + j;
+                x[j] = src >= 0 ? input(first + src) : on ? load4(past + (size_t)(src + KT - 1) * CH + c0 + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            }
+        }
+        x[KT - 1] = next;
+        if (r + 1 < count) next = input(t + 1);
+        float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+        for (int j = 0; j < KT; ++j) {
+            y.x = fmaf(w[j].x, x[j].x, y.x); y.y = fmaf(w[j].y, x[j].y, y.y);
+            y.z = fmaf(w[j].z, x[j].z, y.z); y.w = fmaf(w[j].w, x[j].w, y.w);
+        }
+#pragma unroll
+        for (int j = 0; j < KT - 1; ++j) x[j] = x[j + 1];
+        y.x = y.x / (1.0f + expf(-y.x)); y.y = y.y / (1.0f + expf(-y.y)); y.z = y.z / (1.0f + expf(-y.z)); y.w = y.w / (1.0f + expf(-y.w));
+        float f = 1.0f;
+        if (kind < 2) {
+            float ss = 0.0f;
+            ss += y.x * y.x; ss += y.y * y.y; ss += y.z * y.z; ss += y.w * y.w;
+            f = rsqrtf(warp_sum(ss) + UNIT_EPS) * (kind == 0 ? p.q_scale : 1.0f);
+        }
+        if (on) *reinterpret_cast<float4*>(p.qkv + (size_t)t * CH + c0 + d) = make_float4(y.x * f, y.y * f, y.z * f, y.w * f);
+    }
+}
+
+template <typename TI>
+__device__ __forceinline__ void conv_tokens(const PrepParams& p, int t0, int count, int kind, int c0, int n, int v, int ni) {
+    if (count > 1 && v == 4 && ni == 1 && p.K >= 2 && p.K <= 4) {
+        if (p.K == 2) conv_run<TI, 2>(p, t0, count, kind, c0, n);
+        else if (p.K == 3) conv_run<TI, 3>(p, t0, count, kind, c0, n);
+        else conv_run<TI, 4>(p, t0, count, kind, c0, n);
+        return;
+    }
+    for (int r = 0; r < count; ++r) conv_any<TI>(p, t0 + r, kind, c0, n, v, ni);
+}
+
 // TI: the dtype of the rows; TO: the model's dtype (rows in parts are float32 in a bfloat16 model)
 template <typename TI, typename TO>
-__global__ void __launch_bounds__(PREP_WARPS * 32) delta_prepare_kernel(const PrepParams p) {
+__global__ void __launch_bounds__(PREP_WARPS * 32, 2) delta_prepare_kernel(const PrepParams p, int T, int run) {
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * run, count = min(run, T - t0), lane = threadIdx.x & 31;
     int unit = blockIdx.y * PREP_WARPS + (threadIdx.x >> 5);
     const int QK = 2 * p.G * p.D;
     if (unit < 2 * p.G) {
-        conv_any<TI>(p, t, unit < p.G ? 0 : 1, unit * p.D, p.D, p.qk_v, p.qk_n);
+        conv_tokens<TI>(p, t0, count, unit < p.G ? 0 : 1, unit * p.D, p.D, p.qk_v, p.qk_n);
         return;
     }
     unit -= 2 * p.G;
     if (unit < p.H) {
-        conv_any<TI>(p, t, 2, QK + unit * p.DV, p.DV, p.v_v, p.v_n);
+        conv_tokens<TI>(p, t0, count, 2, QK + unit * p.DV, p.DV, p.v_v, p.v_n);
         return;
     }
     unit -= p.H;
-    const TI* row = static_cast<const TI*>(p.rows) + (size_t)t * p.width;
-    auto value = [&](int c) {
-        float v = to_float<TI>(row[c]);
-        for (int s = 1; s < p.splits; ++s) v += to_float<TI>(row[(size_t)s * p.split_stride + c]);
-        return v;
-    };
-    // the tail: [beta | decay | low rows | gate], TAIL elements per warp
-    const int nb = p.H, na = p.a_col >= 0 ? p.H : 0, all = nb + na + p.low_n + p.gate_n;
-    for (int e = unit * TAIL + lane; e < min(all, (unit + 1) * TAIL); e += 32) {
-        int i = e;
-        if (i < nb) { p.beta[(size_t)t * p.H + i] = 1.0f / (1.0f + expf(-value(p.b_col + i))); continue; }
-        i -= nb;
-        if (i < na) { p.log_decay[(size_t)t * p.H + i] = p.rate[i] * ph_delta::softplus(value(p.a_col + i) + p.a_bias[i]); continue; }
-        i -= na;
-        if (i < p.low_n) { static_cast<TO*>(p.low)[(size_t)t * p.low_n + i] = from_float<TO>(value(p.low_col + i)); continue; }
-        i -= p.low_n;
-        static_cast<TO*>(p.gate)[(size_t)t * p.gate_n + i] = from_float<TO>(value(p.gate_col + i));
+    for (int t = t0; t < t0 + count; ++t) {
+        const TI* row = static_cast<const TI*>(p.rows) + (size_t)t * p.width;
+        auto value = [&](int c) {
+            float v = to_float<TI>(row[c]);
+            for (int s = 1; s < p.splits; ++s) v += to_float<TI>(row[(size_t)s * p.split_stride + c]);
+            return v;
+        };
+        // the tail: [beta | decay | low rows | gate], TAIL elements per warp
+        const int nb = p.H, na = p.a_col >= 0 ? p.H : 0, all = nb + na + p.low_n + p.gate_n;
+        for (int e = unit * TAIL + lane; e < min(all, (unit + 1) * TAIL); e += 32) {
+            int i = e;
+            if (i < nb) { p.beta[(size_t)t * p.H + i] = 1.0f / (1.0f + expf(-value(p.b_col + i))); continue; }
+            i -= nb;
+            if (i < na) { p.log_decay[(size_t)t * p.H + i] = p.rate[i] * ph_delta::softplus(value(p.a_col + i) + p.a_bias[i]); continue; }
+            i -= na;
+            if (i < p.low_n) { static_cast<TO*>(p.low)[(size_t)t * p.low_n + i] = from_float<TO>(value(p.low_col + i)); continue; }
+            i -= p.low_n;
+            static_cast<TO*>(p.gate)[(size_t)t * p.gate_n + i] = from_float<TO>(value(p.gate_col + i));
+        }
     }
 }
 
@@ -330,9 +399,10 @@ PH_EXPORT int ph_delta_prepare(const void* rows, int rows_dtype, int splits, lon
     lanes_for(DV, vec && DV % 4 == 0 && (2LL * G * D) % 4 == 0, &p.v_v, &p.v_n);
     if (D > 512 || DV > 512) return fail(PH_ERR_UNSUPPORTED, "delta_prepare: heads of %d / %d exceed the supported 512", D, DV);
     const int tail = H + (a_col >= 0 ? H : 0) + low_n + gate_n, units = 2 * G + H + (tail + TAIL - 1) / TAIL;
-    const dim3 grid(T, (units + PREP_WARPS - 1) / PREP_WARPS);
+    const int run = T >= 512 ? 8 : 1;              // many rows: a warp walks several tokens
+    const dim3 grid((T + run - 1) / run, (units + PREP_WARPS - 1) / PREP_WARPS);
     PH_DISPATCH(rows_dtype, TI, PH_DISPATCH(model_dtype, TO,
-        launch_overlapped(delta_prepare_kernel<TI, TO>, grid, dim3(PREP_WARPS * 32), 0, stream, p)));
+        launch_overlapped(delta_prepare_kernel<TI, TO>, grid, dim3(PREP_WARPS * 32), 0, stream, p, T, run)));
     return check_launch("delta_prepare");
 }
 

@@ -199,7 +199,8 @@ const CoreKernels& core_kernels() {
     bind(h, "core", "ph_add_scaled_rmsnorm", g_core.add_scaled_rmsnorm);
     bind(h, "core", "ph_delta_prepare", g_core.delta_prepare);
     bind(h, "core", "ph_delta_scan", g_core.delta_scan);
-    bind(h, "core", "ph_delta_chunk", g_core.delta_chunk);
+    bind(h, "core", "ph_delta_chunk_make", g_core.delta_chunk_make);
+    bind(h, "core", "ph_delta_chunk_walk", g_core.delta_chunk_walk);
     bind(h, "core", "ph_delta_chunk_supports", g_core.delta_chunk_supports);
     bind(h, "core", "ph_delta_chunk_tokens", g_core.delta_chunk_tokens);
     bind(h, "core", "ph_delta_chunk_scratch_bytes", g_core.delta_chunk_scratch_bytes);

@@ -262,11 +262,20 @@ public:
             for (int n : ctx.q_lens)
                 if (n >= kChunkRows) { n_long++; rows_long += n; }
             Tensor scratch = ws.get("delta_scratch", {(int64_t)n_chunks * heads_ * k.delta_chunk_scratch_bytes(dim_, vdim_)}, DType::U8);
-            note(n_long, rows_long);
-            QE_LAUNCH(k, k.delta_chunk(qkv.as<float>(), beta.as<float>(), low_decay_ ? nullptr : log_decay.as<float>(), z, up_width_,
-                                       low_decay_ ? dt_bias_.as<float>() : nullptr, rate_.as<float>(), in.tensor.data, in.tensor.code(), in.splits,
-                                       split_stride, width_, state, state_floats(), conv_at(), ctx.seg_start, ctx.seg_slot, ctx.S, chunks.data,
-                                       n_chunks, seg_chunks.data, scratch.data, heads_, kv_heads_, dim_, vdim_, taps_, o.as<float>(), ctx.stream));
+            // (q, k, v and the decays in, the operands out; the operands in, o out, the state in and out)
+            const double made = (double)n_chunks * heads_ * k.delta_chunk_scratch_bytes(dim_, vdim_);
+            if (profile.on())
+                LaunchProfile::get().note_cost(rows_long * 4.0 * (channels_ + (low_decay_ ? decay_width_ : heads_) + heads_) + made,
+                                               (double)rows_long * heads_ * 64.0 * (2.0 * dim_ + dim_ + vdim_));
+            QE_LAUNCH(k, k.delta_chunk_make(qkv.as<float>(), beta.as<float>(), low_decay_ ? nullptr : log_decay.as<float>(), z, up_width_,
+                                            low_decay_ ? dt_bias_.as<float>() : nullptr, rate_.as<float>(), chunks.data, n_chunks, scratch.data,
+                                            heads_, kv_heads_, dim_, vdim_, ctx.stream));
+            if (profile.on())
+                LaunchProfile::get().note_cost(made + rows_long * 4.0 * v_width_ + 2.0 * n_long * (double)state_floats() * 4.0,
+                                               (double)rows_long * heads_ * vdim_ * (6.0 * dim_ + 64.0));
+            QE_LAUNCH(k, k.delta_chunk_walk(in.tensor.data, in.tensor.code(), in.splits, split_stride, width_, state, state_floats(), conv_at(),
+                                            ctx.seg_start, ctx.seg_slot, ctx.S, chunks.data, n_chunks, seg_chunks.data, scratch.data, heads_,
+                                            kv_heads_, dim_, vdim_, taps_, o.as<float>(), ctx.stream));
         }
         if (n_long < ctx.S) {
             note(ctx.S - n_long, T - rows_long);
