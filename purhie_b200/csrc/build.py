@@ -32,7 +32,7 @@ LIBRARIES: Dict[str, dict] = {
                     "random_fill.cu", "layernorm.cu", "gated.cu", "mamba.cu", "moe.cu", "linear_attention.cu", "dyntanh.cu",
                     "latent_attention.cu", "attention_talking.cu", "attention_talking_mma.cu", "min_gru.cu", "lanes.cu",
                     "ssd.cu", "delta_rule.cu", "delta_chunk.cu", "core_lib.cu"],
-        "deps": ["../weights/random.h", "attention_mma.cuh", "delta_rule.cuh"],
+        "deps": ["../weights/random.h", "attention_mma.cuh", "delta_rule.cuh", "mbarrier.cuh"],
         "flags": [],
         "link": [],
     },

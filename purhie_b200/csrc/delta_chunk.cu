@@ -10,20 +10,24 @@
 // The triangular system is solved for its two right-hand sides before S is known: U = U0 - W S with
 // (1 + diag(beta) A) [W | U0] = diag(beta) [k exp(G) | V].
 //
-//   delta_chunk_make   a block per (chunk, head), all chunks side by side: A and P in float32 on packed multiply-adds, row block
-//                      by row block of 16 with the decays taken from the block's first token, so that every exponential of an
-//                      earlier block is at most 1; inside a block the inverse factor may grow, and where it would grow beyond
-//                      2^60 the block takes every pair's exponential itself.  The system is solved by forward
-//                      substitution in float32, two columns per thread.  W, q exp(G), k exp(G_last - G) and P leave as two
-//                      bfloat16 each, the rounded value and the rounded rest.
+//   delta_chunk_make   a block per (chunk, head), all chunks side by side.  The chunk is cut into blocks of 16 tokens: with g_i
+//                      the running sum inside token i's block and t_J block J's total, A and P of block rows I and block
+//                      columns J come from k exp(g), q exp(g), k exp(t_J - g) (never above 1) and one factor per channel and
+//                      pair of blocks, the decay between them; on the diagonal that factor is exp(-t_I), and where it would
+//                      exceed 2^60 the block takes every pair's exponential itself.  Float32 on packed multiply-adds, 2 x 2
+//                      pairs per thread.  The system is solved by forward substitution in float32, a column per thread, by half
+//                      of the warps while the others write the operands.  W, q exp(G), k exp(G_last - G) and P leave as two
+//                      bfloat16 each, the rounded value and the rounded rest, in the layout of the walk's shared memory.
 //   delta_chunk_walk   a block per (request, head, 32 columns of S) that walks the request's chunks in order with S in registers
 //                      (float32, spread over its eight warps) and, split the same way, in shared memory.  Every product is three
 //                      tensor-core products of the split operands, so 16 bits of every factor count, and the sums are float32.
 //                      Four warps make U while four others make (q exp(G)) S, then all add their part to S while the
-//                      second four add P U and store O; the next chunk's operands are on their way meanwhile.
+//                      second four add P U and store O; the next chunk's operands are on their way meanwhile, as bulk copies of
+//                      whole regions that complete on mbarriers (bounded waits, an error word).
 // Tokens beyond a request's last have k = q = v = beta = 0 and a decay of 1.
 #include "attention_mma.cuh"
 #include "delta_rule.cuh"
+#include "mbarrier.cuh"
 
 #include <math.h>
 
@@ -36,20 +40,27 @@ constexpr int C = 64;                  // tokens of a chunk
 constexpr int RB = 16;                 // tokens of a row block
 constexpr int NC = 32;                 // columns of S per block of the walk
 constexpr int MAX_DIM = 128;
-constexpr int MAKE_THREADS = 256, WALK_THREADS = 256;
+constexpr int MAKE_THREADS = 512, WALK_THREADS = 256;
+constexpr int PH_ERR_WAIT_DELTA = 131;
 constexpr float GROW_LIMIT = 60.0f;    // log2 of the largest inverse factor inside a row block
 
 struct ChunkParams {
     ph_delta::ScanParams s;
     const int32_t* chunks;             // [n][2]: first row, rows
     const int32_t* seg_chunks;         // [S + 1]
-    __nv_bfloat16* ops;                // per (chunk, head): [W hi | W lo | Q hi | Q lo | K hi | K lo] of 64 x D, then [P hi | P lo] of 64 x 64
+    uint8_t* ops;                      // per (chunk, head): [W hi | W lo | Q hi | Q lo | K hi | K lo] of 64 rows of D, then [P hi | P lo] of 64 rows of 64
     float* u0;                         // per (chunk, head): [64][DV]
     float* last;                       // per (chunk, head): [D] exp(G_last)
     int rows_bf16;                     // the projections' rows are bfloat16
+    int* error_flag;
 };
 
-__host__ __device__ constexpr long long ops_elems(int D) { return 6LL * C * D + 2LL * C * C; }
+// bytes between two rows of an operand of D (64) columns: 16 more than the row, so that eight rows miss each other's banks
+__host__ __device__ constexpr int op_pitch(int D) { return D * 2 + 16; }
+constexpr int P_PITCH = C * 2 + 16;
+__host__ __device__ constexpr int first_bytes(int D) { return 4 * C * op_pitch(D); }               // W and Q
+__host__ __device__ constexpr int second_bytes(int D) { return 2 * C * op_pitch(D) + 2 * C * P_PITCH; }    // K and P
+__host__ __device__ constexpr long long ops_bytes(int D) { return first_bytes(D) + second_bytes(D); }
 
 __device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
@@ -61,218 +72,248 @@ __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
         : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
     return d;
 }
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("{\n.reg .b64 ra, rb, rd;\n"
+        "mov.b64 ra, {%2, %3};\nmov.b64 rb, {%4, %5};\n"
+        "mul.rn.f32x2 rd, ra, rb;\n"
+        "mov.b64 {%0, %1}, rd;\n}"
+        : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+    return d;
+}
 // v = hi + lo with both in bfloat16 (hi the rounded value, lo the rounded rest), two values at a time
 __device__ __forceinline__ void split2(float u, float v, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(u, v);
     lo = pack_bf16(u - __uint_as_float(hi << 16), v - __uint_as_float(hi & 0xffff0000u));
 }
 
-// floats of shared memory of delta_chunk_make: k, q, G, the scaled keys [64][D + 4], the scaled rows of k and q [16][D + 4],
-// the system [64][64 + 4] and P [64][64 + 4], beta [64]
-__host__ __device__ constexpr int make_floats(int D) { return 4 * C * (D + 4) + 2 * RB * (D + 4) + 2 * C * (C + 4) + C; }
+// floats of shared memory of delta_chunk_make: k exp(g), q exp(g), k exp(t - g) and g [64][D + 4], the system and P [64][64 + 4],
+// the running sums at the blocks' starts [5][D], the factors between blocks [10][D], beta [64]
+__host__ __device__ constexpr int make_floats(int D) { return 4 * C * (D + 4) + 2 * C * (C + 4) + 15 * D + C; }
+constexpr int BLOCKS = C / RB;
 
 __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const ChunkParams p) {
     extern __shared__ __align__(16) float sm[];
-    __shared__ int slow;
+    __shared__ int slow[BLOCKS];
     const int D = p.s.D, DV = p.s.DV, DP = D + 4, H = p.s.H, CH = 2 * p.s.G * D + H * DV;
     constexpr int NP = C + 4;
-    float* ks = sm;                    // [64][DP]
-    float* qs = ks + C * DP;
-    float* Gs = qs + C * DP;           // in units of log2
-    float* kj = Gs + C * DP;
-    float* ki = kj + C * DP;           // [16][DP]
-    float* qi = ki + RB * DP;
-    float* N = qi + RB * DP;           // [64][NP]
+    float* kd = sm;                    // [64][DP]: k exp(g)
+    float* qd = kd + C * DP;           // q exp(g)
+    float* ke = qd + C * DP;           // k exp(t - g)
+    float* gs = ke + C * DP;           // g, in units of log2 (as every logarithm here)
+    float* N = gs + C * DP;            // [64][NP]: -diag(beta) A
     float* P = N + C * NP;
-    float* beta = P + C * NP;
+    float* base = P + C * NP;          // [5][D]: G at the start of each block, and at the chunk's end
+    float* F = base + 5 * D;           // [10][D]
+    float* beta = F + 10 * D;
     const int tid = threadIdx.x, item = blockIdx.x, h = blockIdx.y, g = h / (H / p.s.G);
     pdl_launch_dependents();
     pdl_wait();
     const int row0 = p.chunks[2 * item], n = p.chunks[2 * item + 1];
     const float* rows = p.s.qkv + (size_t)row0 * CH;
+    const float* q_rows = rows + g * D;
+    const float* k_rows = rows + (p.s.G + g) * D;
 
-    // ---- the chunk's rows
-    const int per_row = D / 4;
-    for (int i = tid; i < C * per_row; i += MAKE_THREADS) {
-        const int r = i / per_row, d = (i % per_row) * 4;
-        float4 q4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f), k4 = q4;
-        if (r < n) {
-            q4 = *reinterpret_cast<const float4*>(rows + (size_t)r * CH + g * D + d);
-            k4 = *reinterpret_cast<const float4*>(rows + (size_t)r * CH + (p.s.G + g) * D + d);
-        }
-        *reinterpret_cast<float4*>(qs + r * DP + d) = q4;
-        *reinterpret_cast<float4*>(ks + r * DP + d) = k4;
-    }
+    // ---- the running sums inside the blocks: a thread per (channel, block)
+    if (tid < BLOCKS) slow[tid] = 0;
     if (tid < C) beta[tid] = tid < n ? p.s.beta[(size_t)(row0 + tid) * H + h] : 0.0f;
-    // ---- G: each half of the tokens summed by a thread of its own per channel, then the first half's sum added to the second
-    if (tid < 2 * D) {
-        const int d = tid % D, part = tid / D, first = part * (C / 2);
-        float run = 0.0f;
+    for (int i = tid; i < C * NP; i += MAKE_THREADS) { N[i] = 0.0f; P[i] = 0.0f; }
+    if (tid < BLOCKS * D) {
+        const int d = tid % D, J = tid / D;
+        float run = 0.0f, x[RB];
         if (p.s.z) {
             const float rate = p.s.rate[h] * LOG2E, bias = p.s.z_bias[(size_t)h * D + d];
             const float* z = p.s.z + (size_t)row0 * p.s.z_stride + (size_t)h * D + d;
-#pragma unroll 8
-            for (int t = 0; t < C / 2; ++t) {
-                const int i = first + t;
-                run += i < n ? rate * ph_delta::softplus(z[(size_t)i * p.s.z_stride] + bias) : 0.0f;
-                Gs[i * DP + d] = run;
-            }
+#pragma unroll
+            for (int t = 0; t < RB; ++t) x[t] = J * RB + t < n ? z[(size_t)(J * RB + t) * p.s.z_stride] : 0.0f;
+#pragma unroll
+            for (int t = 0; t < RB; ++t) x[t] = J * RB + t < n ? rate * ph_delta::softplus(x[t] + bias) : 0.0f;
         } else {
             const float* ld = p.s.log_decay + (size_t)row0 * H + h;
-#pragma unroll 8
-            for (int t = 0; t < C / 2; ++t) {
-                const int i = first + t;
-                run += i < n ? ld[(size_t)i * H] * LOG2E : 0.0f;
-                Gs[i * DP + d] = run;
-            }
+#pragma unroll
+            for (int t = 0; t < RB; ++t) x[t] = J * RB + t < n ? ld[(size_t)(J * RB + t) * H] * LOG2E : 0.0f;
+        }
+#pragma unroll
+        for (int t = 0; t < RB; ++t) { run += x[t]; gs[(J * RB + t) * DP + d] = run; }
+    }
+    __syncthreads();
+    if (tid < D) {
+        float run = 0.0f;
+        base[tid] = 0.0f;
+#pragma unroll
+        for (int J = 0; J < BLOCKS; ++J) {
+            const float total = gs[(J * RB + RB - 1) * DP + tid];
+            if (-total > GROW_LIMIT) slow[J] = 1;                       // every writer writes the same
+            run += total;
+            base[(J + 1) * D + tid] = run;
         }
     }
     __syncthreads();
-    for (int i = tid; i < C / 2 * D; i += MAKE_THREADS) {
-        const int r = C / 2 + i / D, d = i % D;
-        Gs[r * DP + d] += Gs[(C / 2 - 1) * DP + d];
+    for (int i = tid; i < 10 * D; i += MAKE_THREADS) {
+        const int pair = i / D, d = i - pair * D;
+        const int I = pair >= 6 ? 3 : pair >= 3 ? 2 : pair >= 1 ? 1 : 0, J = pair - I * (I + 1) / 2;
+        F[i] = ex2(fminf(base[I * D + d] - base[(J + 1) * D + d], GROW_LIMIT));
     }
-    for (int i = tid; i < C * NP; i += MAKE_THREADS) { N[i] = 0.0f; P[i] = 0.0f; }
+    const int per_row = D / 4;
+    for (int i = tid; i < C * per_row; i += MAKE_THREADS) {
+        const int r = i / per_row, d = (i - r * per_row) * 4;
+        float4 q4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f), k4 = q4;
+        if (r < n) { q4 = load4(q_rows + (size_t)r * CH + d); k4 = load4(k_rows + (size_t)r * CH + d); }
+        const float4 g4 = load4(gs + r * DP + d), t4 = load4(gs + (r / RB * RB + RB - 1) * DP + d);
+        const float4 f = make_float4(ex2(g4.x), ex2(g4.y), ex2(g4.z), ex2(g4.w));
+        *reinterpret_cast<float4*>(kd + r * DP + d) = make_float4(k4.x * f.x, k4.y * f.y, k4.z * f.z, k4.w * f.w);
+        *reinterpret_cast<float4*>(qd + r * DP + d) = make_float4(q4.x * f.x, q4.y * f.y, q4.z * f.z, q4.w * f.w);
+        *reinterpret_cast<float4*>(ke + r * DP + d) =
+            make_float4(k4.x * ex2(t4.x - g4.x), k4.y * ex2(t4.y - g4.y), k4.z * ex2(t4.z - g4.z), k4.w * ex2(t4.w - g4.w));
+    }
+    __syncthreads();
 
-    // ---- A and P, 16 rows at a time
-    for (int I = 0; I < C / RB; ++I) {
-        __syncthreads();
-        if (tid == 0) slow = 0;
-        __syncthreads();
-        for (int d = tid; d < D; d += MAKE_THREADS) {
-            const float ref = I ? Gs[(I * RB - 1) * DP + d] : 0.0f;
-            if (ref - Gs[(I * RB + RB - 1) * DP + d] > GROW_LIMIT) slow = 1;       // every writer writes the same
-        }
-        for (int i = tid; i < (I + 1) * RB * D; i += MAKE_THREADS) {
-            const int r = i / D, d = i % D;
-            const float ref = I ? Gs[(I * RB - 1) * DP + d] : 0.0f;
-            kj[r * DP + d] = ks[r * DP + d] * ex2(fminf(ref - Gs[r * DP + d], GROW_LIMIT));
-            if (r >= I * RB) {
-                const float f = ex2(Gs[r * DP + d] - ref);
-                ki[(r - I * RB) * DP + d] = ks[r * DP + d] * f;
-                qi[(r - I * RB) * DP + d] = qs[r * DP + d] * f;
-            }
-        }
-        __syncthreads();
-        const bool every_pair = slow != 0;
-        const int i = tid / RB, j0 = tid % RB;             // this thread's row of the block, and its column of each block of columns
-        const float bi = beta[I * RB + i];
-        const int blocks = every_pair ? I : I + 1;
-        float2 a[C / RB], b[C / RB];
+    // ---- A and P: two warps per pair of blocks, a thread has rows i, i + 8 and columns j, j + 8 of it
+    const int warp = tid >> 5, lane = tid & 31;
+    for (int job = warp; job < 20; job += MAKE_THREADS / 32) {
+        const int pair = job >> 1;
+        const int I = pair >= 6 ? 3 : pair >= 3 ? 2 : pair >= 1 ? 1 : 0, J = pair - I * (I + 1) / 2;
+        const int i0 = I * RB + (lane >> 2), j0 = J * RB + (job & 1) * 4 + (lane & 3);
+        float a[2][2], b[2][2];
+        if (I == J && slow[I]) {
+            for (int u = 0; u < 2; ++u)
+                for (int v = 0; v < 2; ++v) {
+                    const int r = i0 + 8 * u, c = j0 + 8 * v;
+                    float sa = 0.0f, sb = 0.0f;
+                    if (c <= r && r < n)
+                        for (int d = 0; d < D; ++d) {
+                            const float x = k_rows[(size_t)c * CH + d] * ex2(gs[r * DP + d] - gs[c * DP + d]);
+                            sa = fmaf(k_rows[(size_t)r * CH + d], x, sa);
+                            sb = fmaf(q_rows[(size_t)r * CH + d], x, sb);
+                        }
+                    a[u][v] = sa; b[u][v] = sb;
+                }
+        } else {
+            float2 sa[2][2], sb[2][2];
 #pragma unroll
-        for (int m = 0; m < C / RB; ++m) a[m] = b[m] = make_float2(0.0f, 0.0f);
-        const float* kr = ki + i * DP;
-        const float* qr = qi + i * DP;
-        for (int d = 0; d < D; d += 4) {
-            const float4 k4 = *reinterpret_cast<const float4*>(kr + d), q4 = *reinterpret_cast<const float4*>(qr + d);
+            for (int u = 0; u < 2; ++u)
 #pragma unroll
-            for (int m = 0; m < C / RB; ++m) {
-                if (m >= blocks) break;
-                const float4 x = *reinterpret_cast<const float4*>(kj + (m * RB + j0) * DP + d);
-                a[m] = fma2(make_float2(k4.x, k4.y), make_float2(x.x, x.y), a[m]);
-                a[m] = fma2(make_float2(k4.z, k4.w), make_float2(x.z, x.w), a[m]);
-                b[m] = fma2(make_float2(q4.x, q4.y), make_float2(x.x, x.y), b[m]);
-                b[m] = fma2(make_float2(q4.z, q4.w), make_float2(x.z, x.w), b[m]);
+                for (int v = 0; v < 2; ++v) sa[u][v] = sb[u][v] = make_float2(0.0f, 0.0f);
+            const float* f = F + pair * D;
+#pragma unroll 2
+            for (int d = 0; d < D; d += 4) {
+                const float4 f4 = load4(f + d);
+                float2 x[2][2];                                   // the two columns' keys with the factor between the blocks
+#pragma unroll
+                for (int v = 0; v < 2; ++v) {
+                    const float4 e = load4(ke + (j0 + 8 * v) * DP + d);
+                    x[v][0] = mul2(make_float2(e.x, e.y), make_float2(f4.x, f4.y));
+                    x[v][1] = mul2(make_float2(e.z, e.w), make_float2(f4.z, f4.w));
+                }
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    const float4 k4 = load4(kd + (i0 + 8 * u) * DP + d), q4 = load4(qd + (i0 + 8 * u) * DP + d);
+#pragma unroll
+                    for (int v = 0; v < 2; ++v) {
+                        sa[u][v] = fma2(make_float2(k4.x, k4.y), x[v][0], sa[u][v]);
+                        sb[u][v] = fma2(make_float2(q4.x, q4.y), x[v][0], sb[u][v]);
+                        sa[u][v] = fma2(make_float2(k4.z, k4.w), x[v][1], sa[u][v]);
+                        sb[u][v] = fma2(make_float2(q4.z, q4.w), x[v][1], sb[u][v]);
+                    }
+                }
             }
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+#pragma unroll
+                for (int v = 0; v < 2; ++v) { a[u][v] = sa[u][v].x + sa[u][v].y; b[u][v] = sb[u][v].x + sb[u][v].y; }
         }
 #pragma unroll
-        for (int m = 0; m < C / RB; ++m) {
-            if (m >= blocks) break;
-            const int r = I * RB + i, j = m * RB + j0;
-            if (j < r) N[r * NP + j] = bi * (a[m].x + a[m].y);
-            if (j <= r) P[r * NP + j] = b[m].x + b[m].y;
-        }
-        if (every_pair && j0 <= i) {
-            const int r = I * RB + i, j = I * RB + j0;
-            float sa = 0.0f, sb = 0.0f;
-            for (int d = 0; d < D; ++d) {
-                const float x = ks[j * DP + d] * ex2(Gs[r * DP + d] - Gs[j * DP + d]);
-                sa = fmaf(ks[r * DP + d], x, sa);
-                sb = fmaf(qs[r * DP + d], x, sb);
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int v = 0; v < 2; ++v) {
+                const int r = i0 + 8 * u, c = j0 + 8 * v;
+                if (c < r) N[r * NP + c] = -beta[r] * a[u][v];
+                if (c <= r) P[r * NP + c] = b[u][v];
             }
-            if (j < r) N[r * NP + j] = bi * sa;
-            P[r * NP + j] = sb;
-        }
     }
     __syncthreads();
 
     const size_t at = (size_t)item * H + h;
-    uint32_t* ops = reinterpret_cast<uint32_t*>(p.ops + at * ops_elems(D));
-    const int tile = C * D / 2;        // pairs of a 64 x D operand
-    if (tid < MAKE_THREADS / 2) {
-        // ---- the system, two columns of [W | U0] per thread
+    uint8_t* ops = p.ops + at * ops_bytes(D);
+    const int pitch = op_pitch(D), op = C * pitch;
+    constexpr int HALF = MAKE_THREADS / 2;
+    if (tid < HALF) {
+        // ---- the system, a column of [W | U0] per thread; two neighbouring rows of it in a register pair
         float* u0 = p.u0 + at * C * DV;
-        for (int c = 2 * tid; c < D + DV; c += MAKE_THREADS) {
-            const bool is_w = c < D;
-            float2 x[C];
+        for (int c0 = 0; c0 < D + DV; c0 += HALF) {
+            const int c = c0 + tid;                        // (D is even: a pair of lanes is in W or in U0)
+            const bool is_w = c < D, on = c < D + DV;
+            float2 x[C / 2];
+            float first[BLOCKS];
+#pragma unroll
+            for (int J = 0; J < BLOCKS; ++J) first[J] = is_w ? ex2(base[J * D + c]) : 0.0f;
             const float* v = rows + 2 * p.s.G * D + (size_t)h * DV + (c - D);
 #pragma unroll
-            for (int i = 0; i < C; ++i) {
-                float2 r = make_float2(0.0f, 0.0f);
+            for (int i = 0; i < C; i += 2) {
+                float r0 = 0.0f, r1 = 0.0f;
                 if (is_w) {
-                    const float2 k2 = *reinterpret_cast<const float2*>(ks + i * DP + c), g2 = *reinterpret_cast<const float2*>(Gs + i * DP + c);
-                    r = make_float2(k2.x * ex2(g2.x), k2.y * ex2(g2.y));
-                } else if (i < n) {
-                    r = *reinterpret_cast<const float2*>(v + (size_t)i * CH);
+                    r0 = kd[i * DP + c] * first[i / RB];
+                    r1 = kd[(i + 1) * DP + c] * first[i / RB];
+                } else if (on) {
+                    if (i < n) r0 = v[(size_t)i * CH];
+                    if (i + 1 < n) r1 = v[(size_t)(i + 1) * CH];
                 }
-                x[i] = make_float2(r.x * beta[i], r.y * beta[i]);
+                x[i / 2] = make_float2(r0 * beta[i], r1 * beta[i + 1]);
             }
 #pragma unroll
             for (int i = 1; i < C; ++i) {
-                float2 even = x[i], odd = make_float2(0.0f, 0.0f);
+                float2 even = make_float2(0.0f, 0.0f), odd = even;
 #pragma unroll
-                for (int j = 0; j < i; j += 4) {
-                    const float4 m = *reinterpret_cast<const float4*>(N + i * NP + j);     // (zero from j = i on)
-                    even = fma2(make_float2(-m.x, -m.x), x[j], even);
-                    if (j + 1 < i) odd = fma2(make_float2(-m.y, -m.y), x[j + 1], odd);
-                    if (j + 2 < i) even = fma2(make_float2(-m.z, -m.z), x[j + 2], even);
-                    if (j + 3 < i) odd = fma2(make_float2(-m.w, -m.w), x[j + 3], odd);
+                for (int j = 0; j < i; j += 4) {                       // (N is zero from column i on)
+                    const float4 m = load4(N + i * NP + j);
+                    even = fma2(make_float2(m.x, m.y), x[j / 2], even);
+                    if (j + 2 < i) odd = fma2(make_float2(m.z, m.w), x[j / 2 + 1], odd);
                 }
-                x[i] = make_float2(even.x + odd.x, even.y + odd.y);
+                const float sum = (even.x + odd.x) + (even.y + odd.y);
+                if (i & 1) x[i / 2].y += sum; else x[i / 2].x += sum;
             }
 #pragma unroll
             for (int i = 0; i < C; ++i) {
-                if (is_w) {
+                const float own = i & 1 ? x[i / 2].y : x[i / 2].x;
+                const float other = __shfl_xor_sync(0xffffffffu, own, 1);
+                if (is_w) {                                            // the even lane stores the rounded pair, the odd one the rests
                     uint32_t hi, lo;
-                    split2(x[i].x, x[i].y, hi, lo);
-                    ops[(i * D + c) / 2] = hi;
-                    ops[tile + (i * D + c) / 2] = lo;
-                } else {
-                    *reinterpret_cast<float2*>(u0 + (size_t)i * DV + (c - D)) = x[i];
+                    if (c & 1) split2(other, own, hi, lo); else split2(own, other, hi, lo);
+                    *reinterpret_cast<uint32_t*>(ops + (c & 1) * op + i * pitch + (c & ~1) * 2) = c & 1 ? lo : hi;
+                } else if (on) {
+                    u0[(size_t)i * DV + (c - D)] = own;
                 }
             }
         }
     } else {
         // ---- the other operands
-        const int w = tid - MAKE_THREADS / 2;
-        const float* gl = Gs + (C - 1) * DP;
-        for (int e = w; e < tile; e += MAKE_THREADS / 2) {
-            const int i = 2 * e / D, d = 2 * e % D;
-            const float2 q2 = *reinterpret_cast<const float2*>(qs + i * DP + d), k2 = *reinterpret_cast<const float2*>(ks + i * DP + d),
-                         g2 = *reinterpret_cast<const float2*>(Gs + i * DP + d), l2 = *reinterpret_cast<const float2*>(gl + d);
-            uint32_t hi, lo;
-            split2(q2.x * ex2(g2.x), q2.y * ex2(g2.y), hi, lo);
-            ops[2 * tile + e] = hi; ops[3 * tile + e] = lo;
-            split2(k2.x * ex2(l2.x - g2.x), k2.y * ex2(l2.y - g2.y), hi, lo);
-            ops[4 * tile + e] = hi; ops[5 * tile + e] = lo;
+        const int w = tid - HALF;
+        auto put = [&](uint8_t* to, int rest, float4 v) {              // four elements, the rests `rest` bytes behind
+            uint32_t h0, l0, h1, l1;
+            split2(v.x, v.y, h0, l0);
+            split2(v.z, v.w, h1, l1);
+            *reinterpret_cast<uint2*>(to) = make_uint2(h0, h1);
+            *reinterpret_cast<uint2*>(to + rest) = make_uint2(l0, l1);
+        };
+        for (int e = w; e < C * per_row; e += HALF) {
+            const int i = e / per_row, d = (e - i * per_row) * 4, J = i / RB;
+            const float4 q4 = load4(qd + i * DP + d), k4 = load4(ke + i * DP + d);
+            const float4 b4 = load4(base + J * D + d), n4 = load4(base + (J + 1) * D + d), l4 = load4(base + BLOCKS * D + d);
+            uint8_t* to = ops + 2 * op + i * pitch + d * 2;
+            put(to, op, make_float4(q4.x * ex2(b4.x), q4.y * ex2(b4.y), q4.z * ex2(b4.z), q4.w * ex2(b4.w)));
+            put(to + 2 * op, op, make_float4(k4.x * ex2(l4.x - n4.x), k4.y * ex2(l4.y - n4.y), k4.z * ex2(l4.z - n4.z), k4.w * ex2(l4.w - n4.w)));
         }
-        for (int e = w; e < C * C / 2; e += MAKE_THREADS / 2) {
-            const int i = 2 * e / C, j = 2 * e % C;
-            uint32_t hi, lo;
-            split2(P[i * NP + j], P[i * NP + j + 1], hi, lo);
-            ops[6 * tile + e] = hi; ops[6 * tile + C * C / 2 + e] = lo;
+        for (int e = w; e < C * C / 4; e += HALF) {
+            const int i = e / (C / 4), j = e % (C / 4) * 4;
+            put(ops + 6 * op + i * P_PITCH + j * 2, C * P_PITCH, load4(P + i * NP + j));
         }
-        for (int d = w; d < D; d += MAKE_THREADS / 2) p.last[at * D + d] = ex2(gl[d]);
+        for (int d = w; d < D; d += HALF) p.last[at * D + d] = ex2(base[BLOCKS * D + d]);
     }
 }
 
 constexpr int S_PITCH = NC * 2 + 16;   // bytes of a row of the S and U tiles
-constexpr int P_PITCH = C * 2 + 16;
-__host__ __device__ constexpr int op_pitch(int D) { return D * 2 + 16; }
-// W and Q of two chunks, K and P of one, S, U: each as two bfloat16 tiles
-__host__ __device__ constexpr int walk_smem(int D) {
-    return 2 * 4 * C * op_pitch(D) + 2 * C * op_pitch(D) + 2 * C * P_PITCH + 2 * D * S_PITCH + 2 * C * S_PITCH;
-}
+// W and Q of two chunks, K and P of one, S, U (each as two bfloat16 tiles), three barriers
+__host__ __device__ constexpr int walk_smem(int D) { return 2 * first_bytes(D) + second_bytes(D) + 2 * D * S_PITCH + 2 * C * S_PITCH + 32; }
 
 // acc[16 x 32] += (a_hi + a_lo)[16 x 16 KS] (b_hi + b_lo)[16 KS x 32] without the product of the two rests.  a: row-major rows
 // of the warp's 16 (a_t: stored transposed), b: [k][32 columns].
@@ -325,26 +366,21 @@ __global__ void __launch_bounds__(WALK_THREADS, 1) delta_chunk_walk_kernel(const
     const int op = C * pitch;                                  // bytes of a 64 x D tile
     const uint32_t k_tiles = base + 8 * op, p_tiles = k_tiles + 2 * op, s_tiles = p_tiles + 2 * C * P_PITCH, u_tiles = s_tiles + 2 * D * S_PITCH;
     const uint32_t s_lo = (uint32_t)(D * S_PITCH), u_lo = (uint32_t)(C * S_PITCH);
-    const int pieces = D / 8;                                  // 16-byte pieces of a row
-
-    // tiles [from, from + count) of the operands of a chunk (64 x D each) to `to`
-    auto load_ops = [&](int c, int from, int count, uint32_t to) {
-        const __nv_bfloat16* src = p.ops + ((size_t)(first + c) * H + h) * ops_elems(D) + (size_t)from * C * D;
-        for (int i = threadIdx.x; i < count * C * pieces; i += WALK_THREADS) {
-            const int row = i / pieces, piece = i % pieces;
-            cp_async16(to + row * pitch + piece * 16, src + (size_t)row * D + piece * 8, true);
-        }
+    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + (u_tiles - base) + 2 * C * S_PITCH);       // W and Q (two of them), K and P
+    auto load_first = [&](int c) {                             // by one thread
+        const int buf = c & 1;
+        ph_mbar::arrive_expect_tx(&bars[buf], (uint32_t)first_bytes(D));
+        ph_mbar::bulk_copy(smem + buf * first_bytes(D), p.ops + ((size_t)(first + c) * H + h) * ops_bytes(D), (uint32_t)first_bytes(D), &bars[buf]);
     };
-    auto load_p = [&](int c) {
-        const __nv_bfloat16* src = p.ops + ((size_t)(first + c) * H + h) * ops_elems(D) + 6LL * C * D;
-        for (int i = threadIdx.x; i < 2 * C * (C / 8); i += WALK_THREADS) {
-            const int row = i / (C / 8), piece = i % (C / 8);
-            cp_async16(p_tiles + row * P_PITCH + piece * 16, src + (size_t)row * C + piece * 8, true);
-        }
+    auto load_second = [&](int c) {
+        ph_mbar::arrive_expect_tx(&bars[2], (uint32_t)second_bytes(D));
+        ph_mbar::bulk_copy(smem + 2 * first_bytes(D), p.ops + ((size_t)(first + c) * H + h) * ops_bytes(D) + first_bytes(D), (uint32_t)second_bytes(D), &bars[2]);
     };
-
-    load_ops(0, 0, 4, base);
-    cp_async_commit();
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < 3; ++i) ph_mbar::init(&bars[i], 1);
+        ph_mbar::fence_init();
+        load_first(0);
+    }
     // S: warp w holds the channels 16 w .. 16 w + 15 (rows lane / 4 and + 8), columns nt * 8 + 2 (lane % 4) (+ 1)
     const int nc = (lane & 3) * 2, ch = warp * 16 + (lane >> 2);
     const bool holds = warp < tiles;
@@ -392,13 +428,13 @@ __global__ void __launch_bounds__(WALK_THREADS, 1) delta_chunk_walk_kernel(const
                     u0[nt][half] = col < DV ? *reinterpret_cast<const float2*>(p.u0 + (at * C + r0 + half * 8) * DV + col) : make_float2(0.0f, 0.0f);
                 }
         }
-        cp_async_wait<0>();
-        __syncthreads();                                       // W, Q and S are there; everyone is done with the last chunk's K, P and U
-        load_ops(c, 4, 2, k_tiles);
-        load_p(c);
-        cp_async_commit();
-        if (c + 1 < chunks) load_ops(c + 1, 0, 4, base + ((c + 1) & 1) * 4 * op);
-        cp_async_commit();
+        if (c == 0) __syncthreads();                           // the barriers are set up
+        bool late = !ph_mbar::wait(&bars[c & 1], (c >> 1) & 1, p.error_flag, PH_ERR_WAIT_DELTA);
+        if (__syncthreads_or(late)) return;                    // W, Q and S are there; everyone is done with the last chunk's K, P and U
+        if (threadIdx.x == 0) {
+            load_second(c);
+            if (c + 1 < chunks) load_first(c + 1);
+        }
         // W S for the tokens of warps 0 .. 3, Q S for those of warps 4 .. 7
         const uint32_t a = (outputs ? q_tiles : w_tiles) + rows * 16 * pitch;
         split_product<false>(acc, rest, a, a + op, pitch, s_tiles, s_tiles + s_lo, tiles);
@@ -414,8 +450,11 @@ __global__ void __launch_bounds__(WALK_THREADS, 1) delta_chunk_walk_kernel(const
                     *reinterpret_cast<uint32_t*>(to + u_lo) = lo;
                 }
         }
-        cp_async_wait<1>();
-        __syncthreads();                                       // U, K and P are there; everyone is done with S
+        late = !ph_mbar::wait(&bars[2], c & 1, p.error_flag, PH_ERR_WAIT_DELTA);
+        if (__syncthreads_or(late)) {                          // U, K and P are there; everyone is done with S
+            if (threadIdx.x == 0 && c + 1 < chunks) ph_mbar::wait(&bars[(c + 1) & 1], ((c + 1) >> 1) & 1, p.error_flag, PH_ERR_WAIT_DELTA);
+            return;                                            // (nothing of this block's is in flight any more)
+        }
         if (holds) {
             float sr[NC / 8][4];
 #pragma unroll
@@ -466,7 +505,7 @@ __global__ void __launch_bounds__(WALK_THREADS, 1) delta_chunk_walk_kernel(const
 PH_EXPORT int ph_delta_chunk_supports(int D, int DV) { return D >= 16 && D % 16 == 0 && D <= MAX_DIM && DV >= 2 && DV % 2 == 0; }
 PH_EXPORT int ph_delta_chunk_tokens(void) { return C; }
 // bytes of scratch per (chunk, head): the operands, U0, and the chunk's decay
-PH_EXPORT long long ph_delta_chunk_scratch_bytes(int D, int DV) { return (ops_elems(D) * 2 + 4LL * C * DV + 4LL * D + 255) / 256 * 256; }
+PH_EXPORT long long ph_delta_chunk_scratch_bytes(int D, int DV) { return (ops_bytes(D) + 4LL * C * DV + 4LL * D + 255) / 256 * 256; }
 
 namespace {
 int fill(ChunkParams& p, const int32_t* chunks, int n_chunks, const int32_t* seg_chunks, void* scratch, int H, int G, int D, int DV) {
@@ -478,8 +517,8 @@ int fill(ChunkParams& p, const int32_t* chunks, int n_chunks, const int32_t* seg
     const long long units = (long long)n_chunks * H;
     p.s.H = H; p.s.G = G; p.s.D = D; p.s.DV = DV;
     p.chunks = chunks; p.seg_chunks = seg_chunks;
-    p.ops = static_cast<__nv_bfloat16*>(scratch);
-    p.u0 = reinterpret_cast<float*>(p.ops + units * ops_elems(D));
+    p.ops = static_cast<uint8_t*>(scratch);
+    p.u0 = reinterpret_cast<float*>(p.ops + units * ops_bytes(D));
     p.last = p.u0 + units * C * DV;
     return PH_OK;
 }
@@ -511,13 +550,13 @@ PH_EXPORT int ph_delta_chunk_make(const float* qkv, const float* beta, const flo
 PH_EXPORT int ph_delta_chunk_walk(const void* rows, int rows_dtype, int splits, long long split_stride, long long width, float* state,
                                   long long state_stride, long long conv_at, const int32_t* seg_start, const int32_t* seg_slot, int S,
                                   const int32_t* chunks, int n_chunks, const int32_t* seg_chunks, const void* scratch, int H, int G, int D,
-                                  int DV, int K, float* o, cudaStream_t stream) {
-    if (!rows || !state || !seg_start || !seg_slot || !seg_chunks || !o || S < 1 || K < 1 || splits < 1 || !valid_dtype(rows_dtype) || ((uintptr_t)o & 7))
+                                  int DV, int K, float* o, int* error_flag, cudaStream_t stream) {
+    if (!rows || !state || !seg_start || !seg_slot || !seg_chunks || !o || !error_flag || S < 1 || K < 1 || splits < 1 || !valid_dtype(rows_dtype) || ((uintptr_t)o & 7))
         return fail(PH_ERR_ARG, "delta_chunk_walk: bad arguments (S %d)", S);
     ChunkParams p = {};
     if (int rc = fill(p, chunks, n_chunks, seg_chunks, const_cast<void*>(scratch), H, G, D, DV)) return rc;
     p.s.rows = rows; p.s.splits = splits; p.s.split_stride = split_stride; p.s.width = width; p.s.state = state; p.s.state_stride = state_stride;
-    p.s.conv_at = conv_at; p.s.seg_start = seg_start; p.s.seg_slot = seg_slot; p.s.o = o; p.s.K = K;
+    p.s.conv_at = conv_at; p.s.seg_start = seg_start; p.s.seg_slot = seg_slot; p.s.o = o; p.s.K = K; p.error_flag = error_flag;
     p.rows_bf16 = rows_dtype == PH_BF16;
     const size_t smem = (size_t)walk_smem(D);
     static size_t set = 0;

@@ -28,6 +28,7 @@ using namespace ph;
 
 constexpr int PREP_WARPS = 8;
 constexpr int TAIL = 128;               // elements of a tail unit
+constexpr int RUN = 8;                  // tokens that a warp walks where there are many rows
 constexpr float UNIT_EPS = 1e-6f;
 
 struct PrepParams {
@@ -138,8 +139,12 @@ __device__ __forceinline__ void conv_run(const PrepParams& p, int t0, int count,
         return v;
     };
     int seg = -1;
-    float4 next = input(t0);
-    for (int r = 0; r < count; ++r) {
+    float4 own[RUN];                                       // all of the run's rows on their way at once
+#pragma unroll
+    for (int r = 0; r < RUN; ++r) own[r] = r < count ? input(t0 + r) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+    for (int r = 0; r < RUN; ++r) {
+        if (r >= count) break;
         const int t = t0 + r, s = p.row_seg[t];
         if (s != seg) {                                    // the run's first row, or another request's
             seg = s;
@@ -151,8 +156,7 @@ __device__ __forceinline__ void conv_run(const PrepParams& p, int t0, int count,
                 x[j] = src >= 0 ? input(first + src) : on ? load4(past + (size_t)(src + KT - 1) * CH + c0 + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             }
         }
-        x[KT - 1] = next;
-        if (r + 1 < count) next = input(t + 1);
+        x[KT - 1] = own[r];
         float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
         for (int j = 0; j < KT; ++j) {
@@ -201,25 +205,25 @@ __global__ void __launch_bounds__(PREP_WARPS * 32, 2) delta_prepare_kernel(const
         return;
     }
     unit -= p.H;
-    for (int t = t0; t < t0 + count; ++t) {
-        const TI* row = static_cast<const TI*>(p.rows) + (size_t)t * p.width;
-        auto value = [&](int c) {
-            float v = to_float<TI>(row[c]);
-            for (int s = 1; s < p.splits; ++s) v += to_float<TI>(row[(size_t)s * p.split_stride + c]);
-            return v;
-        };
-        // the tail: [beta | decay | low rows | gate], TAIL elements per warp
-        const int nb = p.H, na = p.a_col >= 0 ? p.H : 0, all = nb + na + p.low_n + p.gate_n;
-        for (int e = unit * TAIL + lane; e < min(all, (unit + 1) * TAIL); e += 32) {
-            int i = e;
-            if (i < nb) { p.beta[(size_t)t * p.H + i] = 1.0f / (1.0f + expf(-value(p.b_col + i))); continue; }
-            i -= nb;
-            if (i < na) { p.log_decay[(size_t)t * p.H + i] = p.rate[i] * ph_delta::softplus(value(p.a_col + i) + p.a_bias[i]); continue; }
-            i -= na;
-            if (i < p.low_n) { static_cast<TO*>(p.low)[(size_t)t * p.low_n + i] = from_float<TO>(value(p.low_col + i)); continue; }
-            i -= p.low_n;
-            static_cast<TO*>(p.gate)[(size_t)t * p.gate_n + i] = from_float<TO>(value(p.gate_col + i));
-        }
+    // the tail of one of the run's tokens: [beta | decay | low rows | gate], TAIL elements per warp
+    const int t = t0 + unit % run;
+    unit /= run;
+    if (t >= T) return;
+    const TI* row = static_cast<const TI*>(p.rows) + (size_t)t * p.width;
+    const int nb = p.H, na = p.a_col >= 0 ? p.H : 0, all = nb + na + p.low_n + p.gate_n;
+#pragma unroll
+    for (int k = 0; k < TAIL / 32; ++k) {
+        int i = unit * TAIL + k * 32 + lane;
+        if (i >= all) break;
+        const int which = i < nb ? 0 : i < nb + na ? 1 : i < nb + na + p.low_n ? 2 : 3;
+        i -= which == 0 ? 0 : which == 1 ? nb : which == 2 ? nb + na : nb + na + p.low_n;
+        const TI* from = row + i + (which == 0 ? p.b_col : which == 1 ? p.a_col : which == 2 ? p.low_col : p.gate_col);
+        float v = to_float<TI>(*from);
+        for (int s = 1; s < p.splits; ++s) v += to_float<TI>(from[(size_t)s * p.split_stride]);
+        if (which == 0) p.beta[(size_t)t * p.H + i] = 1.0f / (1.0f + expf(-v));
+        else if (which == 1) p.log_decay[(size_t)t * p.H + i] = p.rate[i] * ph_delta::softplus(v + p.a_bias[i]);
+        else if (which == 2) static_cast<TO*>(p.low)[(size_t)t * p.low_n + i] = from_float<TO>(v);
+        else static_cast<TO*>(p.gate)[(size_t)t * p.gate_n + i] = from_float<TO>(v);
     }
 }
 
@@ -398,8 +402,8 @@ PH_EXPORT int ph_delta_prepare(const void* rows, int rows_dtype, int splits, lon
     lanes_for(D, vec && D % 4 == 0, &p.qk_v, &p.qk_n);
     lanes_for(DV, vec && DV % 4 == 0 && (2LL * G * D) % 4 == 0, &p.v_v, &p.v_n);
     if (D > 512 || DV > 512) return fail(PH_ERR_UNSUPPORTED, "delta_prepare: heads of %d / %d exceed the supported 512", D, DV);
-    const int tail = H + (a_col >= 0 ? H : 0) + low_n + gate_n, units = 2 * G + H + (tail + TAIL - 1) / TAIL;
-    const int run = T >= 512 ? 8 : 1;              // many rows: a warp walks several tokens
+    const int tail = H + (a_col >= 0 ? H : 0) + low_n + gate_n, run = T >= 512 ? RUN : 1;
+    const int units = 2 * G + H + (tail + TAIL - 1) / TAIL * run;
     const dim3 grid((T + run - 1) / run, (units + PREP_WARPS - 1) / PREP_WARPS);
     PH_DISPATCH(rows_dtype, TI, PH_DISPATCH(model_dtype, TO,
         launch_overlapped(delta_prepare_kernel<TI, TO>, grid, dim3(PREP_WARPS * 32), 0, stream, p, T, run)));

@@ -218,7 +218,7 @@ struct CoreKernels {
     int (*delta_chunk_make)(const float*, const float*, const float*, const float*, long long, const float*, const float*, const int32_t*, int,
                             void*, int, int, int, int, cudaStream_t);
     int (*delta_chunk_walk)(const void*, int, int, long long, long long, float*, long long, long long, const int32_t*, const int32_t*, int,
-                            const int32_t*, int, const int32_t*, const void*, int, int, int, int, int, float*, cudaStream_t);
+                            const int32_t*, int, const int32_t*, const void*, int, int, int, int, int, float*, int*, cudaStream_t);
     int (*delta_chunk_supports)(int, int);
     int (*delta_chunk_tokens)(void);
     long long (*delta_chunk_scratch_bytes)(int, int);

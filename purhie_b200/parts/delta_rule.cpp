@@ -275,7 +275,7 @@ public:
                                                (double)rows_long * heads_ * vdim_ * (6.0 * dim_ + 64.0));
             QE_LAUNCH(k, k.delta_chunk_walk(in.tensor.data, in.tensor.code(), in.splits, split_stride, width_, state, state_floats(), conv_at(),
                                             ctx.seg_start, ctx.seg_slot, ctx.S, chunks.data, n_chunks, seg_chunks.data, scratch.data, heads_,
-                                            kv_heads_, dim_, vdim_, taps_, o.as<float>(), ctx.stream));
+                                            kv_heads_, dim_, vdim_, taps_, o.as<float>(), ctx.gemm_error, ctx.stream));
         }
         if (n_long < ctx.S) {
             note(ctx.S - n_long, T - rows_long);
