@@ -15,9 +15,11 @@
 //                      columns J come from k exp(g), q exp(g), k exp(t_J - g) (never above 1) and one factor per channel and
 //                      pair of blocks, the decay between them; on the diagonal that factor is exp(-t_I), and where it would
 //                      exceed 2^60 the block takes every pair's exponential itself.  Float32 on packed multiply-adds, 2 x 2
-//                      pairs per thread.  The system is solved by forward substitution in float32, a column per thread, by half
-//                      of the warps while the others write the operands.  W, q exp(G), k exp(G_last - G) and P leave as two
-//                      bfloat16 each, the rounded value and the rounded rest, in the layout of the walk's shared memory.
+//                      pairs per thread.  M = (1 + diag(beta) A)^-1 in float32, block by block: the diagonal blocks by forward
+//                      substitution, M_IJ = -M_II sum_K (diag(beta) A)_IK M_KJ below them, one distance from the diagonal
+//                      after the other.  W and U0 are M diag(beta) times k exp(G) and V on the tensor cores, split operands as
+//                      in the walk.  W, q exp(G), k exp(G_last - G) and P leave as two bfloat16 each, the rounded value and the
+//                      rounded rest, in the layout of the walk's shared memory.
 //   delta_chunk_walk   a block per (request, head, 32 columns of S) that walks the request's chunks in order with S in registers
 //                      (float32, spread over its eight warps) and, split the same way, in shared memory.  Every product is three
 //                      tensor-core products of the split operands, so 16 bits of every factor count, and the sums are float32.
@@ -62,6 +64,13 @@ __host__ __device__ constexpr int first_bytes(int D) { return 4 * C * op_pitch(D
 __host__ __device__ constexpr int second_bytes(int D) { return 2 * C * op_pitch(D) + 2 * C * P_PITCH; }    // K and P
 __host__ __device__ constexpr long long ops_bytes(int D) { return first_bytes(D) + second_bytes(D); }
 
+// log(1 + exp(v)) from the hardware's exponential and logarithm; where exp(-|v|) is small its series, so that slow decays keep
+// their relative precision
+__device__ __forceinline__ float fast_softplus(float v) {
+    const float e = __expf(-fabsf(v));
+    const float l = e < 0.01f ? e * (1.0f - e * (0.5f - e * (1.0f / 3.0f))) : __logf(1.0f + e);
+    return l + fmaxf(v, 0.0f);
+}
 __device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
     float2 d;
@@ -87,10 +96,15 @@ __device__ __forceinline__ void split2(float u, float v, uint32_t& hi, uint32_t&
     lo = pack_bf16(u - __uint_as_float(hi << 16), v - __uint_as_float(hi & 0xffff0000u));
 }
 
-// floats of shared memory of delta_chunk_make: k exp(g), q exp(g), k exp(t - g) and g [64][D + 4], the system and P [64][64 + 4],
-// the running sums at the blocks' starts [5][D], the factors between blocks [10][D], beta [64]
-__host__ __device__ constexpr int make_floats(int D) { return 4 * C * (D + 4) + 2 * C * (C + 4) + 15 * D + C; }
 constexpr int BLOCKS = C / RB;
+constexpr int YP = RB + 1;
+// floats of shared memory of delta_chunk_make: k exp(g), q exp(g), k exp(t - g) and g [64][D + 4], the system, P and the inverse
+// [64][64 + 4], the running sums at the blocks' starts [5][D], the factors between blocks [10][D], beta [64], three blocks of
+// 16 x 16.  Once the operands are written, the tensor cores' tiles of k exp(G) and V take the place of the second to fourth,
+// and the inverse's that of the system and P.
+__host__ __device__ constexpr int make_floats(int D) { return 4 * C * (D + 4) + 3 * C * (C + 4) + 15 * D + C + 3 * RB * YP; }
+// columns of V that fit there at a time
+__host__ __device__ constexpr int v_group(int D) { return (2 * D - 4) / 16 * 16; }
 
 __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const ChunkParams p) {
     extern __shared__ __align__(16) float sm[];
@@ -101,11 +115,13 @@ __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const
     float* qd = kd + C * DP;           // q exp(g)
     float* ke = qd + C * DP;           // k exp(t - g)
     float* gs = ke + C * DP;           // g, in units of log2 (as every logarithm here)
-    float* N = gs + C * DP;            // [64][NP]: -diag(beta) A
+    float* N = gs + C * DP;            // [64][NP]: diag(beta) A
     float* P = N + C * NP;
-    float* base = P + C * NP;          // [5][D]: G at the start of each block, and at the chunk's end
+    float* M = P + C * NP;             // (1 + N)^-1
+    float* base = M + C * NP;          // [5][D]: G at the start of each block, and at the chunk's end
     float* F = base + 5 * D;           // [10][D]
     float* beta = F + 10 * D;
+    float* Y = beta + C;               // [3][16][YP]
     const int tid = threadIdx.x, item = blockIdx.x, h = blockIdx.y, g = h / (H / p.s.G);
     pdl_launch_dependents();
     pdl_wait();
@@ -117,7 +133,7 @@ __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const
     // ---- the running sums inside the blocks: a thread per (channel, block)
     if (tid < BLOCKS) slow[tid] = 0;
     if (tid < C) beta[tid] = tid < n ? p.s.beta[(size_t)(row0 + tid) * H + h] : 0.0f;
-    for (int i = tid; i < C * NP; i += MAKE_THREADS) { N[i] = 0.0f; P[i] = 0.0f; }
+    for (int i = tid; i < C * NP; i += MAKE_THREADS) { N[i] = 0.0f; P[i] = 0.0f; M[i] = 0.0f; }
     if (tid < BLOCKS * D) {
         const int d = tid % D, J = tid / D;
         float run = 0.0f, x[RB];
@@ -127,7 +143,7 @@ __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const
 #pragma unroll
             for (int t = 0; t < RB; ++t) x[t] = J * RB + t < n ? z[(size_t)(J * RB + t) * p.s.z_stride] : 0.0f;
 #pragma unroll
-            for (int t = 0; t < RB; ++t) x[t] = J * RB + t < n ? rate * ph_delta::softplus(x[t] + bias) : 0.0f;
+            for (int t = 0; t < RB; ++t) x[t] = J * RB + t < n ? rate * fast_softplus(x[t] + bias) : 0.0f;
         } else {
             const float* ld = p.s.log_decay + (size_t)row0 * H + h;
 #pragma unroll
@@ -227,7 +243,7 @@ __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const
 #pragma unroll
             for (int v = 0; v < 2; ++v) {
                 const int r = i0 + 8 * u, c = j0 + 8 * v;
-                if (c < r) N[r * NP + c] = -beta[r] * a[u][v];
+                if (c < r) N[r * NP + c] = beta[r] * a[u][v];
                 if (c <= r) P[r * NP + c] = b[u][v];
             }
     }
@@ -236,58 +252,21 @@ __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const
     const size_t at = (size_t)item * H + h;
     uint8_t* ops = p.ops + at * ops_bytes(D);
     const int pitch = op_pitch(D), op = C * pitch;
-    constexpr int HALF = MAKE_THREADS / 2;
-    if (tid < HALF) {
-        // ---- the system, a column of [W | U0] per thread; two neighbouring rows of it in a register pair
-        float* u0 = p.u0 + at * C * DV;
-        for (int c0 = 0; c0 < D + DV; c0 += HALF) {
-            const int c = c0 + tid;                        // (D is even: a pair of lanes is in W or in U0)
-            const bool is_w = c < D, on = c < D + DV;
-            float2 x[C / 2];
-            float first[BLOCKS];
+    if (tid < C) {
+        // ---- the inverse's diagonal blocks, a column per thread
+        const int J = tid / RB, c = tid % RB;
+        float m[RB];
 #pragma unroll
-            for (int J = 0; J < BLOCKS; ++J) first[J] = is_w ? ex2(base[J * D + c]) : 0.0f;
-            const float* v = rows + 2 * p.s.G * D + (size_t)h * DV + (c - D);
+        for (int i = 0; i < RB; ++i) {
+            float sum = 0.0f;
 #pragma unroll
-            for (int i = 0; i < C; i += 2) {
-                float r0 = 0.0f, r1 = 0.0f;
-                if (is_w) {
-                    r0 = kd[i * DP + c] * first[i / RB];
-                    r1 = kd[(i + 1) * DP + c] * first[i / RB];
-                } else if (on) {
-                    if (i < n) r0 = v[(size_t)i * CH];
-                    if (i + 1 < n) r1 = v[(size_t)(i + 1) * CH];
-                }
-                x[i / 2] = make_float2(r0 * beta[i], r1 * beta[i + 1]);
-            }
-#pragma unroll
-            for (int i = 1; i < C; ++i) {
-                float2 even = make_float2(0.0f, 0.0f), odd = even;
-#pragma unroll
-                for (int j = 0; j < i; j += 4) {                       // (N is zero from column i on)
-                    const float4 m = load4(N + i * NP + j);
-                    even = fma2(make_float2(m.x, m.y), x[j / 2], even);
-                    if (j + 2 < i) odd = fma2(make_float2(m.z, m.w), x[j / 2 + 1], odd);
-                }
-                const float sum = (even.x + odd.x) + (even.y + odd.y);
-                if (i & 1) x[i / 2].y += sum; else x[i / 2].x += sum;
-            }
-#pragma unroll
-            for (int i = 0; i < C; ++i) {
-                const float own = i & 1 ? x[i / 2].y : x[i / 2].x;
-                const float other = __shfl_xor_sync(0xffffffffu, own, 1);
-                if (is_w) {                                            // the even lane stores the rounded pair, the odd one the rests
-                    uint32_t hi, lo;
-                    if (c & 1) split2(other, own, hi, lo); else split2(own, other, hi, lo);
-                    *reinterpret_cast<uint32_t*>(ops + (c & 1) * op + i * pitch + (c & ~1) * 2) = c & 1 ? lo : hi;
-                } else if (on) {
-                    u0[(size_t)i * DV + (c - D)] = own;
-                }
-            }
+            for (int j = 0; j < i; ++j) sum = fmaf(N[(J * RB + i) * NP + J * RB + j], m[j], sum);
+            m[i] = i == c ? 1.0f : i > c ? -sum : 0.0f;
+            M[(J * RB + i) * NP + J * RB + c] = m[i];
         }
     } else {
-        // ---- the other operands
-        const int w = tid - HALF;
+        // ---- the operands that need no inverse
+        const int w = tid - C, step = MAKE_THREADS - C;
         auto put = [&](uint8_t* to, int rest, float4 v) {              // four elements, the rests `rest` bytes behind
             uint32_t h0, l0, h1, l1;
             split2(v.x, v.y, h0, l0);
@@ -295,7 +274,7 @@ __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const
             *reinterpret_cast<uint2*>(to) = make_uint2(h0, h1);
             *reinterpret_cast<uint2*>(to + rest) = make_uint2(l0, l1);
         };
-        for (int e = w; e < C * per_row; e += HALF) {
+        for (int e = w; e < C * per_row; e += step) {
             const int i = e / per_row, d = (e - i * per_row) * 4, J = i / RB;
             const float4 q4 = load4(qd + i * DP + d), k4 = load4(ke + i * DP + d);
             const float4 b4 = load4(base + J * D + d), n4 = load4(base + (J + 1) * D + d), l4 = load4(base + BLOCKS * D + d);
@@ -303,11 +282,115 @@ __global__ void __launch_bounds__(MAKE_THREADS, 1) delta_chunk_make_kernel(const
             put(to, op, make_float4(q4.x * ex2(b4.x), q4.y * ex2(b4.y), q4.z * ex2(b4.z), q4.w * ex2(b4.w)));
             put(to + 2 * op, op, make_float4(k4.x * ex2(l4.x - n4.x), k4.y * ex2(l4.y - n4.y), k4.z * ex2(l4.z - n4.z), k4.w * ex2(l4.w - n4.w)));
         }
-        for (int e = w; e < C * C / 4; e += HALF) {
+        for (int e = w; e < C * C / 4; e += step) {
             const int i = e / (C / 4), j = e % (C / 4) * 4;
             put(ops + 6 * op + i * P_PITCH + j * 2, C * P_PITCH, load4(P + i * NP + j));
         }
-        for (int d = w; d < D; d += HALF) p.last[at * D + d] = ex2(base[BLOCKS * D + d]);
+        for (int d = w; d < D; d += step) p.last[at * D + d] = ex2(base[BLOCKS * D + d]);
+    }
+    __syncthreads();
+    // ---- the blocks below, `apart` blocks from the diagonal
+    for (int apart = 1; apart < BLOCKS; ++apart) {
+        for (int e = tid; e < (BLOCKS - apart) * RB * RB; e += MAKE_THREADS) {
+            const int J = e / (RB * RB), I = J + apart, i = e / RB % RB, j = e % RB;
+            const float* nr = N + (I * RB + i) * NP;
+            float sum = 0.0f;
+            for (int k = J * RB; k < I * RB; k += 4) {
+                const float4 a = load4(nr + k);
+                const float* mc = M + k * NP + J * RB + j;
+                sum = fmaf(a.x, mc[0], sum); sum = fmaf(a.y, mc[NP], sum); sum = fmaf(a.z, mc[2 * NP], sum); sum = fmaf(a.w, mc[3 * NP], sum);
+            }
+            Y[(J * RB + i) * YP + j] = sum;
+        }
+        __syncthreads();
+        for (int e = tid; e < (BLOCKS - apart) * RB * RB; e += MAKE_THREADS) {
+            const int J = e / (RB * RB), I = J + apart, i = e / RB % RB, j = e % RB;
+            const float* mr = M + (I * RB + i) * NP + I * RB;
+            float sum = 0.0f;
+#pragma unroll
+            for (int k = 0; k < RB; ++k) sum = fmaf(mr[k], Y[(J * RB + k) * YP + j], sum);
+            M[(I * RB + i) * NP + J * RB + j] = -sum;
+        }
+        __syncthreads();
+    }
+    // ---- [W | U0] = M diag(beta) [k exp(G) | V] on the tensor cores
+    uint8_t* t_tile = reinterpret_cast<uint8_t*>(N);                  // [hi, lo][64][P_PITCH]
+    uint8_t* k_tile = reinterpret_cast<uint8_t*>(qd);                 // [hi, lo][64][pitch]
+    uint8_t* v_tile = k_tile + 2 * op;                                // [hi, lo][64][v_pitch]
+    const int group = min(v_group(D), (DV + 15) / 16 * 16), v_pitch = op_pitch(group);
+    auto tile4 = [&](uint8_t* to, int rest, float4 v) {
+        uint32_t h0, l0, h1, l1;
+        split2(v.x, v.y, h0, l0);
+        split2(v.z, v.w, h1, l1);
+        *reinterpret_cast<uint2*>(to) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2*>(to + rest) = make_uint2(l0, l1);
+    };
+    for (int e = tid; e < C * C / 4; e += MAKE_THREADS) {
+        const int i = e / (C / 4), j = e % (C / 4) * 4;
+        const float4 m = load4(M + i * NP + j), b4 = load4(beta + j);
+        tile4(t_tile + i * P_PITCH + j * 2, C * P_PITCH, make_float4(m.x * b4.x, m.y * b4.y, m.z * b4.z, m.w * b4.w));
+    }
+    for (int e = tid; e < C * per_row; e += MAKE_THREADS) {
+        const int i = e / per_row, d = (e - i * per_row) * 4;
+        const float4 k4 = load4(kd + i * DP + d), b4 = load4(base + i / RB * D + d);
+        tile4(k_tile + i * pitch + d * 2, op, make_float4(k4.x * ex2(b4.x), k4.y * ex2(b4.y), k4.z * ex2(b4.z), k4.w * ex2(b4.w)));
+    }
+    float* u0 = p.u0 + at * C * DV;
+    const float* v_rows = rows + 2 * p.s.G * D + (size_t)h * DV;
+    const int row_tile = warp & 3, r0 = row_tile * 16 + (lane >> 2), nc = (lane & 3) * 2;
+    const uint32_t ta = smem_u32(t_tile) + (row_tile * 16 + (lane & 15)) * P_PITCH + (lane >> 4) * 16;
+    for (int v0 = 0; v0 < DV; v0 += group) {
+        const int quads = group / 4;
+        for (int e = tid; e < C * quads; e += MAKE_THREADS) {
+            const int i = e / quads, c = (e - i * quads) * 4;
+            float x[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+            for (int u = 0; u < 4; ++u)
+                if (i < n && v0 + c + u < DV) x[u] = v_rows[(size_t)i * CH + v0 + c + u];
+            tile4(v_tile + i * v_pitch + c * 2, C * v_pitch, make_float4(x[0], x[1], x[2], x[3]));
+        }
+        __syncthreads();
+        const int w_tiles = v0 == 0 ? D / 16 : 0, all = w_tiles + group / 16;
+        for (int ct = warp >> 2; ct < all; ct += MAKE_THREADS / 128) {
+            const bool is_w = ct < w_tiles;
+            const int col = (is_w ? ct : ct - w_tiles) * 16, bp = is_w ? pitch : v_pitch;
+            const uint32_t b_hi = smem_u32(is_w ? k_tile : v_tile) + col * 2, b_lo = b_hi + C * bp;
+            float acc[2][4], rest[2][4];
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) acc[u][i] = rest[u][i] = 0.0f;
+            for (int ks = 0; ks <= row_tile; ++ks) {                  // M is lower triangular
+                uint32_t a[4], l[4], b0, b1, b2, b3, c0, c1, c2, c3;
+                ldmatrix_x4(ta + ks * 32, a[0], a[1], a[2], a[3]);
+                ldmatrix_x4(ta + C * P_PITCH + ks * 32, l[0], l[1], l[2], l[3]);
+                const int from = (ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * bp + (lane >> 4) * 16;
+                ldmatrix_x4_trans(b_hi + from, b0, b1, b2, b3);
+                ldmatrix_x4_trans(b_lo + from, c0, c1, c2, c3);
+                mma_bf16(acc[0], a[0], a[1], a[2], a[3], b0, b1);
+                mma_bf16(acc[1], a[0], a[1], a[2], a[3], b2, b3);
+                mma_bf16(rest[0], l[0], l[1], l[2], l[3], b0, b1);
+                mma_bf16(rest[1], l[0], l[1], l[2], l[3], b2, b3);
+                mma_bf16(rest[0], a[0], a[1], a[2], a[3], c0, c1);
+                mma_bf16(rest[1], a[0], a[1], a[2], a[3], c2, c3);
+            }
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int i = r0 + half * 8, c = col + u * 8 + nc;
+                    const float x = acc[u][2 * half] + rest[u][2 * half], y = acc[u][2 * half + 1] + rest[u][2 * half + 1];
+                    if (is_w) {
+                        uint32_t hi, lo;
+                        split2(x, y, hi, lo);
+                        *reinterpret_cast<uint32_t*>(ops + i * pitch + c * 2) = hi;
+                        *reinterpret_cast<uint32_t*>(ops + op + i * pitch + c * 2) = lo;
+                    } else if (v0 + c < DV) {                         // DV is even: a pair is inside or outside
+                        *reinterpret_cast<float2*>(u0 + (size_t)i * DV + v0 + c) = make_float2(x, y);
+                    }
+                }
+        }
+        if (v0 + group < DV) __syncthreads();                          // the tile is read before the next columns take its place
     }
 }
 

@@ -28,7 +28,8 @@ using namespace ph;
 
 constexpr int PREP_WARPS = 8;
 constexpr int TAIL = 128;               // elements of a tail unit
-constexpr int RUN = 8;                  // tokens that a warp walks where there are many rows
+constexpr int RUN = 8;                  // tokens that a warp walks where there are many rows (RUN_FROM of them)
+constexpr int RUN_FROM = 256;
 constexpr float UNIT_EPS = 1e-6f;
 
 struct PrepParams {
@@ -117,103 +118,73 @@ __device__ __forceinline__ void conv_any(const PrepParams& p, int t, int kind, i
     }
 }
 
-// The same for the tokens t0 .. t0 + count - 1 with the last KT inputs in registers, so that a row is read once: heads of up to
-// 128 channels, four per lane.  The order of each sum is the one above.
-template <typename TI, int KT>
-__device__ __forceinline__ void conv_run(const PrepParams& p, int t0, int count, int kind, int c0, int n) {
+// silu; in a bfloat16 model from the hardware's exponential and reciprocal, still float32 (relative error about 1e-6)
+template <bool FAST> __device__ __forceinline__ float silu(float v) { return FAST ? __fdividef(v, 1.0f + __expf(-v)) : v / (1.0f + expf(-v)); }
+
+// The same for the tokens t .. t_end - 1 with the last KT inputs in registers, so that a row is read once, R rows on their
+// way at a time: heads of up to 128 channels, four per lane.  The order of each sum is the one above.
+template <typename TI, int KT, bool FAST, int R>
+__device__ __forceinline__ void conv_run(const PrepParams& p, int t, int t_end, int kind, int c0, int n) {
     const int lane = threadIdx.x & 31, d = lane * 4, CH = 2 * p.G * p.D + p.H * p.DV;
     const bool on = d < n;
-    const TI* rows = static_cast<const TI*>(p.rows);
-    float4 w[KT], x[KT];
+    const float4 none = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    const TI* rows = static_cast<const TI*>(p.rows) + c0 + d;
+    float4 w[KT], x[KT + R - 1];
 #pragma unroll
-    for (int j = 0; j < KT; ++j) w[j] = on ? load4(p.taps + (size_t)j * CH + c0 + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int j = 0; j < KT; ++j) w[j] = on ? load4(p.taps + (size_t)j * CH + c0 + d) : none;
     auto input = [&](int row) {
-        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (!on) return v;
-        const TI* at = rows + (size_t)row * p.width + c0 + d;
-        v = load4(at);
+        if (!on) return none;
+        float4 v = load4(rows + (size_t)row * p.width);
         for (int sp = 1; sp < p.splits; ++sp) {
-            const float4 m = load4(at + (size_t)sp * p.split_stride);
+            const float4 m = load4(rows + (size_t)row * p.width + (size_t)sp * p.split_stride);
             v.x += m.x; v.y += m.y; v.z += m.z; v.w += m.w;
         }
         return v;
     };
-    int seg = -1;
-    float4 own[RUN];                                       // all of the run's rows on their way at once
+    while (t < t_end) {
+        const int s = p.row_seg[t], first = p.seg_start[s], stop = min(t_end, p.seg_start[s + 1]);
+        const float* past = p.state + (size_t)p.seg_slot[s] * p.state_stride + p.conv_at + c0 + d;
 #pragma unroll
-    for (int r = 0; r < RUN; ++r) own[r] = r < count ? input(t0 + r) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (int j = 0; j < KT - 1; ++j) {
+            const int src = t - first - (KT - 1) + j;
+            x[j] = src >= 0 ? input(first + src) : on ? load4(past + (size_t)(src + KT - 1) * CH) : none;
+        }
+        for (; t < stop; t += R) {
 #pragma unroll
-    for (int r = 0; r < RUN; ++r) {
-        if (r >= count) break;
-        const int t = t0 + r, s = p.row_seg[t];
-        if (s != seg) {                                    // the run's first row, or another request's
-            seg = s;
-            const int first = p.seg_start[s], i0 = t - first;
-            const float* past = p.state + (size_t)p.seg_slot[s] * p.state_stride + p.conv_at;
+            for (int r = 0; r < R; ++r) x[KT - 1 + r] = t + r < stop ? input(t + r) : none;
 #pragma unroll
-            for (int j = 0; j < KT - 1; ++j) {
-                const int src = i0 - (KT - 1) + j;
-                x[j] = src >= 0 ? input(first + src) : on ? load4(past + (size_t)(src + KT - 1) * CH + c0 + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            for (int r = 0; r < R; ++r) {
+                float4 y = none;
+#pragma unroll
+                for (int j = 0; j < KT; ++j) {
+                    y.x = fmaf(w[j].x, x[r + j].x, y.x); y.y = fmaf(w[j].y, x[r + j].y, y.y);
+                    y.z = fmaf(w[j].z, x[r + j].z, y.z); y.w = fmaf(w[j].w, x[r + j].w, y.w);
+                }
+                y.x = silu<FAST>(y.x); y.y = silu<FAST>(y.y); y.z = silu<FAST>(y.z); y.w = silu<FAST>(y.w);
+                float f = 1.0f;
+                if (kind < 2) {
+                    float ss = 0.0f;
+                    ss += y.x * y.x; ss += y.y * y.y; ss += y.z * y.z; ss += y.w * y.w;
+                    f = rsqrtf(warp_sum(ss) + UNIT_EPS) * (kind == 0 ? p.q_scale : 1.0f);
+                }
+                if (on && t + r < stop)
+                    *reinterpret_cast<float4*>(p.qkv + (size_t)(t + r) * CH + c0 + d) = make_float4(y.x * f, y.y * f, y.z * f, y.w * f);
             }
-        }
-        x[KT - 1] = own[r];
-        float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
-        for (int j = 0; j < KT; ++j) {
-            y.x = fmaf(w[j].x, x[j].x, y.x); y.y = fmaf(w[j].y, x[j].y, y.y);
-            y.z = fmaf(w[j].z, x[j].z, y.z); y.w = fmaf(w[j].w, x[j].w, y.w);
+            for (int j = 0; j < KT - 1; ++j) x[j] = x[j + R];
         }
-#pragma unroll
-        for (int j = 0; j < KT - 1; ++j) x[j] = x[j + 1];
-        y.x = y.x / (1.0f + expf(-y.x)); y.y = y.y / (1.0f + expf(-y.y)); y.z = y.z / (1.0f + expf(-y.z)); y.w = y.w / (1.0f + expf(-y.w));
-        float f = 1.0f;
-        if (kind < 2) {
-            float ss = 0.0f;
-            ss += y.x * y.x; ss += y.y * y.y; ss += y.z * y.z; ss += y.w * y.w;
-            f = rsqrtf(warp_sum(ss) + UNIT_EPS) * (kind == 0 ? p.q_scale : 1.0f);
-        }
-        if (on) *reinterpret_cast<float4*>(p.qkv + (size_t)t * CH + c0 + d) = make_float4(y.x * f, y.y * f, y.z * f, y.w * f);
+        t = stop;
     }
 }
 
-template <typename TI>
-__device__ __forceinline__ void conv_tokens(const PrepParams& p, int t0, int count, int kind, int c0, int n, int v, int ni) {
-    if (count > 1 && v == 4 && ni == 1 && p.K >= 2 && p.K <= 4) {
-        if (p.K == 2) conv_run<TI, 2>(p, t0, count, kind, c0, n);
-        else if (p.K == 3) conv_run<TI, 3>(p, t0, count, kind, c0, n);
-        else conv_run<TI, 4>(p, t0, count, kind, c0, n);
-        return;
-    }
-    for (int r = 0; r < count; ++r) conv_any<TI>(p, t0 + r, kind, c0, n, v, ni);
-}
-
-// TI: the dtype of the rows; TO: the model's dtype (rows in parts are float32 in a bfloat16 model)
+// The tail of a token's row, [beta | decay | low rows | gate]: TAIL elements by a warp.  TO: the model's dtype.
 template <typename TI, typename TO>
-__global__ void __launch_bounds__(PREP_WARPS * 32, 2) delta_prepare_kernel(const PrepParams p, int T, int run) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const int t0 = blockIdx.x * run, count = min(run, T - t0), lane = threadIdx.x & 31;
-    int unit = blockIdx.y * PREP_WARPS + (threadIdx.x >> 5);
-    const int QK = 2 * p.G * p.D;
-    if (unit < 2 * p.G) {
-        conv_tokens<TI>(p, t0, count, unit < p.G ? 0 : 1, unit * p.D, p.D, p.qk_v, p.qk_n);
-        return;
-    }
-    unit -= 2 * p.G;
-    if (unit < p.H) {
-        conv_tokens<TI>(p, t0, count, 2, QK + unit * p.DV, p.DV, p.v_v, p.v_n);
-        return;
-    }
-    unit -= p.H;
-    // the tail of one of the run's tokens: [beta | decay | low rows | gate], TAIL elements per warp
-    const int t = t0 + unit % run;
-    unit /= run;
-    if (t >= T) return;
+__device__ __forceinline__ void finish_tail(const PrepParams& p, int t, int part) {
     const TI* row = static_cast<const TI*>(p.rows) + (size_t)t * p.width;
     const int nb = p.H, na = p.a_col >= 0 ? p.H : 0, all = nb + na + p.low_n + p.gate_n;
 #pragma unroll
     for (int k = 0; k < TAIL / 32; ++k) {
-        int i = unit * TAIL + k * 32 + lane;
+        int i = part * TAIL + k * 32 + (threadIdx.x & 31);
         if (i >= all) break;
         const int which = i < nb ? 0 : i < nb + na ? 1 : i < nb + na + p.low_n ? 2 : 3;
         i -= which == 0 ? 0 : which == 1 ? nb : which == 2 ? nb + na : nb + na + p.low_n;
@@ -225,6 +196,44 @@ __global__ void __launch_bounds__(PREP_WARPS * 32, 2) delta_prepare_kernel(const
         else if (which == 2) static_cast<TO*>(p.low)[(size_t)t * p.low_n + i] = from_float<TO>(v);
         else static_cast<TO*>(p.gate)[(size_t)t * p.gate_n + i] = from_float<TO>(v);
     }
+}
+
+// TI: the dtype of the rows (rows in parts are float32 in a bfloat16 model too)
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(PREP_WARPS * 32, 2) delta_prepare_kernel(const PrepParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    int unit = blockIdx.y * PREP_WARPS + (threadIdx.x >> 5);
+    if (unit < 2 * p.G) {
+        conv_any<TI>(p, t, unit < p.G ? 0 : 1, unit * p.D, p.D, p.qk_v, p.qk_n);
+        return;
+    }
+    unit -= 2 * p.G;
+    if (unit < p.H) {
+        conv_any<TI>(p, t, 2, 2 * p.G * p.D + unit * p.DV, p.DV, p.v_v, p.v_n);
+        return;
+    }
+    finish_tail<TI, TO>(p, t, unit - p.H);
+}
+
+// The form for the usual heads and taps: a warp per (`run` tokens, head), and per (token, part of the tail).
+template <typename TI, typename TO, int KT, int R>
+__global__ void __launch_bounds__(PREP_WARPS * 32, 3) delta_prepare_run_kernel(const PrepParams p, int T) {
+    constexpr int run = R == 1 ? 1 : RUN;
+    constexpr bool FAST = sizeof(TO) == 2;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t0 = blockIdx.x * run;
+    int unit = blockIdx.y * PREP_WARPS + (threadIdx.x >> 5);
+    const int heads = 2 * p.G + p.H;
+    if (unit < heads) {
+        const int kind = unit < p.G ? 0 : unit < 2 * p.G ? 1 : 2;
+        conv_run<TI, KT, FAST, R>(p, t0, min(T, t0 + run), kind, kind < 2 ? unit * p.D : 2 * p.G * p.D + (unit - 2 * p.G) * p.DV, kind < 2 ? p.D : p.DV);
+        return;
+    }
+    unit -= heads;
+    if (t0 + unit % run < T) finish_tail<TI, TO>(p, t0 + unit % run, unit / run);
 }
 
 constexpr int SCAN_THREADS = 128, SCAN_COLS = 4;
@@ -402,11 +411,27 @@ PH_EXPORT int ph_delta_prepare(const void* rows, int rows_dtype, int splits, lon
     lanes_for(D, vec && D % 4 == 0, &p.qk_v, &p.qk_n);
     lanes_for(DV, vec && DV % 4 == 0 && (2LL * G * D) % 4 == 0, &p.v_v, &p.v_n);
     if (D > 512 || DV > 512) return fail(PH_ERR_UNSUPPORTED, "delta_prepare: heads of %d / %d exceed the supported 512", D, DV);
-    const int tail = H + (a_col >= 0 ? H : 0) + low_n + gate_n, run = T >= 512 ? RUN : 1;
-    const int units = 2 * G + H + (tail + TAIL - 1) / TAIL * run;
-    const dim3 grid((T + run - 1) / run, (units + PREP_WARPS - 1) / PREP_WARPS);
+    const int tail = H + (a_col >= 0 ? H : 0) + low_n + gate_n, parts = (tail + TAIL - 1) / TAIL;
+    if (p.qk_v == 4 && p.qk_n == 1 && p.v_v == 4 && p.v_n == 1 && K >= 2 && K <= 4) {
+        const int run = T >= RUN_FROM ? RUN : 1;
+        const dim3 grid((T + run - 1) / run, (2 * G + H + parts * run + PREP_WARPS - 1) / PREP_WARPS);
+#define LAUNCH_RUN(TI, TO, KT)                                                                               \
+    do {                                                                                                     \
+        if (run == 1) launch_overlapped(delta_prepare_run_kernel<TI, TO, KT, 1>, grid, dim3(PREP_WARPS * 32), 0, stream, p, T); \
+        else launch_overlapped(delta_prepare_run_kernel<TI, TO, KT, 4>, grid, dim3(PREP_WARPS * 32), 0, stream, p, T); \
+    } while (0)
+#define LAUNCH_K(TI, TO)                                                                                     \
+    do {                                                                                                     \
+        if (K == 2) LAUNCH_RUN(TI, TO, 2); else if (K == 3) LAUNCH_RUN(TI, TO, 3); else LAUNCH_RUN(TI, TO, 4); \
+    } while (0)
+        PH_DISPATCH(rows_dtype, TI, PH_DISPATCH(model_dtype, TO, LAUNCH_K(TI, TO)));
+#undef LAUNCH_K
+#undef LAUNCH_RUN
+        return check_launch("delta_prepare");
+    }
+    const dim3 grid(T, (2 * G + H + parts + PREP_WARPS - 1) / PREP_WARPS);
     PH_DISPATCH(rows_dtype, TI, PH_DISPATCH(model_dtype, TO,
-        launch_overlapped(delta_prepare_kernel<TI, TO>, grid, dim3(PREP_WARPS * 32), 0, stream, p, T, run)));
+        launch_overlapped(delta_prepare_kernel<TI, TO>, grid, dim3(PREP_WARPS * 32), 0, stream, p)));
     return check_launch("delta_prepare");
 }
 
