@@ -75,6 +75,11 @@ struct GemmParams {
     // sums (plain or with the activation), boxes of 64 columns; 2: float32 (whole or partial sums), boxes of 32 columns
     // of out seen as [splits][rows][columns].  0: the warps store.
     int tma_store;
+    // Pair kernel over several weights of rows_b rows each, one behind the other in w: the tile of 256 rows number i of A
+    // belongs to the weight tile_group[i], or to none (below zero: nothing is computed or stored).  row_factor ([rows_a] or
+    // null) multiplies the rows of the accumulator in front of the activation.
+    const int32_t* tile_group;
+    const float* row_factor;
     int* error_flag;
 };
 
@@ -205,6 +210,10 @@ __device__ __forceinline__ float plain_row_factor(const GemmParams& p, int a) {
     float s = 0.0f;
     for (int k = 0; k < p.row_chunks; ++k) s += p.row_sumsq[(size_t)a * p.row_chunks + k];
     return rsqrtf(s / (float)p.row_width + p.row_eps);
+}
+
+__device__ __forceinline__ float group_row_factor(const GemmParams& p, int a) {
+    return p.row_factor != nullptr && a < p.rows_a ? p.row_factor[a] : 1.0f;
 }
 
 // The gated activation of a (gate, up) pair, by the family the parameters name.
@@ -760,8 +769,9 @@ __device__ __forceinline__ void umma_commit_pair(uint64_t* bar) {
                  ::"r"(smem_u32(bar)), "h"((uint16_t)3) : "memory");
 }
 
-// ADDS: the instance for out += product (its epilogue keeps two chunks of out in registers); the other instance stores.
-template <bool ADDS>
+// ADDS: the instance for out += product (its epilogue keeps two chunks of out in registers); the other instances store.
+// GROUPED: the instance for several weights (tile_group).
+template <bool ADDS, bool GROUPED>
 __global__ void __launch_bounds__(PAIR_THREADS, 1)
 gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                          const __grid_constant__ CUtensorMap map_out, GemmParams p) {
@@ -805,6 +815,9 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
         kb1 = (int)((long long)p.kblocks * (split + 1) / p.splits);
     };
 
+    // which weight a tile belongs to, and whether it belongs to any: every role skips the same tiles
+    auto group_of = [&](int tile) { return GROUPED ? p.tile_group[tile % a_tiles] : 0; };
+
     pdl_launch_dependents();
     if (warp == 0) {
         if (lane == 0) {
@@ -813,8 +826,10 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
             uint32_t phase = 0;
             bool ok = true;
             for (int w = first; w < work_total && ok; w += stride) {
-                const int tile = w / p.splits;
-                const int a0 = (tile % a_tiles) * 2 * BM + (int)rank * BM, b0 = (tile / a_tiles) * PAIR_BN + (int)rank * PAIR_HALF;
+                const int tile = w / p.splits, group = group_of(tile);
+                if (group < 0) continue;
+                const int a0 = (tile % a_tiles) * 2 * BM + (int)rank * BM;
+                const int b0 = (tile / a_tiles) * PAIR_BN + (int)rank * PAIR_HALF + (GROUPED ? group * p.rows_b : 0);
                 int kb0, kb1;
                 k_range(w, kb0, kb1);
                 for (int kb = kb0; kb < kb1; ++kb) {
@@ -842,6 +857,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
             uint32_t phase = 0, acc_phase = 0;
             bool ok = true;
             for (int w = first; w < work_total && ok; w += stride) {
+                if (group_of(w / p.splits) < 0) continue;
                 if (!mbar_wait(&acc_empty[acc], acc_phase ^ 1, p.error_flag, PH_ERR_WAIT_MMA)) { ok = false; break; }
                 tc_fence_after();
                 const uint32_t d_addr = tmem_base + (uint32_t)(acc * PAIR_BN);
@@ -873,11 +889,12 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
         bool ok = true;
         for (int w = first; w < work_total && ok; w += stride) {
             const int tile = w / p.splits;
+            if (group_of(tile) < 0) continue;
             const int a0 = (tile % a_tiles) * 2 * BM + (int)rank * BM, b0 = (tile / a_tiles) * PAIR_BN;
             const size_t split_off = (size_t)(w % p.splits) * (size_t)p.split_stride;
             if (!ADDS && p.tma_store) {
                 const int a = a0 + q * 32 + lane;
-                const float row_f = p.row_sumsq != nullptr ? plain_row_factor(p, a) : 1.0f;   // fetched while the products run
+                const float row_f = GROUPED ? group_row_factor(p, a) : p.row_sumsq != nullptr ? plain_row_factor(p, a) : 1.0f;   // fetched while the products run
                 if (!mbar_wait(&acc_full[acc], acc_phase, p.error_flag, PH_ERR_WAIT_EPILOGUE)) { ok = false; break; }
                 tc_fence_after();
                 const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(acc * PAIR_BN);
@@ -954,8 +971,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
             if constexpr (ADDS) { if (vectors) load_accumulate_chunk(p, a0 + q * 32, lane, b0, c_first, old_next); }
             // ... and so is the factor of this thread's row
             const int a = a0 + q * 32 + lane;
-            const bool scale_row = !ADDS && p.row_sumsq != nullptr;       // a product that adds takes finished rows
-            const float row_f = scale_row ? plain_row_factor(p, a) : 1.0f;
+            const bool scale_row = !ADDS && (GROUPED ? p.row_factor != nullptr : p.row_sumsq != nullptr);       // a product that adds takes finished rows
+            const float row_f = !scale_row ? 1.0f : GROUPED ? group_row_factor(p, a) : plain_row_factor(p, a);
             if (!mbar_wait(&acc_full[acc], acc_phase, p.error_flag, PH_ERR_WAIT_EPILOGUE)) { ok = false; break; }
             tc_fence_after();
             const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(acc * PAIR_BN);
@@ -1103,8 +1120,9 @@ int launch_pair(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap&
                 cudaStream_t stream) {
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, PAIR_SMEM_BYTES) != cudaSuccess ||
-            cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, PAIR_SMEM_BYTES) != cudaSuccess)
+        if (cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, PAIR_SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, PAIR_SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, PAIR_SMEM_BYTES) != cudaSuccess)
             return fail(PH_ERR_LAUNCH, "gemm_tcgen05_pair: cannot reserve %d bytes of shared memory", PAIR_SMEM_BYTES);
         configured = true;
     }
@@ -1126,8 +1144,8 @@ int launch_pair(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap&
     attr[0].val.clusterDim.x = 2; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
-    if (p.accumulate) { if (cudaLaunchKernelEx(&cfg, gemm_tcgen05_pair_kernel<true>, ma, mb, mo, p) != cudaSuccess) {} }
-    else if (cudaLaunchKernelEx(&cfg, gemm_tcgen05_pair_kernel<false>, ma, mb, mo, p) != cudaSuccess) {}
+    auto kernel = p.accumulate ? gemm_tcgen05_pair_kernel<true, false> : p.tile_group ? gemm_tcgen05_pair_kernel<false, true> : gemm_tcgen05_pair_kernel<false, false>;
+    if (cudaLaunchKernelEx(&cfg, kernel, ma, mb, mo, p) != cudaSuccess) {}
     return check_launch("gemm_tcgen05_pair");
 }
 
@@ -1180,7 +1198,7 @@ PH_EXPORT int ph_gemm_bf16_tcgen05_pair(const void* x, const void* w, void* out,
     p.rows_a = M; p.rows_b = N; p.K = K;
     p.a_tiles = 0; p.b_tiles = (N + PAIR_BN - 1) / PAIR_BN; p.splits = splits; p.kblocks = kblocks;
     p.out = out; p.out_bf16 = out_dtype == PH_BF16; p.swapped = 0; p.swiglu = swiglu; p.gate_kind = gate ? (int)gate[3] : 0; p.gate_alpha = gate ? gate[0] : 1.0f; p.gate_limit = gate ? gate[1] : 0.0f; p.gate_shift = gate ? gate[2] : 0.0f; p.accumulate = accumulate; p.ld = swiglu ? N / 2 : N;
-    p.split_stride = (long long)M * N; p.error_flag = error_flag;
+    p.split_stride = (long long)M * N; p.error_flag = error_flag; p.tile_group = nullptr; p.row_factor = nullptr;
     p.row_sumsq = row_sumsq; p.row_chunks = row_chunks; p.row_width = row_width; p.row_eps = row_eps;
     p.norm_weight = norm_weight; p.norm_rows = (__nv_bfloat16*)norm_rows; p.norm_sumsq = norm_sumsq;
     // bfloat16 results of whole sums leave through the copy engine where its rules allow (rows of a multiple of 16 bytes)
@@ -1193,6 +1211,32 @@ PH_EXPORT int ph_gemm_bf16_tcgen05_pair(const void* x, const void* w, void* out,
              make_map_f32_out(&mo, out, M, N, splits))
         p.tma_store = 2;
     return launch_pair(ma, mb, mo, p, max_clusters, stream);
+}
+
+// Several products in one launch: x [M, K] in tiles of 256 rows, tile i times the weight tile_group[i] of w [groups, N, K] (a
+// device array of ceil(M / 256) numbers; below zero: the tile is left out, its rows of out untouched).  swiglu, gate and out
+// as above, out [M, N] or [M, N / 2]; row_factor [M] (or null): a factor per row in front of the activation.
+PH_EXPORT int ph_gemm_bf16_tcgen05_grouped(const void* x, const void* w, void* out, int out_dtype, int M, int N, int K, int groups,
+                                           const int32_t* tile_group, int swiglu, const float* gate, const float* row_factor, int* error_flag,
+                                           cudaStream_t stream) {
+    if (!x || !w || !out || !tile_group || !error_flag || M < 1 || N < 1 || K < 1 || groups < 1 || !valid_dtype(out_dtype))
+        return fail(PH_ERR_ARG, "gemm_tcgen05_grouped: bad arguments (M %d, N %d, K %d, groups %d)", M, N, K, groups);
+    if (K % 8) return fail(PH_ERR_UNSUPPORTED, "gemm_tcgen05_grouped: K = %d must be a multiple of 8 (16-byte rows for TMA)", K);
+    if (((uintptr_t)x | (uintptr_t)w) & 15) return fail(PH_ERR_UNSUPPORTED, "gemm_tcgen05_grouped: operands must be 16-byte aligned");
+    if (swiglu && (N & 1)) return fail(PH_ERR_ARG, "gemm_tcgen05_grouped: the SwiGLU epilogue needs an even N");
+    if ((long long)groups * N > 0x7fffffffLL) return fail(PH_ERR_UNSUPPORTED, "gemm_tcgen05_grouped: the weights have too many rows");
+    CUtensorMap ma, mb;
+    if (!make_map(&ma, x, M, K, BM) || !make_map(&mb, w, groups * N, K, PAIR_HALF))
+        return fail(PH_ERR_LAUNCH, "gemm_tcgen05_grouped: cuTensorMapEncodeTiled failed (rows %d / %d, K %d)", M, N, K);
+    GemmParams p = {};
+    p.rows_a = M; p.rows_b = N; p.K = K; p.b_tiles = (N + PAIR_BN - 1) / PAIR_BN; p.splits = 1; p.kblocks = (K + BK - 1) / BK;
+    p.out = out; p.out_bf16 = out_dtype == PH_BF16; p.swiglu = swiglu;
+    p.gate_kind = gate ? (int)gate[3] : 0; p.gate_alpha = gate ? gate[0] : 1.0f; p.gate_limit = gate ? gate[1] : 0.0f; p.gate_shift = gate ? gate[2] : 0.0f;
+    p.ld = swiglu ? N / 2 : N; p.split_stride = (long long)M * N; p.tile_group = tile_group; p.row_factor = row_factor; p.error_flag = error_flag;
+    CUtensorMap mo = ma;
+    if (out_dtype == PH_BF16 && p.ld % 8 == 0 && (((uintptr_t)out) & 15) == 0 && make_map(&mo, out, M, (int)p.ld, 32)) p.tma_store = 1;
+    else if (out_dtype == PH_F32 && !swiglu && N % 4 == 0 && (((uintptr_t)out) & 15) == 0 && make_map_f32_out(&mo, out, M, N, 1)) p.tma_store = 2;
+    return launch_pair(ma, mb, mo, p, 0, stream);
 }
 
 // out[M, N] (or float32 partials [splits][M, N]) = x[M, K] * w[N, K]^T.  swapped: the weight fills the 128-row
@@ -1243,7 +1287,7 @@ PH_EXPORT int ph_gemm_bf16_tcgen05(const void* x, const void* w, void* out, int 
     p.a_tiles = (rows_a + BM - 1) / BM; p.b_tiles = (rows_b + block_n - 1) / block_n;
     p.splits = splits; p.kblocks = kblocks;
     p.out = out; p.out_bf16 = out_dtype == PH_BF16; p.swapped = swapped; p.swiglu = swiglu; p.gate_kind = gate ? (int)gate[3] : 0; p.gate_alpha = gate ? gate[0] : 1.0f; p.gate_limit = gate ? gate[1] : 0.0f; p.gate_shift = gate ? gate[2] : 0.0f; p.accumulate = accumulate; p.ld = swiglu ? N / 2 : N;
-    p.split_stride = (long long)M * N; p.error_flag = error_flag;
+    p.split_stride = (long long)M * N; p.error_flag = error_flag; p.tile_group = nullptr; p.row_factor = nullptr;
     p.row_sumsq = row_sumsq; p.row_chunks = row_chunks; p.row_width = row_width; p.row_eps = row_eps;
     p.norm_weight = norm_weight; p.norm_rows = (__nv_bfloat16*)norm_rows; p.norm_sumsq = norm_sumsq;
     p.tma_store = 0;

@@ -215,6 +215,55 @@ __global__ void route_sort_kernel(const int32_t* __restrict__ choice, int R, int
     }
 }
 
+// One block.  The same with every expert's rows starting at a multiple of TILE_ROWS: position[pair], pair_at[row] (-1 where no
+// pair is), tile_expert[tile of TILE_ROWS rows] (-1 where no pair is), and factor[row] = weight[pair] (weight not null).
+constexpr int TILE_ROWS = 256, SORT_THREADS = 1024;
+__global__ void __launch_bounds__(SORT_THREADS) route_sort_tiles_kernel(const int32_t* __restrict__ choice, const float* __restrict__ weight, int R,
+                                                                        int E, int rows, int32_t* __restrict__ position,
+                                                                        int32_t* __restrict__ pair_at, int32_t* __restrict__ tile_expert,
+                                                                        float* __restrict__ factor) {
+    __shared__ int count[MAX_EXPERTS], offset[MAX_EXPERTS];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    for (int e = threadIdx.x; e < E; e += SORT_THREADS) count[e] = 0;
+    for (int i = threadIdx.x; i < rows; i += SORT_THREADS) pair_at[i] = -1;
+    __syncthreads();
+    const int all = (R + 31) / 32 * 32;
+    for (int i = threadIdx.x; i < all; i += SORT_THREADS) {           // whole warps: lanes with the same expert add as one
+        const int e = i < R ? choice[i] : -1;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        if (e >= 0 && lane == __ffs(same) - 1) atomicAdd(&count[e], __popc(same));
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int at = 0, tile = 0;
+        for (int e = 0; e < E; ++e) {
+            offset[e] = at;
+            const int tiles = (count[e] + TILE_ROWS - 1) / TILE_ROWS;
+            for (int k = 0; k < tiles; ++k) tile_expert[tile++] = e;
+            at += tiles * TILE_ROWS;
+            count[e] = 0;
+        }
+        for (; tile < rows / TILE_ROWS; ++tile) tile_expert[tile] = -1;
+    }
+    __syncthreads();
+    // which of an expert's places a pair gets is left to chance: a row's result does not depend on its place
+    for (int i = threadIdx.x; i < all; i += SORT_THREADS) {
+        const int e = i < R ? choice[i] : -1;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        const int first = __ffs(same) - 1;
+        int base = 0;
+        if (e >= 0 && lane == first) base = atomicAdd(&count[e], __popc(same));
+        base = __shfl_sync(0xffffffffu, base, first);
+        if (e < 0) continue;
+        const int at = offset[e] + base + __popc(same & ((1u << lane) - 1));
+        position[i] = at;
+        pair_at[at] = i;
+        if (factor) factor[at] = weight[i];
+    }
+}
+
 template <typename TX, typename TW, typename TY>
 __global__ void __launch_bounds__(256) gemm_grouped_kernel(const TX* __restrict__ x, const int32_t* __restrict__ pair_at,
                                                            int pairs_per_row, const TW* __restrict__ w,
@@ -337,7 +386,8 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_grouped_kernel(const TX* _
     }
 }
 
-// out[i] = x[token of the pair at sorted position i]: the rows of x in the order of the experts
+// out[i] = x[token of the pair at sorted position i]: the rows of x in the order of the experts (places without a pair, -1,
+// are left alone)
 template <typename TX>
 __global__ void route_gather_kernel(const TX* __restrict__ x, const int32_t* __restrict__ pair_at, int pairs_per_row,
                                     TX* __restrict__ out, int K, long long total) {
@@ -347,6 +397,7 @@ __global__ void route_gather_kernel(const TX* __restrict__ x, const int32_t* __r
     if (idx >= total) return;
     const long long i = idx / K;
     const int k = (int)(idx % K);
+    if (pair_at[i] < 0) return;
     out[idx] = x[(size_t)(pair_at[i] / pairs_per_row) * K + k];
 }
 // the same, 16 bytes per thread (vec = elements of 16 bytes; K a multiple of it)
@@ -360,6 +411,7 @@ __global__ void route_gather_vec_kernel(const TX* __restrict__ x, const int32_t*
     const int per_row = K / vec;
     const long long i = idx / per_row;
     const int k = (int)(idx % per_row) * vec;
+    if (pair_at[i] < 0) return;
     *reinterpret_cast<uint4*>(out + (size_t)i * K + k) =
         *reinterpret_cast<const uint4*>(x + (size_t)(pair_at[i] / pairs_per_row) * K + k);
 }
@@ -449,6 +501,21 @@ PH_EXPORT int ph_route_sort(const int32_t* choice, int R, int E, int32_t* positi
     launch_overlapped(route_sort_kernel, dim3(1), dim3(E < 256 ? 256 : 1024), 0, stream, choice, R, E, position, pair_at, tiles,
                       max_tiles, scratch);
     return check_launch("route_sort");
+}
+
+// Rows that route_sort_tiles may need for R pairs and E experts (a multiple of the tile's 256 rows).
+PH_EXPORT int ph_route_tile_rows(int R, int E) { return (int)(((long long)R + (long long)E * (TILE_ROWS - 1)) / TILE_ROWS) * TILE_ROWS; }
+
+// choice [R] -> position [R], pair_at [rows], tile_expert [rows / 256], factor [rows] (null: none) from weight [R]; rows =
+// ph_route_tile_rows(R, E).
+PH_EXPORT int ph_route_sort_tiles(const int32_t* choice, const float* weight, int R, int E, int rows, int32_t* position, int32_t* pair_at,
+                                  int32_t* tile_expert, float* factor, cudaStream_t stream) {
+    if (!choice || !position || !pair_at || !tile_expert || (factor && !weight) || R < 1 || E < 1 || rows < ph_route_tile_rows(R, E))
+        return fail(PH_ERR_ARG, "route_sort_tiles: bad arguments (pairs %d, experts %d, rows %d)", R, E, rows);
+    if (E > MAX_EXPERTS) return fail(PH_ERR_UNSUPPORTED, "route_sort_tiles: %d experts exceed the supported %d", E, MAX_EXPERTS);
+    launch_overlapped(route_sort_tiles_kernel, dim3(1), dim3(SORT_THREADS), 0, stream, choice, weight, R, E, rows, position, pair_at, tile_expert,
+                      factor);
+    return check_launch("route_sort_tiles");
 }
 
 // y [R, N] at the sorted positions; x rows are looked up through pair_at / pairs_per_row (null: x is already sorted);

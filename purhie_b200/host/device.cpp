@@ -169,6 +169,8 @@ const CoreKernels& core_kernels() {
     bind(h, "core", "ph_route", g_core.route);
     bind(h, "core", "ph_route_max_tiles", g_core.route_max_tiles);
     bind(h, "core", "ph_route_sort", g_core.route_sort);
+    bind(h, "core", "ph_route_tile_rows", g_core.route_tile_rows);
+    bind(h, "core", "ph_route_sort_tiles", g_core.route_sort_tiles);
     bind(h, "core", "ph_gemm_grouped", g_core.gemm_grouped);
     bind(h, "core", "ph_gemv_grouped", g_core.gemv_grouped);
     bind(h, "core", "ph_route_gather", g_core.route_gather);
@@ -235,6 +237,7 @@ const GemmKernels& gemm_kernels() {
     void* h = open_library("gemm100");
     bind(h, "gemm100", "ph_gemm_bf16_tcgen05", g_gemm.gemm);
     bind(h, "gemm100", "ph_gemm_bf16_tcgen05_pair", g_gemm.gemm_pair);
+    bind(h, "gemm100", "ph_gemm_bf16_tcgen05_grouped", g_gemm.gemm_experts);
     bind(h, "gemm100", "ph_gemm100_last_error", g_gemm.last_error);
     g_gemm_ok = true;
     return g_gemm;

@@ -143,6 +143,8 @@ struct CoreKernels {
                  float, const float*, float*, cudaStream_t);
     int (*route_max_tiles)(int, int);
     int (*route_sort)(const int32_t*, int, int, int32_t*, int32_t*, int32_t*, int, int32_t*, cudaStream_t);
+    int (*route_tile_rows)(int, int);          // the sort with every expert's rows at a multiple of the product's tile
+    int (*route_sort_tiles)(const int32_t*, const float*, int, int, int, int32_t*, int32_t*, int32_t*, float*, cudaStream_t);
     int (*gemm_grouped)(const void*, int, const int32_t*, int, const void*, int, const int32_t*, int, void*, int, int, int,
                         cudaStream_t);
     int (*gemv_grouped)(const void*, int, const int32_t*, int, const void*, int, const int32_t*, int, void*, int, int, int,
@@ -268,6 +270,9 @@ struct GemmKernels {
                 float, const float*, void*, float*, int*, cudaStream_t);
     int (*gemm_pair)(const void*, const void*, void*, int, int, int, int, int, int, int, const float*, int, const float*, int, int, float,
                      const float*, void*, float*, int*, cudaStream_t);
+    // several weights in one launch, a weight per tile of 256 rows
+    int (*gemm_experts)(const void*, const void*, void*, int, int, int, int, int, const int32_t*, int, const float*, const float*, int*,
+                        cudaStream_t);
     const char* (*last_error)(void);
 };
 

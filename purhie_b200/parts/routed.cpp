@@ -19,7 +19,11 @@
 // The (token, choice) pairs are sorted by expert on the device.  Which kernels then multiply:
 //   * few pairs (decoding): one launch per matrix of a kernel that streams each chosen expert's weight rows once
 //     (gemv_grouped); no count reaches the host, so the step is captured as a graph like any other;
-//   * a step with prompt portions in bfloat16: the counts per expert are read back (one small copy and a wait per
+//   * a step with prompt portions in bfloat16 and many rows per expert: the token rows are gathered in expert order, every
+//     expert's rows starting at a multiple of the tensor-core tile's 256, and each of the two products is one launch whose
+//     tiles know their expert (the gated activation, with a weight on the input, in the first one's epilogue); no count
+//     reaches the host;
+//   * with fewer rows per expert: the counts per expert are read back (one small copy and a wait per
 //     layer; such steps are launched kernel by kernel anyway), the token rows are gathered in expert order, and every
 //     expert's rows go through the tensor-core product as one contiguous slice;
 //   * float32, or shapes the fast kernels refuse: gemm_grouped, the CUDA-core product over row tiles that never cross
@@ -176,6 +180,48 @@ public:
                              (int)hidden_, top_, choice.as<int32_t>(), weight.as<float>(), scoring_,
                              correction_.defined() ? correction_.as<float>() : nullptr, groups_, keep_, weight_scale_,
                              shared_gate_.defined() ? shared_gate_.as<float>() : nullptr, shared_scale, ctx.stream));
+        const bool fast = !ctx.decode_only && R > kFewPairs && compute_dtype == DType::BF16 && x.dtype == DType::BF16 &&
+                          expert_gate_up_[0].fast() && expert_down_[0].fast() && hidden_ % 8 == 0 && inter_ % 8 == 0;
+        Tensor out = ws.get("moe_out", {T, hidden_}, DType::F32);
+        auto combine = [&](const Tensor& y, const Tensor& position) {
+            QE_LAUNCH(k, k.route_combine(y.data, y.code(), position.as<int32_t>(), weight_on_input_ ? nullptr : weight.as<float>(), T, top_,
+                                         (int)hidden_, out.as<float>(), always.tensor.defined() ? always.tensor.as<float>() : nullptr,
+                                         always.tensor.defined() ? always.splits : 0, (long long)T * hidden_,
+                                         always.tensor.defined() ? shared_scale : nullptr, ctx.stream));
+        };
+        if (fast && R >= kTileRowsPerExpert * experts_ && ctx.option("experts") != "slices") {
+            // every expert's rows at a multiple of the product's tile: one launch per product, nothing read back
+            const GemmKernels& g = gemm_kernels();
+            const int rows = k.route_tile_rows(R, experts_);
+            Tensor position = ws.get("moe_position", {R}, DType::I32), pair_at = ws.get("moe_pair_at", {rows}, DType::I32);
+            Tensor tile_expert = ws.get("moe_tile_expert", {rows / 256}, DType::I32);
+            Tensor factor = weight_on_input_ ? ws.get("moe_row_factor", {rows}, DType::F32) : Tensor();
+            QE_LAUNCH(k, k.route_sort_tiles(choice.as<int32_t>(), weight.as<float>(), R, experts_, rows, position.as<int32_t>(), pair_at.as<int32_t>(),
+                                            tile_expert.as<int32_t>(), weight_on_input_ ? factor.as<float>() : nullptr, ctx.stream));
+            Tensor xs = ws.get("moe_x_sorted", {rows, hidden_}, x.dtype);
+            if (LaunchProfile::get().on()) LaunchProfile::get().note_cost(2.0 * R * hidden_ * dtype_size(x.dtype), 0.0);
+            QE_LAUNCH(k, k.route_gather(x.data, x.code(), pair_at.as<int32_t>(), top_, xs.data, rows, (int)hidden_, ctx.stream));
+            float constants[4];
+            if (gated_) gate_.constants(constants);
+            Tensor act = ws.get("moe_act", {rows, inter_}, DType::BF16), first_out = act;
+            if (!gated_) first_out = ws.get("moe_gate_up", {rows, inter_}, DType::BF16);
+            auto note = [&](int64_t N, int64_t K, int64_t width, size_t es) {
+                if (LaunchProfile::get().on())
+                    LaunchProfile::get().note_cost(2.0 * experts_ * N * K + (double)R * (2.0 * K + width * es), 2.0 * R * N * K);
+            };
+            note(up_width_, hidden_, inter_, 2);
+            QE_LAUNCH(g, g.gemm_experts(xs.data, gate_up_.data, first_out.data, first_out.code(), rows, (int)up_width_, (int)hidden_, experts_,
+                                        tile_expert.as<int32_t>(), gated_ ? 1 : 0, gated_ && gate_.kind ? constants : nullptr,
+                                        weight_on_input_ ? factor.as<float>() : nullptr, ctx.gemm_error, ctx.stream));
+            if (!gated_)
+                QE_LAUNCH(k, k.unary_act(first_out.data, first_out.code(), 1, 0, act.data, act.code(), (long long)rows * inter_, unary_, ctx.stream));
+            Tensor y = ws.get("moe_down", {rows, hidden_}, DType::F32);
+            note(hidden_, inter_, hidden_, 4);
+            QE_LAUNCH(g, g.gemm_experts(act.data, down_.data, y.data, y.code(), rows, (int)hidden_, (int)inter_, experts_,
+                                        tile_expert.as<int32_t>(), 0, nullptr, nullptr, ctx.gemm_error, ctx.stream));
+            combine(y, position);
+            return Addend(out, 1);
+        }
         const int tiles = k.route_max_tiles(R, experts_);
         Tensor position = ws.get("moe_position", {R}, DType::I32), pair_at = ws.get("moe_pair_at", {R}, DType::I32);
         Tensor tile_list = ws.get("moe_tiles", {tiles, 3}, DType::I32), scratch = ws.get("moe_sort_scratch", {3 * experts_ + 1}, DType::I32);
@@ -184,8 +230,7 @@ public:
         Tensor gu = ws.get("moe_gate_up", {R, up_width_}, compute_dtype);
         Tensor act = ws.get("moe_act", {R, inter_}, compute_dtype);
         Tensor y = ws.get("moe_down", {R, hidden_}, DType::F32);
-        const bool slices = !ctx.decode_only && R > kFewPairs && compute_dtype == DType::BF16 && x.dtype == DType::BF16 &&
-                            expert_gate_up_[0].fast() && expert_down_[0].fast() && hidden_ % 8 == 0 && inter_ % 8 == 0;
+        const bool slices = fast;
         const bool few = !slices && R <= kFewPairs && hidden_ % 8 == 0 && inter_ % 8 == 0;
         auto grouped = [&](const Tensor& in, const int32_t* pairs, int per_row, const Tensor& w, Tensor& out, int64_t N, int64_t K) {
             if (LaunchProfile::get().on()) {     // the matrices of the experts that can have been chosen, the rows in and out
@@ -234,14 +279,12 @@ public:
         } else {
             grouped(act, nullptr, 1, down_, y, hidden_, inter_);
         }
-        Tensor out = ws.get("moe_out", {T, hidden_}, DType::F32);
-        QE_LAUNCH(k, k.route_combine(y.data, y.code(), position.as<int32_t>(), weight_on_input_ ? nullptr : weight.as<float>(), T, top_, (int)hidden_, out.as<float>(),
-                                     always.tensor.defined() ? always.tensor.as<float>() : nullptr, always.tensor.defined() ? always.splits : 0,
-                                     (long long)T * hidden_, always.tensor.defined() ? shared_scale : nullptr, ctx.stream));
+        combine(y, position);
         return Addend(out, 1);
     }
 
 private:
+    static constexpr int kTileRowsPerExpert = 96;       // from this many pairs per expert on average an expert's rows fill tiles of their own
     static constexpr int kFewPairs = 256;       // up to this many (token, choice) pairs a step streams the experts' rows
     int64_t hidden_, inter_;
     int experts_, top_;

@@ -473,6 +473,32 @@ def test_experts_take_their_weight_on_the_input(tmp_path, rows, dtype):
         close(got[clear], ref[clear], 2e-4 if dtype == "float32" else 3e-2)
 
 
+@pytest.mark.parametrize("weight_on", ["output", "input"])
+@pytest.mark.parametrize("activation", [None, {"kind": "clamped_swish", "alpha": 1.5, "limit": 1.0, "shift": 0.5}, {"kind": "gelu_tanh"}, "relu2"])
+def test_experts_with_tiles_of_their_own_give_a_row_what_it_gets_alone(activation, weight_on):
+    """bfloat16, hundreds of rows per expert (one launch per product over row tiles that know their expert) against the same
+    rows a few at a time (streamed weights); with a shared expert, and with experts that get no row at all."""
+    from purhie_b200.parts import PartProbe
+    gated = activation != "relu2"
+    if not gated and weight_on == "input":
+        pytest.skip("experts without a gate take their weight on the output")
+    E, width, ff = 6, 72, 40
+    for shared in (False, True):
+        unit = lambda stem: dict({"up_proj": stem + "up", "down_proj": stem + "down"}, **({"gate_proj": stem + "gate"} if gated else {}))
+        params = {"hidden_size": width, "intermediate_size": ff, "experts": E, "top": 2, "gated": gated, "activation": activation,
+                  "scoring": {"kind": "sigmoid"}, "weight_on": weight_on, "names": {"router": "r"}, "expert_names": [unit(f"e{e}.") for e in range(E)]}
+        if shared:
+            params["shared"] = {"kind": "swiglu" if gated else "mlp",
+                                "params": {"hidden_size": width, "intermediate_size": 24, "activation": activation, "names": unit("s.")}}
+        p = PartProbe("feed_forward", "routed_glu", params, dtype="bfloat16")
+        p.bind_random(7, 0.2)
+        x = inputs(700, width, 3, "bfloat16")
+        x[:, :16] = bf16_round(x[:, :16] + 2.0)                     # a common direction: some experts get most rows, some none
+        many = p.feed_forward(x)
+        few = np.concatenate([p.feed_forward(x[at:at + 100]) for at in range(0, 700, 100)])
+        close(many, few, 1.5e-2)
+
+
 def test_a_norm_whose_weight_is_stored_around_zero(tmp_path):
     from purhie_b200.parts import PartProbe
     cfg = config(24, 20, [(channel(1, 1, 4, 4, 1, 2, 2), None)])
@@ -501,7 +527,7 @@ def test_rotation_tables_follow_the_wavelengths():
 # ---- kernels' own choices inside whole models --------------------------------------------------------------------------
 def test_key_splits_and_kernel_choices_agree_with_the_plain_implementation(models):
     from purhie_b200.engine import StepEntry
-    for name, choices in (("C", [{}, {"tile16_splits": 3}, {"delta": "scan"}]),
+    for name, choices in (("C", [{}, {"tile16_splits": 3}, {"delta": "scan"}, {"experts": "slices"}]),
                           ("D", [{"decode_splits": 3, "prefill_splits": 2}, {"decode_splits": 8, "prefill_splits": 5}, {"sink_kernel": "tile"}])):
         folder, cfg, w = models[name, "bfloat16"]
         toks = tokens(300, cfg["vocab"], 6)
