@@ -482,8 +482,8 @@ def test_experts_with_tiles_of_their_own_give_a_row_what_it_gets_alone(activatio
     gated = activation != "relu2"
     if not gated and weight_on == "input":
         pytest.skip("experts without a gate take their weight on the output")
-    E, width, ff = 6, 72, 40
-    for shared in (False, True):
+    # (the second case: several tiles of features, several blocks of K, more tiles than the device holds at a time)
+    for E, width, ff, rows, shared in ((6, 72, 40, 700, False), (6, 72, 40, 700, True), (5, 576, 328, 4000, activation is None)):
         unit = lambda stem: dict({"up_proj": stem + "up", "down_proj": stem + "down"}, **({"gate_proj": stem + "gate"} if gated else {}))
         params = {"hidden_size": width, "intermediate_size": ff, "experts": E, "top": 2, "gated": gated, "activation": activation,
                   "scoring": {"kind": "sigmoid"}, "weight_on": weight_on, "names": {"router": "r"}, "expert_names": [unit(f"e{e}.") for e in range(E)]}
@@ -492,10 +492,10 @@ def test_experts_with_tiles_of_their_own_give_a_row_what_it_gets_alone(activatio
                                 "params": {"hidden_size": width, "intermediate_size": 24, "activation": activation, "names": unit("s.")}}
         p = PartProbe("feed_forward", "routed_glu", params, dtype="bfloat16")
         p.bind_random(7, 0.2)
-        x = inputs(700, width, 3, "bfloat16")
+        x = inputs(rows, width, 3, "bfloat16")
         x[:, :16] = bf16_round(x[:, :16] + 2.0)                     # a common direction: some experts get most rows, some none
         many = p.feed_forward(x)
-        few = np.concatenate([p.feed_forward(x[at:at + 100]) for at in range(0, 700, 100)])
+        few = np.concatenate([p.feed_forward(x[at:at + 100]) for at in range(0, rows, 100)])
         close(many, few, 1.5e-2)
 
 
